@@ -1,7 +1,10 @@
 // ctd_generate: the reference's token generation subprocess (emberlm tools/ctd_generate/main.cpp) on
 // the B200 decode path.
 //
-//   ctd_generate --model <path-to-fp32.safetensors>
+//   ctd_generate --model <path-to-fp32.safetensors | model folder> [--precision fp32|tf32|bf16]
+//
+// A folder with a layer-list config.json (served_model.hpp) is served through the same protocol, loop and
+// sampler; it runs in bf16 unless --precision fp32 is given.
 //
 // Protocol as there: one JSON request on stdin ({"input_ids": [...], "max_new_tokens", "max_seq_len",
 // "temperature", "top_k", "top_p", "seed", "eos_ids", "thinking_token_budget", "think_open_ids",
@@ -28,22 +31,9 @@
 
 #include <cuda_runtime.h>
 
-#include "../../include/ctdk.h"
-#include "../../include/ctdk_util/minijson.hpp"
-#include "model_desc.hpp"
-#include "../../include/ctdk_util/safetensors.hpp"
+#include "served_model.hpp"
 
 namespace {
-
-#define CUDA_OK(expr)                                                                          \
-  do {                                                                                         \
-    const cudaError_t e_ = (expr);                                                             \
-    if (e_ != cudaSuccess) throw std::runtime_error(std::string(#expr) + ": " + cudaGetErrorString(e_)); \
-  } while (0)
-#define CTDK_OK_OR_THROW(expr)                                                     \
-  do {                                                                             \
-    if ((expr) != CTDK_OK) throw std::runtime_error(std::string(ctdk_last_error())); \
-  } while (0)
 
 struct Sampler {
   float temperature = 1.0f;
@@ -65,7 +55,7 @@ std::string parse_model_path(int argc, char** argv) {
   for (int i = 1; i < argc; ++i)
     if (std::string(argv[i]) == "--model" && i + 1 < argc) model = argv[++i];
   if (model.empty()) {
-    std::cerr << "usage: " << argv[0] << " --model <path-to-fp32.safetensors> [--precision fp32|tf32]\n";
+    std::cerr << "usage: " << argv[0] << " --model <path-to-fp32.safetensors | model folder> [--precision fp32|tf32|bf16]\n";
     std::exit(2);
   }
   return model;
@@ -74,16 +64,18 @@ std::string parse_model_path(int argc, char** argv) {
 // The prompt pass: exact fp32 products by default, like the reference's generator (the token steps are
 // fp32 GEMVs in either case), so that a request draws the same tokens; --precision tf32 runs the prompt
 // on the TF32 tensor cores (long prompts, where a rounding difference of 1e-3 in the cache is acceptable).
-int parse_precision(int argc, char** argv) {
+// Layer-list models run in bf16 unless fp32 is asked for.
+cli::Precision parse_precision(int argc, char** argv) {
   for (int i = 1; i + 1 < argc; ++i)
     if (std::string(argv[i]) == "--precision") {
       const std::string v = argv[i + 1];
-      if (v == "tf32") return CTDK_GEMM_TF32;
-      if (v == "fp32" || v == "3xtf32") return CTDK_GEMM_3XTF32;
-      std::cerr << "--precision: expected fp32 or tf32\n";
+      if (v == "tf32") return cli::Precision::kTf32;
+      if (v == "bf16") return cli::Precision::kBf16;
+      if (v == "fp32" || v == "3xtf32") return cli::Precision::kFp32;
+      std::cerr << "--precision: expected fp32, tf32 or bf16\n";
       std::exit(2);
     }
-  return CTDK_GEMM_3XTF32;
+  return cli::Precision::kDefault;
 }
 
 }  // namespace
@@ -110,26 +102,13 @@ int main(int argc, char** argv) try {
 
   const auto t0 = std::chrono::steady_clock::now();
   std::cerr << "[ctd_generate] loading " << model_path << "\n";
-  st::File wfile(model_path);
-  const st::Entry& emb = wfile.entry("model.embed_tokens.weight");
-  if (emb.shape.size() != 2) throw std::runtime_error("autodetect_config: model.embed_tokens.weight must be 2-D");
-  ctdk_model_config mc = cli::autodetect_config(emb.shape[0], emb.shape[1]);
-  mc.precision = parse_precision(argc, argv);
-  std::cerr << "[ctd_generate] arch: hidden=" << mc.hidden_size << " layers=" << mc.num_hidden_layers << "\n";
+  const cli::ServedModel model(model_path, parse_precision(argc, argv));
+  std::cerr << "[ctd_generate] arch: " << model.summary() << "\n";
   const int prompt_len = static_cast<int>(input_ids.size());
   for (const int64_t id : input_ids)
-    if (id < 0 || id >= mc.vocab_size) throw std::runtime_error("input_ids: token id out of range");
-
-  int64_t arena = 0;
-  const std::vector<cli::ParamDesc> params = cli::describe_parameters(mc, &arena);
-  std::vector<float> h_arena(static_cast<size_t>(arena), 0.0f);
-  for (const auto& p : params) wfile.read_f32(p.name, h_arena.data() + p.offset, p.numel);
-  CUDA_OK(cudaSetDevice(0));
+    if (id < 0 || id >= model.vocab()) throw std::runtime_error("input_ids: token id out of range");
   cudaStream_t stream;
   CUDA_OK(cudaStreamCreate(&stream));
-  float* d_params = nullptr;
-  CUDA_OK(cudaMalloc(reinterpret_cast<void**>(&d_params), arena * sizeof(float)));
-  CUDA_OK(cudaMemcpy(d_params, h_arena.data(), arena * sizeof(float), cudaMemcpyHostToDevice));
   std::cerr << "[ctd_generate] model ready in " << std::chrono::duration<double>(std::chrono::steady_clock::now() - t0).count()
             << " s\n";
 
@@ -142,22 +121,19 @@ int main(int argc, char** argv) try {
     return 0;
   }
 
-  const int64_t ws_bytes = ctdk_decode_workspace_bytes(&mc, max_seq);
-  if (ws_bytes < 0) throw std::runtime_error(ctdk_last_error());
-  void* d_ws = nullptr;
-  CUDA_OK(cudaMalloc(&d_ws, static_cast<size_t>(ws_bytes)));
-  void* dec = nullptr;
-  CTDK_OK_OR_THROW(ctdk_decode_create(&mc, d_params, d_ws, ws_bytes, max_seq, &dec));
+  cli::ServedModel::Sequence sequence;
+  model.make_sequence(max_seq, &sequence);
+  void* dec = sequence.decoder;
   int64_t* d_ids = nullptr;
   CUDA_OK(cudaMalloc(reinterpret_cast<void**>(&d_ids), static_cast<size_t>(std::max(max_seq, 16)) * sizeof(int64_t)));
   CUDA_OK(cudaMemcpy(d_ids, input_ids.data(), static_cast<size_t>(prompt_len) * sizeof(int64_t), cudaMemcpyHostToDevice));
   const auto t1 = std::chrono::steady_clock::now();
-  CTDK_OK_OR_THROW(ctdk_decode_prefill(dec, d_ids, prompt_len, stream));
+  cli::ctdk_ok(ctdk_decode_prefill(dec, d_ids, prompt_len, stream));
   CUDA_OK(cudaStreamSynchronize(stream));
   std::cerr << "[ctd_generate] prefill (" << prompt_len << " tok) in "
             << std::chrono::duration<double>(std::chrono::steady_clock::now() - t1).count() << " s\n";
 
-  const int64_t V = mc.vocab_size;
+  const int64_t V = model.vocab();
   std::mt19937_64 rng(seed);
   int generated = 0;
   std::string stop = "max_tokens";
@@ -174,7 +150,7 @@ int main(int argc, char** argv) try {
         stop = "max_seq_len";
         break;
       }
-      CTDK_OK_OR_THROW(ctdk_decode_greedy(dec, n, d_ids, stream));
+      cli::ctdk_ok(ctdk_decode_greedy(dec, n, d_ids, stream));
       CUDA_OK(cudaMemcpyAsync(chunk.data(), d_ids + generated, static_cast<size_t>(n) * sizeof(int64_t), cudaMemcpyDeviceToHost, stream));
       CUDA_OK(cudaStreamSynchronize(stream));
       for (int i = 0; i < n; ++i) {
@@ -196,7 +172,7 @@ int main(int argc, char** argv) try {
     // Sampling on the device (ctdk_sample: the reference sampler's semantics and draw order): the
     // uniform draw goes there, the token id comes back; the V logits never leave the GPU.
     const float* d_logits = nullptr;
-    CTDK_OK_OR_THROW(ctdk_decode_logits(dec, &d_logits));
+    cli::ctdk_ok(ctdk_decode_logits(dec, &d_logits));
     void* d_sample_ws = nullptr;
     double* d_u = nullptr;
     int64_t* d_tok = nullptr;
@@ -220,7 +196,7 @@ int main(int argc, char** argv) try {
       } else {
         const double u = sampler.temperature > 0.0f ? uniform(rng) : 0.0;   // greedy takes no draw (sampling.cpp:33)
         CUDA_OK(cudaMemcpyAsync(d_u, &u, sizeof u, cudaMemcpyHostToDevice, stream));
-        CTDK_OK_OR_THROW(ctdk_sample(d_logits, 1, V, sampler.temperature, sampler.top_k, sampler.top_p, d_u, d_sample_ws, d_tok, stream));
+        cli::ctdk_ok(ctdk_sample(d_logits, 1, V, sampler.temperature, sampler.top_k, sampler.top_p, d_u, d_sample_ws, d_tok, stream));
         CUDA_OK(cudaMemcpyAsync(&tok, d_tok, sizeof tok, cudaMemcpyDeviceToHost, stream));
         CUDA_OK(cudaStreamSynchronize(stream));
       }
@@ -247,7 +223,7 @@ int main(int argc, char** argv) try {
         stop = "max_seq_len";
         break;
       }
-      CTDK_OK_OR_THROW(ctdk_decode_step(dec, tok, stream));
+      cli::ctdk_ok(ctdk_decode_step(dec, tok, stream));
       ++fed;
     }
     CUDA_OK(cudaStreamSynchronize(stream));
@@ -259,7 +235,6 @@ int main(int argc, char** argv) try {
   std::cerr << "[ctd_generate] generated " << generated << " tok in " << decode_s << " s  ("
             << (generated / std::max(decode_s, 1e-9)) << " tok/s)\n";
   emit(minijson::Line().add_bool("done", true).add("reason", stop).add("generated_tokens", static_cast<long long>(generated)).dump());
-  ctdk_decode_destroy(dec);
   return 0;
 } catch (const std::exception& e) {
   std::cerr << "[ctd_generate] error: " << e.what() << "\n";

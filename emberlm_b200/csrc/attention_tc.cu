@@ -67,6 +67,9 @@ struct FwdArgs {
   int T, H, Hk, B;
   int n_qtiles;   // ceil(T / 128)
   int n_items;    // n_qtiles * H * B
+  // Only query rows [row_lo, row_hi) of the flattened [B, T] rows are wanted, and rows from row_hi on
+  // hold no keys: tiles outside are skipped (everything: 0 and B * T).
+  int64_t row_lo, row_hi;
   float scale_log2;
   int* status;
 };
@@ -82,7 +85,7 @@ constexpr float kRescaleSlack = 8.0f;
 // run fastest (the query heads of one key/value group sit side by side). CTA c takes items
 // c, c + gridDim.x, ...
 struct FwdItem {
-  int qi, h, b, q0, n_steps;
+  int qi, h, b, q0, n_steps;   // n_steps 0: no wanted row in this tile
 };
 __device__ __forceinline__ FwdItem fwd_item(const FwdArgs& a, int it) {
   FwdItem w;
@@ -93,7 +96,10 @@ __device__ __forceinline__ FwdItem fwd_item(const FwdArgs& a, int it) {
   w.h = r % a.H;
   w.q0 = w.qi * TQ;
   // key steps up to and including the diagonal, never past the end of the sequence
-  w.n_steps = min((w.q0 + TQ) / TK, (a.T + TK - 1) / TK);
+  const int64_t base = static_cast<int64_t>(w.b) * a.T;
+  const int rows = static_cast<int>(min(static_cast<int64_t>(a.T), a.row_hi - base));   // of this sequence; may be <= 0
+  w.n_steps = min((w.q0 + TQ) / TK, (rows + TK - 1) / TK);
+  if (w.q0 >= rows || base + w.q0 + TQ <= a.row_lo) w.n_steps = 0;
   return w;
 }
 
@@ -164,11 +170,13 @@ __global__ void __launch_bounds__(192, FwdCfg<D>::kCtasPerSm)
     if (lane == 0) {
       uint32_t g0 = 0, n_it = 0;
       bool ok = true;
-      for (int it = blockIdx.x; it < args.n_items && ok; it += gridDim.x, ++n_it) {
+      for (int it = blockIdx.x; it < args.n_items && ok; it += gridDim.x) {
         const FwdItem w = fwd_item(args, it);
+        if (w.n_steps <= 0) continue;
         const int hk = w.h / (args.H / args.Hk);
         const int col_q = w.h * D, col_k = (args.H + hk) * D, col_v = (args.H + args.Hk + hk) * D;
         if (!mbar_wait_bounded(q_empty, (n_it & 1u) ^ 1u, args.status, 10)) break;
+        ++n_it;
         mbar_expect_tx(q_full, C::kQBytes);
 #pragma unroll
         for (int c = 0; c < NC; ++c) tma_load_3d(q_s + c * kQChunk, &tm_q, q_full, col_q + 32 * c, w.q0, w.b);
@@ -210,8 +218,9 @@ __global__ void __launch_bounds__(192, FwdCfg<D>::kCtasPerSm)
       const uint64_t qd_ = make_smem_desc(smem_u32(q_s), 16, 1024, kLayoutSw128);
       uint32_t g0 = 0, n_it = 0;
       bool ok = true;
-      for (int it = blockIdx.x; it < args.n_items && ok; it += gridDim.x, ++n_it) {
+      for (int it = blockIdx.x; it < args.n_items && ok; it += gridDim.x) {
         const FwdItem w = fwd_item(args, it);
+        if (w.n_steps <= 0) continue;
         auto issue_s = [&](int j) {
           const uint32_t g = g0 + static_cast<uint32_t>(j), s = g & 1u;
           {
@@ -231,6 +240,7 @@ __global__ void __launch_bounds__(192, FwdCfg<D>::kCtasPerSm)
         };
         {
           if (!mbar_wait_bounded_w(q_full, n_it & 1u, args.status, 21)) break;
+          ++n_it;
         }
         tc_fence_after();
         // Tensor-pipe order: S(0) S(1) | PV(0) S(2) | PV(1) S(3) | ... S(j+2) reuses the columns
@@ -274,8 +284,9 @@ __global__ void __launch_bounds__(192, FwdCfg<D>::kCtasPerSm)
     const uint32_t to = tm_o + lane_off;
     uint32_t g0 = 0, n_done = 0;
     bool ok = true;
-    for (int it = blockIdx.x; it < args.n_items && ok; it += gridDim.x, ++n_done) {
+    for (int it = blockIdx.x; it < args.n_items && ok; it += gridDim.x) {
       const FwdItem w = fwd_item(args, it);
+      if (w.n_steps <= 0) continue;
       const int row = w.q0 + qd * 32 + lane;   // query position inside the sequence
       float m_ref = 0.0f, l_run = 0.0f;
       for (int j = 0; j < w.n_steps && ok; ++j) {
@@ -352,6 +363,7 @@ __global__ void __launch_bounds__(192, FwdCfg<D>::kCtasPerSm)
       // threads have read O and arrived at its p_ready.
       {
         if (!ok || !mbar_wait_bounded(o_full, n_done & 1u, args.status, 33)) { ok = false; break; }
+        ++n_done;
       }
       tc_fence_after();
       // Normalised output rows go through a small per-warp staging area (16 rows x 32 floats,
@@ -391,7 +403,7 @@ __global__ void __launch_bounds__(192, FwdCfg<D>::kCtasPerSm)
         }
       }
       tc_fence_before();
-      if (row < args.T)
+      if (args.lse != nullptr && row < args.T)
         args.lse[(static_cast<int64_t>(w.b) * args.H + w.h) * args.T + row] = (m_ref + log2f(l_run)) * kLn2f;
     }
   }
@@ -459,10 +471,46 @@ int attn_fwd_tcgen05(const float* qkv, float* out, float* lse, int64_t B, int64_
   const int64_t items = static_cast<int64_t>(a.n_qtiles) * H * B;
   if (items > INT32_MAX) return 1;
   a.n_items = static_cast<int>(items);
+  a.row_lo = 0;
+  a.row_hi = B * T;
   a.scale_log2 = (1.0f / sqrtf(static_cast<float>(D))) * 1.4426950408889634f;
   a.status = device_status_word();
   if (a.status == nullptr) return fail(CTDK_ELAUNCH, "attn_fwd(tcgen05): no status word");
   // persistent CTAs: as many as fit on the device at once
+  const int64_t slots = static_cast<int64_t>(sm_budget()) * (D == 64 ? 2 : 1);
+  dim3 grid(static_cast<unsigned>(items < slots ? items : slots));
+  return D == 64 ? launch_fwd<64>(tq, tk, tv, a, grid, stream) : launch_fwd<128>(tq, tk, tv, a, grid, stream);
+}
+
+// Chunked causal attention over `rows` packed rows [rows, (H + 2 Hk) * D] that start at a chunk's
+// first position: a row sees the rows up to itself inside its own `chunk`-long chunk, so the chunks are
+// the sequences of the kernel above. Only rows >= first are queries (rows before it carry cached keys
+// and values only). The buffers hold whole chunks (rows rounded up to a multiple of `chunk`), and rows
+// past the end contain finite values. D is 64 or 128; scores are multiplied by `scale`.
+int attn_chunked_tcgen05(const float* qkv, float* out, int64_t rows, int64_t first, int64_t chunk, int H, int Hk, int D,
+                         float scale, cudaStream_t stream) {
+  CTDK_REQUIRE(rows > 0 && first >= 0 && first < rows && chunk > 0 && (D == 64 || D == 128), "attn_chunked: bad shape");
+  const int RS = (H + 2 * Hk) * D;
+  const int64_t B = (rows + chunk - 1) / chunk;
+  CUtensorMap tq, tk, tv;
+  const int rc = make_qkv_maps(qkv, B, chunk, RS, &tq, &tk, &tv);
+  if (rc != CTDK_OK) return rc;
+  FwdArgs a;
+  a.out = out;
+  a.lse = nullptr;
+  a.T = static_cast<int>(chunk);
+  a.H = H;
+  a.Hk = Hk;
+  a.B = static_cast<int>(B);
+  a.n_qtiles = static_cast<int>((chunk + TQ - 1) / TQ);
+  const int64_t items = static_cast<int64_t>(a.n_qtiles) * H * B;
+  CTDK_REQUIRE(items <= INT32_MAX, "attn_chunked: too many tiles");
+  a.n_items = static_cast<int>(items);
+  a.row_lo = first;
+  a.row_hi = rows;
+  a.scale_log2 = scale * 1.4426950408889634f;
+  a.status = device_status_word();
+  if (a.status == nullptr) return fail(CTDK_ELAUNCH, "attn_chunked: no status word");
   const int64_t slots = static_cast<int64_t>(sm_budget()) * (D == 64 ? 2 : 1);
   dim3 grid(static_cast<unsigned>(items < slots ? items : slots));
   return D == 64 ? launch_fwd<64>(tq, tk, tv, a, grid, stream) : launch_fwd<128>(tq, tk, tv, a, grid, stream);

@@ -18,7 +18,7 @@
 #include <algorithm>
 #include <cstdlib>
 
-#include "common.cuh"
+#include "decode_core.h"
 
 namespace ctdk {
 namespace {
@@ -274,65 +274,6 @@ __global__ void __launch_bounds__(128)
   }
 }
 
-// First index of the maximum (the reference's greedy sampler, src/core/sampling.cpp:13-20) over
-// many CTAs: each reduces its share of the logits and folds (value, index) into one 64-bit word
-// with atomicMax. The key orders floats as unsigned integers in the high half and prefers the
-// smaller index in the low half; argmax_finish_kernel turns the word into the next input token.
-__device__ __forceinline__ unsigned long long argmax_key(float v, int idx) {
-  unsigned u = __float_as_uint(v);
-  u = (u & 0x80000000u) ? ~u : (u | 0x80000000u);
-  return (static_cast<unsigned long long>(u) << 32) | (0xFFFFFFFFu - static_cast<unsigned>(idx));
-}
-__global__ void __launch_bounds__(256)
-    argmax_kernel(const float* __restrict__ logits, int V, unsigned long long* __restrict__ word) {
-  __shared__ unsigned long long best_s[8];
-  pdl_launch();
-  pdl_wait();
-  unsigned long long best = 0ull;
-  for (int i = blockIdx.x * blockDim.x + threadIdx.x; i < V; i += gridDim.x * blockDim.x) {
-    const unsigned long long k = argmax_key(logits[i], i);
-    best = k > best ? k : best;
-  }
-#pragma unroll
-  for (int o = 16; o > 0; o >>= 1) {
-    const unsigned long long other = __shfl_xor_sync(0xffffffffu, best, o);
-    best = other > best ? other : best;
-  }
-  const int lane = threadIdx.x & 31, wid = threadIdx.x >> 5;
-  if (lane == 0) best_s[wid] = best;
-  __syncthreads();
-  if (threadIdx.x == 0) {
-    for (int i = 1; i < (blockDim.x >> 5); ++i) best = best_s[i] > best ? best_s[i] : best;
-    atomicMax(word, best);
-  }
-}
-// Stores the winning token as the next input, appends it to out_tokens[*count], clears the word and
-// advances the counters (pos may point at a scratch int when the position must not move).
-__global__ void argmax_finish_kernel(unsigned long long* word, int64_t* cur_token, int64_t* out_tokens, int* pos,
-                                     int* count) {
-  pdl_launch();
-  pdl_wait();
-  const int64_t idx = static_cast<int64_t>(0xFFFFFFFFu - static_cast<unsigned>(*word & 0xFFFFFFFFull));
-  *cur_token = idx;
-  if (out_tokens != nullptr) out_tokens[*count] = idx;
-  *word = 0ull;
-  *pos += 1;
-  *count += 1;
-}
-
-__global__ void bump_kernel(int* pos, int* count) {
-  pdl_launch();
-  pdl_wait();
-  *pos += 1;
-  *count += 1;
-}
-__global__ void set_counters_kernel(int* pos, int* count, int p, int c) {
-  *pos = p;
-  *count = c;
-  *reinterpret_cast<unsigned long long*>(pos + 4) = 0ull;   // the argmax word lives behind the counters
-}
-
-
 // ----------------------------------------------------------------------------------------
 // Persistent token loop. The kernel-per-phase path above spends most of a token in the ~200
 // launch-to-launch dependencies (each kernel streams 8-25 MB of weights in 2-4 us but waits ~8 us
@@ -371,55 +312,6 @@ struct PersistArgs {
   int* status;
 };
 
-__device__ __forceinline__ unsigned int ld_acquire_u32(const unsigned int* p) {
-  unsigned int v;
-  asm volatile("ld.acquire.gpu.global.u32 %0, [%1];" : "=r"(v) : "l"(p) : "memory");
-  return v;
-}
-__device__ __forceinline__ void prefetch_l2(const void* p) { asm volatile("prefetch.global.L2 [%0];" ::"l"(p)); }
-
-// All CTAs of the grid meet here: one release reduction on a counter per CTA (no value comes back,
-// so the arriving thread does not wait for it; the CTA's earlier writes are ordered before it by
-// the bar.sync and the release), then one thread per CTA polls the counter. A flag per CTA watched
-// by every other CTA measured twice as slow (all pollers hit the same few L2 lines). `epoch` counts
-// the barriers this CTA has passed. Returns false once any CTA has given up (the abort flag is
-// set): the caller unwinds.
-__device__ __forceinline__ bool grid_barrier(const PersistArgs& a, unsigned int& epoch) {
-  __shared__ int s_ok;
-  __syncthreads();
-  if (threadIdx.x == 0) {
-    ++epoch;
-    const unsigned int target = epoch * gridDim.x;
-    asm volatile("red.release.gpu.global.add.u32 [%0], 1;" ::"l"(&a.sync[0]) : "memory");
-    int ok = 1;
-    if (ld_acquire_u32(&a.sync[0]) < target) {
-      const uint64_t t0 = globaltimer_ns();
-      unsigned int spins = 0;
-      while (ld_acquire_u32(&a.sync[0]) < target) {
-        if ((++spins & 0xffu) == 0u) {
-          if (ld_acquire_u32(&a.sync[2]) != 0u) {   // someone else gave up
-            ok = 0;
-            break;
-          }
-          if (globaltimer_ns() - t0 > kWaitBudgetNs) {
-            if (atomicCAS(a.status, 0, CTDK_ETIMEOUT) == 0) {
-              a.status[1] = 90;
-              a.status[2] = static_cast<int>(blockIdx.x);
-              a.status[3] = static_cast<int>(epoch);
-            }
-            atomicExch(&a.sync[2], 1u);
-            ok = 0;
-            break;
-          }
-        }
-      }
-    }
-    if (ok && ld_acquire_u32(&a.sync[2]) != 0u) ok = 0;
-    s_ok = ok;
-  }
-  __syncthreads();
-  return s_ok != 0;
-}
 // Rows n = first, first + step, ... of W[N, K] for this warp when WPR warps of a CTA share a row.
 template <int WPR>
 __device__ __forceinline__ void row_walk(int& first, int& step) {
@@ -544,7 +436,7 @@ __global__ void __launch_bounds__(256, 2) decode_persistent_kernel(const __grid_
       stage_rmsnorm(xin, a.P + w.w_in, a.eps, hid, sm, red);
       gemv_rows<1>(a.P + w.wq, sm, a.qkv, nullptr, a.QKVN, hid, pair_red);
       prefetch_rows<2>(a.P + w.wo, hid, H * D);
-      if (!(alive = grid_barrier(a, epoch))) break;
+      if (!(alive = grid_barrier(a.sync, a.status, 90, epoch))) break;
 
       // ---- phase 2: attention of the new row, split over key ranges; the last split of a head merges ----
       {
@@ -700,20 +592,20 @@ __global__ void __launch_bounds__(256, 2) decode_persistent_kernel(const __grid_
         }
       }
       prefetch_rows<1>(a.P + w.wg, 2 * I, hid);
-      if (!(alive = grid_barrier(a, epoch))) break;
+      if (!(alive = grid_barrier(a.sync, a.status, 90, epoch))) break;
 
       // ---- phase 3: hm = x + Wo attn ----
       for (int i = threadIdx.x; i < H * D; i += blockDim.x) sm[i] = __ldcg(a.attn + i);
       __syncthreads();
       gemv_rows<2>(a.P + w.wo, sm, a.hm, xin, hid, H * D, pair_red);
       prefetch_rows<2>(a.P + w.wd, hid, I);
-      if (!(alive = grid_barrier(a, epoch))) break;
+      if (!(alive = grid_barrier(a.sync, a.status, 90, epoch))) break;
 
       // ---- phase 4: gu = Wgu rmsnorm(hm) ----
       stage_rmsnorm(a.hm, a.P + w.w_post, a.eps, hid, sm, red);
       gemv_rows<1>(a.P + w.wg, sm, a.gu, nullptr, 2 * I, hid, pair_red);
       if (l + 1 < a.L) prefetch_rows<1>(a.P + a.lw[l + 1].wq, a.QKVN, hid);
-      if (!(alive = grid_barrier(a, epoch))) break;
+      if (!(alive = grid_barrier(a.sync, a.status, 90, epoch))) break;
 
       // ---- phase 5: x = hm + Wd (silu(gate) * up) ----
       for (int i = threadIdx.x; i < I; i += blockDim.x) {
@@ -722,7 +614,7 @@ __global__ void __launch_bounds__(256, 2) decode_persistent_kernel(const __grid_
       }
       __syncthreads();
       gemv_rows<2>(a.P + w.wd, sm, a.x, a.hm, hid, I, pair_red);
-      if (!(alive = grid_barrier(a, epoch))) break;
+      if (!(alive = grid_barrier(a.sync, a.status, 90, epoch))) break;
       xin = a.x;
     }
     if (!alive) break;
@@ -759,7 +651,7 @@ __global__ void __launch_bounds__(256, 2) decode_persistent_kernel(const __grid_
         atomicMax(&words[t & 1], best);
       }
     }
-    if (!(alive = grid_barrier(a, epoch))) break;
+    if (!(alive = grid_barrier(a.sync, a.status, 90, epoch))) break;
     {
       const unsigned long long wv = *reinterpret_cast<volatile unsigned long long*>(&words[t & 1]);
       tok = static_cast<int64_t>(0xFFFFFFFFu - static_cast<unsigned>(wv & 0xFFFFFFFFull));
@@ -790,41 +682,27 @@ struct LayerW {
   int64_t w_in, wq, wo, wqn, wkn, w_post, wg, wd;
 };
 
-struct Decoder {
+struct Decoder : DecoderBase {
   ctdk_model_config cfg;
-  const float* params;
-  int64_t embed, norm;
+  const float* params = nullptr;
+  int64_t embed = 0, norm = 0;
   std::vector<LayerW> lw;
-  int max_seq, QKVN;
+  int QKVN = 0;
   // workspace
-  float *rope_table, *kcache, *vcache;  // caches: [L][Hk][max_seq][D]
-  float *x, *h1, *qkv, *q, *attn, *hm, *gu, *act, *logits;
+  float *rope_table = nullptr, *kcache = nullptr, *vcache = nullptr;  // caches: [L][Hk][max_seq][D]
+  float *x, *h1, *qkv, *q, *attn, *hm, *gu, *act;
   float* attn_part;   // [H][kAttnSplits][D + 2] partial results of the decode attention
   float *pa, *pb, *pqkv, *pattn, *plse, *pgu, *pact;  // prefill buffers ([max_seq, ...])
-  int64_t* cur_token;
-  int* counters;  // [0] = position of the next token, [1] = tokens generated
   unsigned int* sync = nullptr;
   int persistent_grid = -1;   // CTAs of the persistent token kernel; 0 = not usable here; -1 = not decided yet
-  cudaGraphExec_t graph = nullptr;
-  int64_t* graph_out = nullptr;
-  cudaStream_t graph_stream = nullptr;
-  int64_t prompt_len = 0, generated = 0;
-  int64_t stepped = 0;   // tokens fed one by one through ctdk_decode_step since the prefill
+
+  int portion(const int64_t* ids, int64_t T, int64_t pos, const int32_t* want, int64_t n_want, float* want_logits,
+              cudaStream_t s) override;
+  int token_forward(cudaStream_t s) override;
+  int burst(int64_t n, int64_t* out_tokens, cudaStream_t s) override;
 };
 
-struct Bump2 {
-  char* base;
-  int64_t used = 0;
-  explicit Bump2(void* b) : base(static_cast<char*>(b)) {}
-  float* floats(int64_t n) {
-    const int64_t bytes = (n * 4 + 255) / 256 * 256;
-    float* p = base ? reinterpret_cast<float*>(base + used) : nullptr;
-    used += bytes;
-    return p;
-  }
-};
-
-void carve_decoder(Decoder& d, Bump2& b) {
+void carve_decoder(Decoder& d, Bump& b) {
   const ctdk_model_config& c = d.cfg;
   const int64_t hid = c.hidden_size, I = c.intermediate_size, D = c.head_dim, H = c.num_attention_heads,
                 Hk = c.num_key_value_heads, L = c.num_hidden_layers, S = d.max_seq;
@@ -858,6 +736,7 @@ int init_decoder(Decoder& d, const ctdk_model_config* cfg, int64_t max_seq) {
   const int64_t n = ctdk_model_num_tensors(cfg);
   if (n < 0) return CTDK_EINVAL;
   d.cfg = *cfg;
+  d.vocab = cfg->vocab_size;
   d.max_seq = static_cast<int>(max_seq);
   d.QKVN = (cfg->num_attention_heads + 2 * cfg->num_key_value_heads) * cfg->head_dim;
   std::vector<int64_t> off(n);
@@ -888,12 +767,6 @@ int init_decoder(Decoder& d, const ctdk_model_config* cfg, int64_t max_seq) {
   return CTDK_OK;
 }
 
-#define DTRY(expr)                    \
-  do {                                \
-    int rc_ = (expr);                 \
-    if (rc_ != CTDK_OK) return rc_;   \
-  } while (0)
-
 int gemv(const float* W, const float* x, float* y, const float* residual, int N, int K, cudaStream_t s,
          int pre = kPreNone, const float* nw = nullptr, float eps = 0.0f) {
   CTDK_REQUIRE(K % 4 == 0 && K <= 12288, "gemv: K must be a multiple of 4 and at most 12288");
@@ -918,7 +791,7 @@ ctdk_rope_params decode_rope_params(const ctdk_model_config& c) {
   return p;
 }
 
-// One token: embedding of *cur_token at position *pos -> logits -> argmax -> counters += 1.
+// One token: embedding of *cur_token at position *pos -> logits.
 int enqueue_token_forward(Decoder& d, cudaStream_t s) {
   const ctdk_model_config& c = d.cfg;
   const int hid = c.hidden_size, I = c.intermediate_size, D = c.head_dim, H = c.num_attention_heads,
@@ -949,17 +822,6 @@ int enqueue_token_forward(Decoder& d, cudaStream_t s) {
     DTRY(gemv(P + w.wd, d.gu, d.x, d.hm, hid, I, s, kPreSwiglu));
   }
   return gemv(P + d.embed, d.x, d.logits, nullptr, c.vocab_size, hid, s, kPreRmsNorm, P + d.norm, c.rms_norm_eps);
-}
-
-int enqueue_token_step(Decoder& d, int64_t* out_tokens, cudaStream_t s) {
-  DTRY(enqueue_token_forward(d, s));
-  unsigned long long* word = reinterpret_cast<unsigned long long*>(d.counters + 4);
-  if (launch_pdl(argmax_kernel, 64, 256, 0, s, d.logits, d.cfg.vocab_size, word) != cudaSuccess)
-    return fail(CTDK_ELAUNCH, "decode argmax: launch failed");
-  DTRY(check_launch("decode argmax"));
-  if (launch_pdl(argmax_finish_kernel, 1, 1, 0, s, word, d.cur_token, out_tokens, d.counters, d.counters + 1) != cudaSuccess)
-    return fail(CTDK_ELAUNCH, "decode argmax finish: launch failed");
-  return check_launch("decode argmax finish");
 }
 
 // Returns CTDK_OK when the persistent kernel was launched for `n` tokens, 1 when it does not apply
@@ -1032,69 +894,9 @@ int launch_persistent(Decoder& d, int64_t n, int64_t* out_tokens, cudaStream_t s
   return check_launch("decode persistent");
 }
 
-__global__ void set_token_kernel(int64_t* cur, int64_t value) { *cur = value; }
-__global__ void bump_position_kernel(int* position) { *position += 1; }
-
-}  // namespace
-}  // namespace ctdk
-
-using namespace ctdk;
-
-extern "C" {
-
-int64_t ctdk_decode_workspace_bytes(const ctdk_model_config* cfg, int64_t max_seq) {
-  Decoder d;
-  if (init_decoder(d, cfg, max_seq) != CTDK_OK) return -1;
-  Bump2 b(nullptr);
-  carve_decoder(d, b);
-  return b.used;
-}
-
-int ctdk_decode_create(const ctdk_model_config* cfg, const float* params, void* workspace,
-                       int64_t workspace_bytes, int64_t max_seq, void** decoder) {
-  CTDK_REQUIRE(decoder && params && workspace, "ctdk_decode_create: null pointer");
-  CTDK_REQUIRE((reinterpret_cast<uintptr_t>(params) & 255u) == 0 && (reinterpret_cast<uintptr_t>(workspace) & 255u) == 0,
-               "ctdk_decode_create: arenas must be 256-byte aligned");
-  Decoder* d = new (std::nothrow) Decoder();
-  if (d == nullptr) return fail(CTDK_ENOMEM, "ctdk_decode_create: out of host memory");
-  int rc = init_decoder(*d, cfg, max_seq);
-  if (rc != CTDK_OK) {
-    delete d;
-    return rc;
-  }
-  const int64_t attn_smem = ((static_cast<int64_t>(max_seq) + kAttnSplits - 1) / kAttnSplits + 4 + cfg->head_dim + 256) * 4;
-  CTDK_REQUIRE(attn_smem <= 200 * 1024, "ctdk_decode_create: max_seq too large for the decode attention kernel");
-  CTDK_REQUIRE(cfg->head_dim <= 256 && 256 % cfg->head_dim == 0, "ctdk_decode_create: head_dim must divide 256");
-  d->params = params;
-  Bump2 b(workspace);
-  carve_decoder(*d, b);
-  if (b.used > workspace_bytes) {
-    delete d;
-    return fail(CTDK_EINVAL, "ctdk_decode_create: workspace too small");
-  }
-  cudaError_t e = cudaFuncSetAttribute(decode_attn_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                       static_cast<int>(attn_smem));
-  if (e != cudaSuccess) {
-    delete d;
-    return fail(CTDK_ELAUNCH, "ctdk_decode_create: %s", cudaGetErrorString(e));
-  }
-  *decoder = d;
-  return CTDK_OK;
-}
-
-int ctdk_decode_destroy(void* decoder) {
-  Decoder* d = static_cast<Decoder*>(decoder);
-  if (d != nullptr && d->graph != nullptr) cudaGraphExecDestroy(d->graph);
-  delete d;
-  return CTDK_OK;
-}
-
-int ctdk_decode_prefill(void* decoder, const int64_t* ids, int64_t T, void* stream) {
-  CTDK_REQUIRE(decoder && ids, "ctdk_decode_prefill: null pointer");
-  Decoder& d = *static_cast<Decoder*>(decoder);
+// The prompt pass: every position at once with the training-path kernels, K / V rows into the cache.
+int prompt_pass(Decoder& d, const int64_t* ids, int64_t T, cudaStream_t s) {
   const ctdk_model_config& c = d.cfg;
-  CTDK_REQUIRE(T > 0 && T < d.max_seq, "ctdk_decode_prefill: prompt length must be in [1, max_seq)");
-  cudaStream_t s = static_cast<cudaStream_t>(stream);
   const int hid = c.hidden_size, I = c.intermediate_size, D = c.head_dim, H = c.num_attention_heads,
             Hk = c.num_key_value_heads;
   const float* P = d.params;
@@ -1127,105 +929,89 @@ int ctdk_decode_prefill(void* decoder, const int64_t* ids, int64_t T, void* stre
     DTRY(ctdk_swiglu_fwd(d.pgu, d.pact, T, I, s));
     DTRY(ctdk_gemm(d.pact, P + w.wd, d.pa, T, hid, I, I, I, hid, 0, 1, prec, CTDK_EPI_RESIDUAL, d.pb, s));
   }
-  // logits of the last prompt position only, then the first generated token
-  DTRY(ctdk_rmsnorm_fwd(d.pa + (T - 1) * hid, P + d.norm, d.h1, nullptr, 1, hid, c.rms_norm_eps, s));
-  DTRY(gemv(P + d.embed, d.h1, d.logits, nullptr, c.vocab_size, hid, s));
-  set_counters_kernel<<<1, 1, 0, s>>>(d.counters, d.counters + 1, static_cast<int>(T), 0);
-  d.prompt_len = T;
-  d.generated = 0;
-  d.stepped = 0;
-  return check_launch("decode counters");
-}
-
-int ctdk_decode_logits(void* decoder, const float** logits) {
-  CTDK_REQUIRE(decoder && logits, "ctdk_decode_logits: null pointer");
-  *logits = static_cast<Decoder*>(decoder)->logits;
   return CTDK_OK;
 }
 
-int ctdk_decode_step(void* decoder, int64_t token, void* stream) {
-  CTDK_REQUIRE(decoder != nullptr, "ctdk_decode_step: null decoder");
-  Decoder& d = *static_cast<Decoder*>(decoder);
-  CTDK_REQUIRE(d.prompt_len > 0, "ctdk_decode_step: call ctdk_decode_prefill first");
-  CTDK_REQUIRE(d.generated == 0, "ctdk_decode_step: cannot be mixed with ctdk_decode_greedy after one prefill");
-  CTDK_REQUIRE(token >= 0 && token < d.cfg.vocab_size, "ctdk_decode_step: token id out of range");
-  CTDK_REQUIRE(d.prompt_len + d.stepped < d.max_seq, "ctdk_decode_step: the cache is full (max_seq %d)", d.max_seq);
-  cudaStream_t s = static_cast<cudaStream_t>(stream);
-  set_token_kernel<<<1, 1, 0, s>>>(d.cur_token, token);
-  DTRY(check_launch("decode set token"));
-  DTRY(enqueue_token_forward(d, s));
-  bump_position_kernel<<<1, 1, 0, s>>>(d.counters);
-  DTRY(check_launch("decode bump"));
-  ++d.stepped;
+// logits row of one prompt position: final norm of its residual row, then the tied head.
+int prompt_logits(Decoder& d, int64_t row, float* out, cudaStream_t s) {
+  const int hid = d.cfg.hidden_size;
+  DTRY(ctdk_rmsnorm_fwd(d.pa + row * hid, d.params + d.norm, d.h1, nullptr, 1, hid, d.cfg.rms_norm_eps, s));
+  return gemv(d.params + d.embed, d.h1, out, nullptr, d.cfg.vocab_size, hid, s);
+}
+
+__global__ void place_token_kernel(int64_t* cur, int* counters, const int64_t* id, int pos) {
+  *cur = *id;
+  counters[0] = pos;
+}
+
+int Decoder::token_forward(cudaStream_t s) { return enqueue_token_forward(*this, s); }
+int Decoder::burst(int64_t n, int64_t* out_tokens, cudaStream_t s) { return launch_persistent(*this, n, out_tokens, s); }
+
+// The whole-prompt pass has no entry for keys that are already cached, so a later portion runs as token passes.
+int Decoder::portion(const int64_t* ids, int64_t T, int64_t pos, const int32_t* want, int64_t n_want, float* want_logits,
+                     cudaStream_t s) {
+  if (pos == 0) {
+    DTRY(prompt_pass(*this, ids, T, s));
+    if (n_want < 0) return prompt_logits(*this, T - 1, logits, s);
+    for (int64_t i = 0; i < n_want; ++i) DTRY(prompt_logits(*this, want[i], want_logits + i * vocab, s));
+    return CTDK_OK;
+  }
+  for (int64_t t = 0; t < T; ++t) {
+    place_token_kernel<<<1, 1, 0, s>>>(cur_token, counters, ids + t, static_cast<int>(pos + t));
+    DTRY(check_launch("decode place token"));
+    DTRY(token_forward(s));
+    for (int64_t i = 0; i < n_want; ++i)
+      if (want[i] == t &&
+          cudaMemcpyAsync(want_logits + i * vocab, logits, sizeof(float) * vocab, cudaMemcpyDeviceToDevice, s) != cudaSuccess)
+        return fail(CTDK_ELAUNCH, "decode: copying a logits row failed");
+  }
   return CTDK_OK;
 }
 
-int ctdk_decode_greedy(void* decoder, int64_t n_new, int64_t* out_tokens, void* stream) {
-  CTDK_REQUIRE(decoder && out_tokens, "ctdk_decode_greedy: null pointer");
-  CTDK_REQUIRE(n_new >= 0, "ctdk_decode_greedy: negative token count");
-  Decoder& d = *static_cast<Decoder*>(decoder);
-  CTDK_REQUIRE(d.prompt_len > 0, "ctdk_decode_greedy: call ctdk_decode_prefill first");
-  CTDK_REQUIRE(d.stepped == 0, "ctdk_decode_greedy: cannot be mixed with ctdk_decode_step after one prefill");
-  // n tokens after the prompt need n - 1 cache positions (the first comes from the prompt's logits, the
-  // last is not fed back): the reference's loop emits max_seq - prompt + 1 tokens before it reports
-  // max_seq_len (tools/ctd_generate/main.cpp:143-179)
-  CTDK_REQUIRE(d.prompt_len + d.generated + n_new <= d.max_seq + 1,
-               "ctdk_decode_greedy: %lld more tokens would exceed max_seq %d", static_cast<long long>(n_new),
-               d.max_seq);
-  cudaStream_t s = static_cast<cudaStream_t>(stream);
-  int64_t todo = n_new;
-  if (todo > 0 && d.generated == 0) {
-    // the first new token comes from the prefill logits; its position is the prompt length
-    unsigned long long* word = reinterpret_cast<unsigned long long*>(d.counters + 4);
-    argmax_kernel<<<64, 256, 0, s>>>(d.logits, d.cfg.vocab_size, word);
-    DTRY(check_launch("decode argmax"));
-    // count += 1; the position is unchanged (a scratch int takes the increment)
-    argmax_finish_kernel<<<1, 1, 0, s>>>(word, d.cur_token, out_tokens, d.counters + 2, d.counters + 1);
-    DTRY(check_launch("decode argmax finish"));
-    d.generated = 1;
-    --todo;
+}  // namespace
+}  // namespace ctdk
+
+using namespace ctdk;
+
+extern "C" {
+
+int64_t ctdk_decode_workspace_bytes(const ctdk_model_config* cfg, int64_t max_seq) {
+  Decoder d;
+  if (init_decoder(d, cfg, max_seq) != CTDK_OK) return -1;
+  Bump b(nullptr);
+  carve_decoder(d, b);
+  return b.used;
+}
+
+int ctdk_decode_create(const ctdk_model_config* cfg, const float* params, void* workspace,
+                       int64_t workspace_bytes, int64_t max_seq, void** decoder) {
+  CTDK_REQUIRE(decoder && params && workspace, "ctdk_decode_create: null pointer");
+  CTDK_REQUIRE((reinterpret_cast<uintptr_t>(params) & 255u) == 0 && (reinterpret_cast<uintptr_t>(workspace) & 255u) == 0,
+               "ctdk_decode_create: arenas must be 256-byte aligned");
+  Decoder* d = new (std::nothrow) Decoder();
+  if (d == nullptr) return fail(CTDK_ENOMEM, "ctdk_decode_create: out of host memory");
+  int rc = init_decoder(*d, cfg, max_seq);
+  if (rc != CTDK_OK) {
+    delete d;
+    return rc;
   }
-  if (todo == 0) return CTDK_OK;
-  // All remaining tokens in one cooperative launch of the persistent kernel where it applies.
-  {
-    const int rc = launch_persistent(d, todo, out_tokens, s);
-    if (rc <= 0) {
-      if (rc == CTDK_OK) d.generated += todo;
-      return rc;
-    }
+  const int64_t attn_smem = ((static_cast<int64_t>(max_seq) + kAttnSplits - 1) / kAttnSplits + 4 + cfg->head_dim + 256) * 4;
+  CTDK_REQUIRE(attn_smem <= 200 * 1024, "ctdk_decode_create: max_seq too large for the decode attention kernel");
+  CTDK_REQUIRE(cfg->head_dim <= 256 && 256 % cfg->head_dim == 0, "ctdk_decode_create: head_dim must divide 256");
+  d->params = params;
+  Bump b(workspace);
+  carve_decoder(*d, b);
+  if (b.used > workspace_bytes) {
+    delete d;
+    return fail(CTDK_EINVAL, "ctdk_decode_create: workspace too small");
   }
-  // One token step = ~9 kernels per layer; captured once and replayed, so a step costs one launch.
-  const bool can_capture = s != nullptr;
-  if (can_capture && (d.graph == nullptr || d.graph_out != out_tokens || d.graph_stream != s)) {
-    if (d.graph != nullptr) {
-      cudaGraphExecDestroy(d.graph);
-      d.graph = nullptr;
-    }
-    cudaGraph_t g = nullptr;
-    cudaError_t e = cudaStreamBeginCapture(s, cudaStreamCaptureModeThreadLocal);
-    if (e != cudaSuccess) return fail(CTDK_ELAUNCH, "decode: begin capture: %s", cudaGetErrorString(e));
-    const int rc = enqueue_token_step(d, out_tokens, s);
-    e = cudaStreamEndCapture(s, &g);
-    if (rc != CTDK_OK) {
-      if (g != nullptr) cudaGraphDestroy(g);
-      return rc;
-    }
-    if (e != cudaSuccess) return fail(CTDK_ELAUNCH, "decode: end capture: %s", cudaGetErrorString(e));
-    e = cudaGraphInstantiate(&d.graph, g, 0);
-    cudaGraphDestroy(g);
-    if (e != cudaSuccess) return fail(CTDK_ELAUNCH, "decode: graph instantiate: %s", cudaGetErrorString(e));
-    d.graph_out = out_tokens;
-    d.graph_stream = s;
+  cudaError_t e = cudaFuncSetAttribute(decode_attn_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                       static_cast<int>(attn_smem));
+  if (e != cudaSuccess) {
+    delete d;
+    return fail(CTDK_ELAUNCH, "ctdk_decode_create: %s", cudaGetErrorString(e));
   }
-  for (int64_t i = 0; i < todo; ++i) {
-    if (can_capture) {
-      cudaError_t e = cudaGraphLaunch(d.graph, s);
-      if (e != cudaSuccess) return fail(CTDK_ELAUNCH, "decode: graph launch: %s", cudaGetErrorString(e));
-    } else {
-      DTRY(enqueue_token_step(d, out_tokens, s));
-    }
-  }
-  d.generated += todo;
+  *decoder = static_cast<DecoderBase*>(d);
   return CTDK_OK;
 }
 

@@ -1,5 +1,5 @@
 // TF32 GEMM on the 5th-generation tensor cores: C[M,N] = op(A)·op(B) with fp32 operands in
-// HBM, fp32 accumulators in tensor memory.
+// HBM, fp32 accumulators in tensor memory; and C = A·B^T with bfloat16 operands on the same kernel.
 //
 // One persistent CTA per SM, 6 warps:
 //   warp 0   TMA producer: fills a ring of shared-memory stages (128-byte swizzled tiles),
@@ -28,6 +28,7 @@ namespace {
 
 constexpr int BM = 128;
 constexpr int BK = 32;                    // floats per stage along K = one 128-byte swizzle row
+constexpr int BKH = 64;                   // the same row in bfloat16
 constexpr int kATileBytes = BM * BK * 4;  // 16 KB
 constexpr int kChunkBytes = 32 * BK * 4;  // 4 KB: one {32 x 32} box of an MN-major operand
 constexpr int kThreads = 192;
@@ -53,10 +54,10 @@ struct GemmArgs {
   int* status;
 };
 
-// Instruction descriptor for kind::tf32: D=F32 (bit 4), A,B=TF32 (value 2 at bits 7 and 10),
-// major-ness bits 15/16 (0 = K-major, 1 = MN-major), N>>3 at bit 17, M>>4 at bit 24.
-__host__ __device__ constexpr uint32_t make_idesc(bool a_mn, bool b_mn, int n) {
-  return (1u << 4) | (2u << 7) | (2u << 10) | (static_cast<uint32_t>(a_mn) << 15) |
+// Instruction descriptor: D=F32 (bit 4), A,B format at bits 7 and 10 (kind::tf32: 2 = TF32;
+// kind::f16: 1 = BF16), major-ness bits 15/16 (0 = K-major, 1 = MN-major), N>>3 at bit 17, M>>4 at bit 24.
+__host__ __device__ constexpr uint32_t make_idesc(bool a_mn, bool b_mn, int n, uint32_t fmt = 2u) {
+  return (1u << 4) | (fmt << 7) | (fmt << 10) | (static_cast<uint32_t>(a_mn) << 15) |
          (static_cast<uint32_t>(b_mn) << 16) | (static_cast<uint32_t>(n >> 3) << 17) |
          (static_cast<uint32_t>(BM >> 4) << 24);
 }
@@ -72,11 +73,15 @@ __device__ __forceinline__ void tile_coords(int tile, int m_blocks, int n_blocks
   nb = local / gm;
 }
 
-template <int BN, bool A_MN, bool B_MN>
+// BF16: bfloat16 operands, both K-major. A stage row is 128 bytes either way and an MMA takes 32 of
+// them (8 TF32 or 16 bfloat16 values), so tiles, swizzle and descriptors are the same bytes.
+template <int BN, bool A_MN, bool B_MN, bool BF16>
 __global__ void __launch_bounds__(kThreads, 1)
     gemm_tf32_kernel(const __grid_constant__ CUtensorMap tmA,
                      const __grid_constant__ CUtensorMap tmB, const GemmArgs args) {
+  static_assert(!BF16 || (!A_MN && !B_MN), "bfloat16 operands are K-major");
   using C = Cfg<BN>;
+  constexpr int kElems = BF16 ? BKH : BK;   // values of a stage row
   extern __shared__ unsigned char smem_raw[];
   const uint32_t raw = smem_u32(smem_raw);
   unsigned char* smem = smem_raw + ((1024u - (raw & 1023u)) & 1023u);
@@ -92,7 +97,7 @@ __global__ void __launch_bounds__(kThreads, 1)
   const int m_blocks = (args.M + BM - 1) / BM;
   const int n_blocks = (args.N + BN - 1) / BN;
   const int num_tiles = m_blocks * n_blocks;
-  const int k_blocks = (args.K + BK - 1) / BK;
+  const int k_blocks = (args.K + kElems - 1) / kElems;
   const int num_units = num_tiles * args.splits;  // unit u: tile u % num_tiles, k-range u / num_tiles
 
   if (threadIdx.x == 0) {
@@ -139,7 +144,7 @@ __global__ void __launch_bounds__(kThreads, 1)
           unsigned char* a_dst = smem + s * C::kStageBytes;
           unsigned char* b_dst = a_dst + kATileBytes;
           mbar_expect_tx(&full[s], C::kStageBytes);
-          const int k0 = kb * BK;
+          const int k0 = kb * kElems;
           if (A_MN) {
 #pragma unroll
             for (int c = 0; c < BM / 32; ++c)
@@ -165,7 +170,7 @@ __global__ void __launch_bounds__(kThreads, 1)
   } else if (warp == 1) {
     // ------------------------------- MMA issuer -------------------------------
     if (lane == 0) {
-      constexpr uint32_t idesc = make_idesc(A_MN, B_MN, BN);
+      constexpr uint32_t idesc = make_idesc(A_MN, B_MN, BN, BF16 ? 1u : 2u);
       int s = 0;
       uint32_t ph = 0;
       bool ok = true;
@@ -203,7 +208,8 @@ __global__ void __launch_bounds__(kThreads, 1)
             const uint64_t bdesc =
                 B_MN ? make_smem_desc(b_addr + ks * 1024, kChunkBytes, 512, kLayoutSw128Base32)
                      : make_smem_desc(b_addr + ks * 32, 16, 1024, kLayoutSw128);
-            umma_tf32(d_tmem, adesc, bdesc, idesc, (kb != kb0 || ks != 0) ? 1u : 0u);
+            if (BF16) umma_bf16(d_tmem, adesc, bdesc, idesc, (kb != kb0 || ks != 0) ? 1u : 0u);
+            else umma_tf32(d_tmem, adesc, bdesc, idesc, (kb != kb0 || ks != 0) ? 1u : 0u);
           }
           umma_commit(&empty[s]);  // stage is free once these MMAs have read it
           if (++s == C::kStages) {
@@ -400,14 +406,14 @@ int encode_tensor_map(CUtensorMap* map, const float* base, int rank, const uint6
 
 namespace {
 
-template <int BN, bool A_MN, bool B_MN>
+template <int BN, bool A_MN, bool B_MN, bool BF16 = false>
 int launch(const CUtensorMap& ta, const CUtensorMap& tb, const GemmArgs& args,
            cudaStream_t stream) {
   using C = Cfg<BN>;
   static bool attr_set[64] = {false};
   int dev = 0;
   cudaGetDevice(&dev);
-  auto* kern = gemm_tf32_kernel<BN, A_MN, B_MN>;
+  auto* kern = gemm_tf32_kernel<BN, A_MN, B_MN, BF16>;
   if (dev >= 0 && dev < 64 && !attr_set[dev]) {
     cudaError_t e =
         cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, C::kSmemBytes);
@@ -525,25 +531,16 @@ int gemm_dattn_delta_tcgen05(const float* dy, const float* Wo, const float* out,
 static thread_local int t_kblock_limit = 0;
 void gemm_set_kblock_limit(int k_blocks) { t_kblock_limit = k_blocks; }
 
-// Returns CTDK_OK after enqueueing, or 1 when the shape/alignment is not eligible for the
-// tensor-core path (the caller then uses the SIMT kernel).
-int gemm_tcgen05(const float* A, const float* B, float* Cp, int64_t M, int64_t N, int64_t K,
-                 int64_t lda, int64_t ldb, int64_t ldc, int transa, int transb, int epilogue,
-                 const float* aux, cudaStream_t stream) {
-  auto a16 = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15u) == 0; };
-  if (!a16(A) || !a16(B) || (lda & 3) || (ldb & 3)) return 1;
-  if (M > INT32_MAX || N > INT32_MAX || K > INT32_MAX) return 1;
-  if (M < 1 || N < 8 || K < 1) return 1;
+namespace {
 
-  const bool a_mn = transa != 0;  // A stored [K,M]: contiguous along M
-  const bool b_mn = transb == 0;  // B stored [K,N]: contiguous along N
+// Tile width, K split and one-CTA / paired-CTA kernel for an M x N product of k_blocks stage rows.
+void choose_tile(int64_t M, int64_t N, int64_t k_blocks, int* bn_out, int* splits_out, bool* pair_out) {
   // Tile width and K split: estimated time = rounds of the persistent grid x k-blocks per
   // unit x relative cost of a k-block (a 128-wide tile does half the work of a 256-wide one
   // but moves 2/3 of the operand bytes, hence the 0.6). Splitting K only pays when the output
   // tiles alone cannot fill the SMs (weight gradients: few tiles, K = all tokens).
   const int sms = sm_budget();
   const int64_t m_blocks = (M + BM - 1) / BM;
-  const int64_t k_blocks = (K + BK - 1) / BK;
   int bn = 64, splits = 1;
   if (N > 64) {
     double best = 1e300;
@@ -605,6 +602,29 @@ int gemm_tcgen05(const float* A, const float* B, float* Cp, int64_t M, int64_t N
       bn = 256;
     }
   }
+  *bn_out = bn;
+  *splits_out = splits;
+  *pair_out = use_pair;
+}
+
+}  // namespace
+
+// Returns CTDK_OK after enqueueing, or 1 when the shape/alignment is not eligible for the
+// tensor-core path (the caller then uses the SIMT kernel).
+int gemm_tcgen05(const float* A, const float* B, float* Cp, int64_t M, int64_t N, int64_t K,
+                 int64_t lda, int64_t ldb, int64_t ldc, int transa, int transb, int epilogue,
+                 const float* aux, cudaStream_t stream) {
+  auto a16 = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15u) == 0; };
+  if (!a16(A) || !a16(B) || (lda & 3) || (ldb & 3)) return 1;
+  if (M > INT32_MAX || N > INT32_MAX || K > INT32_MAX) return 1;
+  if (M < 1 || N < 8 || K < 1) return 1;
+
+  const bool a_mn = transa != 0;  // A stored [K,M]: contiguous along M
+  const bool b_mn = transb == 0;  // B stored [K,N]: contiguous along N
+  const int64_t k_blocks = (K + BK - 1) / BK;
+  int bn, splits;
+  bool use_pair;
+  choose_tile(M, N, k_blocks, &bn, &splits, &use_pair);
 
   if (t_kblock_limit > 0) {
     int64_t need = (k_blocks + t_kblock_limit - 1) / t_kblock_limit;
@@ -680,6 +700,64 @@ int gemm_tcgen05(const float* A, const float* B, float* Cp, int64_t M, int64_t N
     case 64: return dispatch_major<64>(a_mn, b_mn, ta, tb, args, stream);
     case 128: return dispatch_major<128>(a_mn, b_mn, ta, tb, args, stream);
     default: return dispatch_major<256>(a_mn, b_mn, ta, tb, args, stream);
+  }
+}
+
+int gemm_tcgen05_2cta_bf16(const CUtensorMap& ta, const CUtensorMap& tb, const CUtensorMap& tc, int tma_out, float* C,
+                           int64_t ldc, int M, int N, int K, int vec_ok, int splits, int* status, cudaStream_t stream);
+
+// C[M, N] (fp32) = A[M, K] B[N, K]^T with bfloat16 operands in memory, fp32 accumulation. Pointers
+// 16-byte aligned, lda and ldb multiples of 8.
+int gemm_bf16_tcgen05(const void* A, const void* B, float* Cp, int64_t M, int64_t N, int64_t K, int64_t lda, int64_t ldb,
+                      int64_t ldc, cudaStream_t stream) {
+  auto a16 = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15u) == 0; };
+  CTDK_REQUIRE(a16(A) && a16(B) && (lda & 7) == 0 && (ldb & 7) == 0, "gemm_bf16: operands must be 16-byte aligned");
+  CTDK_REQUIRE(M >= 1 && N >= 8 && K >= 1 && M <= INT32_MAX && N <= INT32_MAX && K <= INT32_MAX, "gemm_bf16: bad shape");
+  const int64_t k_blocks = (K + BKH - 1) / BKH;
+  int bn, splits;
+  bool use_pair;
+  choose_tile(M, N, k_blocks, &bn, &splits, &use_pair);
+  auto map_bf16 = [](CUtensorMap* map, const void* base, int64_t inner, int64_t outer, int64_t ld, int box_rows) {
+    auto enc = encode_fn();
+    if (enc == nullptr) return fail(CTDK_ELAUNCH, "cuTensorMapEncodeTiled unavailable");
+    cuuint64_t dims[2] = {static_cast<cuuint64_t>(inner), static_cast<cuuint64_t>(outer)};
+    cuuint64_t strides[1] = {static_cast<cuuint64_t>(ld) * 2};
+    cuuint32_t box[2] = {static_cast<cuuint32_t>(BKH), static_cast<cuuint32_t>(box_rows)};
+    cuuint32_t estr[2] = {1u, 1u};
+    const CUresult r = enc(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(base), dims, strides, box, estr,
+                           CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+                           CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+    if (r != CUDA_SUCCESS) return fail(CTDK_ELAUNCH, "cuTensorMapEncodeTiled failed (%d) for a bfloat16 operand", static_cast<int>(r));
+    return CTDK_OK;
+  };
+  CUtensorMap ta, tb;
+  int rc = map_bf16(&ta, A, K, M, lda, BM);
+  if (rc == CTDK_OK) rc = map_bf16(&tb, B, K, N, ldb, use_pair ? 128 : bn);
+  if (rc != CTDK_OK) return rc;
+  int* st = device_status_word();
+  if (st == nullptr) return fail(CTDK_ELAUNCH, "gemm: no status word");
+  const int vec = (a16(Cp) && (ldc & 3) == 0) ? 1 : 0;
+  if (splits > 1) {
+    const cudaError_t e = cudaMemset2DAsync(Cp, static_cast<size_t>(ldc) * sizeof(float), 0, static_cast<size_t>(N) * sizeof(float),
+                                            static_cast<size_t>(M), stream);
+    if (e != cudaSuccess) return fail(CTDK_ELAUNCH, "gemm: memset failed: %s", cudaGetErrorString(e));
+  }
+  if (use_pair) {
+    int tma_out = 0;
+    CUtensorMap tc = ta;
+    if (vec) {
+      tma_out = splits > 1 ? 2 : 1;
+      rc = make_map(&tc, Cp, N, M, ldc, 32, false, true);
+      if (rc != CTDK_OK) return rc;
+    }
+    return gemm_tcgen05_2cta_bf16(ta, tb, tc, tma_out, Cp, ldc, static_cast<int>(M), static_cast<int>(N), static_cast<int>(K), vec,
+                                  splits, st, stream);
+  }
+  const GemmArgs args{Cp, nullptr, ldc, static_cast<int>(M), static_cast<int>(N), static_cast<int>(K), CTDK_EPI_STORE, vec, splits, st};
+  switch (bn) {
+    case 64: return launch<64, false, false, true>(ta, tb, args, stream);
+    case 128: return launch<128, false, false, true>(ta, tb, args, stream);
+    default: return launch<256, false, false, true>(ta, tb, args, stream);
   }
 }
 

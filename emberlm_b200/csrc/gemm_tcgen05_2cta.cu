@@ -19,6 +19,7 @@ namespace {
 constexpr int BM2 = 128;                 // rows of A per CTA (pair: 256)
 constexpr int BN2 = 256;                 // tile width (each CTA loads 128 columns of B)
 constexpr int BK2 = 32;
+constexpr int BK2H = 64;                  // the same 128-byte stage row in bfloat16
 constexpr int kATile = BM2 * BK2 * 4;    // 16 KB
 constexpr int kBHalf = (BN2 / 2) * BK2 * 4;  // 16 KB
 constexpr int kStage2 = kATile + kBHalf;
@@ -126,6 +127,17 @@ __device__ __forceinline__ void umma_tf32_pair(uint32_t tmem_d, uint64_t adesc, 
       "l"(adesc), "l"(bdesc), "r"(idesc), "r"(accumulate)
       : "memory");
 }
+__device__ __forceinline__ void umma_bf16_pair(uint32_t tmem_d, uint64_t adesc, uint64_t bdesc, uint32_t idesc,
+                                               uint32_t accumulate) {
+  asm volatile(
+      "{\n"
+      ".reg .pred p;\n"
+      "setp.ne.b32 p, %4, 0;\n"
+      "tcgen05.mma.cta_group::2.kind::f16 [%0], %1, %2, %3, p;\n"
+      "}\n" ::"r"(tmem_d),
+      "l"(adesc), "l"(bdesc), "r"(idesc), "r"(accumulate)
+      : "memory");
+}
 // One arrival on the barrier at this offset in BOTH CTAs of the pair once prior MMAs retire.
 __device__ __forceinline__ void umma_commit_pair(uint64_t* bar) {
   asm volatile(
@@ -151,7 +163,8 @@ __device__ __forceinline__ void tile_coords2(int tile, int m_blocks, int n_block
   nb = local / gm;
 }
 
-template <bool A_MN, bool B_MN>
+// BF16: bfloat16 operands, both K-major; a stage row is 128 bytes either way.
+template <bool A_MN, bool B_MN, bool BF16>
 __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(kThreads2, 1)
     gemm_tf32_2cta_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensorMap tmB,
                           const __grid_constant__ CUtensorMap tmC, const __grid_constant__ CUtensorMap tmD,
@@ -176,7 +189,9 @@ __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(kThreads2, 1)
   const int m_blocks = (args.M + 2 * BM2 - 1) / (2 * BM2);
   const int n_blocks = args.swiglu == 1 ? args.N / (BN2 / 2) : (args.N + BN2 - 1) / BN2;
   const int num_tiles = m_blocks * n_blocks;
-  const int k_blocks = (args.K + BK2 - 1) / BK2;
+  static_assert(!BF16 || (!A_MN && !B_MN), "bfloat16 operands are K-major");
+  constexpr int kElems = BF16 ? BK2H : BK2;   // values of a stage row
+  const int k_blocks = (args.K + kElems - 1) / kElems;
   const int num_units = num_tiles * args.splits;  // unit u: tile u % num_tiles, k-range u / num_tiles
   const int pair = blockIdx.x >> 1, n_pairs = gridDim.x >> 1;
 
@@ -234,7 +249,7 @@ __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(kThreads2, 1)
           unsigned char* a_dst = smem + s * kStage2;
           unsigned char* b_dst = a_dst + kATile;
           if (leader) mbar_expect_tx(&full[s], 2 * kStage2);  // bytes of both CTAs
-          const int k0 = kb * BK2;
+          const int k0 = kb * kElems;
           if (A_MN) {
             if (args.a3d) {
               tma_load_3d_pair(a_dst, &tmA, &full[s], 0, k0, m0 >> 5);
@@ -269,7 +284,8 @@ __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(kThreads2, 1)
     // ---------------- MMA issuer (leader CTA only) ----------------
     if (leader && lane == 0) {
       // M = 256 (both CTAs), N = 256
-      const uint32_t idesc = (1u << 4) | (2u << 7) | (2u << 10) | (static_cast<uint32_t>(A_MN) << 15) |
+      constexpr uint32_t fmt = BF16 ? 1u : 2u;
+      const uint32_t idesc = (1u << 4) | (fmt << 7) | (fmt << 10) | (static_cast<uint32_t>(A_MN) << 15) |
                              (static_cast<uint32_t>(B_MN) << 16) | (static_cast<uint32_t>(BN2 >> 3) << 17) |
                              (static_cast<uint32_t>(256 >> 4) << 24);
       int s = 0;
@@ -306,7 +322,8 @@ __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(kThreads2, 1)
                                         : make_smem_desc(a_addr + ks * 32, 16, 1024, kLayoutSw128);
             const uint64_t bdesc = B_MN ? make_smem_desc(b_addr + ks * 1024, kChunk2, 512, kLayoutSw128Base32)
                                         : make_smem_desc(b_addr + ks * 32, 16, 1024, kLayoutSw128);
-            umma_tf32_pair(d_tmem, adesc, bdesc, idesc, (kb != kb0 || ks != 0) ? 1u : 0u);
+            if (BF16) umma_bf16_pair(d_tmem, adesc, bdesc, idesc, (kb != kb0 || ks != 0) ? 1u : 0u);
+            else umma_tf32_pair(d_tmem, adesc, bdesc, idesc, (kb != kb0 || ks != 0) ? 1u : 0u);
           }
           umma_commit_pair(&empty[s]);
           if (++s == n_stages) {
@@ -634,10 +651,10 @@ __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(kThreads2, 1)
   }
 }
 
-template <bool A_MN, bool B_MN>
+template <bool A_MN, bool B_MN, bool BF16 = false>
 int launch2(const CUtensorMap& ta, const CUtensorMap& tb, const CUtensorMap& tc, const CUtensorMap& td,
             const Gemm2Args& args, cudaStream_t stream) {
-  auto* kern = gemm_tf32_2cta_kernel<A_MN, B_MN>;
+  auto* kern = gemm_tf32_2cta_kernel<A_MN, B_MN, BF16>;
   cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem2);
   if (e != cudaSuccess) return fail(CTDK_ELAUNCH, "gemm(2cta): shared memory opt-in failed: %s", cudaGetErrorString(e));
   const int tiles = ((args.M + 255) / 256) * (args.swiglu == 1 ? args.N / (BN2 / 2) : (args.N + BN2 - 1) / BN2) * args.splits;
@@ -661,6 +678,14 @@ int gemm_tcgen05_2cta(const CUtensorMap& ta, const CUtensorMap& tb, const CUtens
   if (!a_mn && b_mn) return launch2<false, true>(ta, tb, tc, tc, args, stream);
   if (a_mn && !b_mn) return launch2<true, false>(ta, tb, tc, tc, args, stream);
   return launch2<true, true>(ta, tb, tc, tc, args, stream);
+}
+
+// C[M, N] = A[M, K] B[N, K]^T with bfloat16 operands (maps with {64, 128} boxes), plain store (tma_out
+// 1) or split-K partial tiles added into a zeroed C (tma_out 2).
+int gemm_tcgen05_2cta_bf16(const CUtensorMap& ta, const CUtensorMap& tb, const CUtensorMap& tc, int tma_out, float* C,
+                           int64_t ldc, int M, int N, int K, int vec_ok, int splits, int* status, cudaStream_t stream) {
+  Gemm2Args args{C, nullptr, ldc, M, N, K, CTDK_EPI_STORE, vec_ok, splits, 0, 0, tma_out, 0, 1, nullptr, 0, 0, 0, kStages2, status};
+  return launch2<false, false, true>(ta, tb, tc, tc, args, stream);
 }
 
 // Fused MLP input projection: gu[M, 2N] = A[M, K] * W[2N, K]^T (gate rows then up rows) and

@@ -10,14 +10,17 @@ optim::AdamW (src/core/optim.cu:132-168), clipping as optim::clip_grad_norm_
 from __future__ import annotations
 
 import ctypes as C
-import os
+import json
 import math
+import os
 from dataclasses import dataclass
+from pathlib import Path
 
 import numpy as np
 import torch
 
 from . import lib
+from .safetensors_io import load_safetensors
 
 _L = lib.raw()
 
@@ -576,26 +579,44 @@ _L.ctdk_decode_greedy.restype = C.c_int
 _L.ctdk_decode_greedy.argtypes = [C.c_void_p, C.c_int64, C.c_void_p, C.c_void_p]
 _L.ctdk_decode_logits.restype = C.c_int
 _L.ctdk_decode_logits.argtypes = [C.c_void_p, C.POINTER(C.c_void_p)]
+_L.ctdk_decode_step.restype = C.c_int
+_L.ctdk_decode_step.argtypes = [C.c_void_p, C.c_int64, C.c_void_p]
+_L.ctdk_decode_extend.restype = C.c_int
+_L.ctdk_decode_extend.argtypes = [C.c_void_p, C.c_void_p, C.c_int64, C.POINTER(C.c_int32), C.c_int64, C.c_void_p, C.c_void_p]
+_L.ctdk_decode_reset.restype = C.c_int
+_L.ctdk_decode_reset.argtypes = [C.c_void_p, C.c_void_p]
 
 
-class Decoder:
-    """Greedy KV-cache generation, batch 1, as ctd_generate with temperature <= 0
-    (tools/ctd_generate/main.cpp:94-184): prefill the prompt, then one token per step."""
+class TensorInfo(C.Structure):
+    """ctdk_tensor_info."""
+    _fields_ = [("name", C.c_char * 96), ("rows", C.c_int64), ("cols", C.c_int64), ("ld", C.c_int64),
+                ("offset", C.c_int64), ("is_matrix", C.c_int)]
 
-    def __init__(self, cfg: ModelConfig, max_seq_len: int, device="cuda:0", params: torch.Tensor | None = None):
-        self.cfg, self.max_seq_len = cfg, max_seq_len
-        self.device = torch.device(device)
-        self.layout = model_layout(cfg)
-        self.params = params if params is not None else torch.zeros(self.layout.total, dtype=torch.float32,
-                                                                    device=self.device)
-        ws = _L.ctdk_decode_workspace_bytes(C.byref(cfg), max_seq_len)
-        if ws < 0:
-            raise lib.CtdkError(-1, lib.last_error())
-        self.workspace = torch.zeros(ws, dtype=torch.uint8, device=self.device)
-        self._h = C.c_void_p()
-        lib.check(_L.ctdk_decode_create(C.byref(cfg), self.params.data_ptr(), self.workspace.data_ptr(), ws,
-                                        max_seq_len, C.byref(self._h)))
-        self.stream = torch.cuda.Stream(device=self.device)
+
+_L.ctdk_hybrid_open.restype = C.c_int
+_L.ctdk_hybrid_open.argtypes = [C.c_char_p, C.c_char_p, C.c_int, C.POINTER(C.c_void_p)]
+_L.ctdk_hybrid_close.restype = C.c_int
+_L.ctdk_hybrid_close.argtypes = [C.c_void_p]
+_L.ctdk_hybrid_num_tensors.restype = C.c_int64
+_L.ctdk_hybrid_num_tensors.argtypes = [C.c_void_p]
+_L.ctdk_hybrid_tensor.restype = C.c_int
+_L.ctdk_hybrid_tensor.argtypes = [C.c_void_p, C.c_int64, C.POINTER(TensorInfo)]
+_L.ctdk_hybrid_arena_bytes.restype = C.c_int64
+_L.ctdk_hybrid_arena_bytes.argtypes = [C.c_void_p]
+_L.ctdk_hybrid_vocab.restype = C.c_int64
+_L.ctdk_hybrid_vocab.argtypes = [C.c_void_p]
+_L.ctdk_hybrid_workspace_bytes.restype = C.c_int64
+_L.ctdk_hybrid_workspace_bytes.argtypes = [C.c_void_p, C.c_int64, C.c_int64]
+_L.ctdk_hybrid_decode_create.restype = C.c_int
+_L.ctdk_hybrid_decode_create.argtypes = [C.c_void_p, C.c_void_p, C.c_void_p, C.c_int64, C.c_int64, C.c_int64,
+                                         C.POINTER(C.c_void_p)]
+_L.ctdk_hybrid_trace_layers.restype = C.c_int
+_L.ctdk_hybrid_trace_layers.argtypes = [C.c_void_p, C.c_void_p]
+
+
+class DecoderBase:
+    """What every decoder family offers on top of the ctdk_decode_* calls; subclasses set cfg, vocab,
+    max_seq_len, device, params, workspace, stream and the handle _h."""
 
     def __del__(self):
         h = getattr(self, "_h", None)
@@ -603,20 +624,13 @@ class Decoder:
             _L.ctdk_decode_destroy(h)
             self._h = None
 
-    def named_parameters(self) -> dict:
-        lo = self.layout
-        return {n: self.params[o:o + k].view(s) for n, s, o, k in zip(lo.names, lo.shapes, lo.offsets, lo.numels)}
-
-    def load_parameters(self, tensors: dict) -> None:
-        for n, v in self.named_parameters().items():
-            src = tensors[n]
-            src = torch.from_numpy(np.ascontiguousarray(src)) if isinstance(src, np.ndarray) else src
-            v.copy_(src.to(torch.float32))
+    def _ids(self, input_ids) -> torch.Tensor:
+        return torch.as_tensor(input_ids, dtype=torch.int64, device=self.device).reshape(-1).contiguous()
 
     def generate(self, input_ids, max_new_tokens: int) -> torch.Tensor:
         """Returns the generated token ids (device int64 [n]); n = min(max_new_tokens, room left in
         max_seq_len). An empty prompt raises, as the reference reports 'empty_prompt'."""
-        ids = torch.as_tensor(input_ids, dtype=torch.int64, device=self.device).reshape(-1).contiguous()
+        ids = self._ids(input_ids)
         if ids.numel() == 0:
             raise RuntimeError("generate: empty_prompt")
         n = min(max_new_tokens, self.max_seq_len - ids.numel() + 1)   # the last token needs no cache position (as the reference's loop)
@@ -631,9 +645,137 @@ class Decoder:
         torch.cuda.current_stream().wait_stream(self.stream)
         return out[:max(n, 0)]
 
+    def extend(self, input_ids, want=()) -> torch.Tensor:
+        """Appends a portion of given tokens to the sequence; returns the logits [len(want), vocab] at
+        the wanted places of the portion."""
+        ids = self._ids(input_ids)
+        w = (C.c_int32 * max(len(want), 1))(*want)
+        out = torch.empty((len(want), self.vocab), dtype=torch.float32, device=self.device)
+        self.stream.wait_stream(torch.cuda.current_stream())
+        with torch.cuda.stream(self.stream):
+            lib.check(_L.ctdk_decode_extend(self._h, ids.data_ptr(), ids.numel(), w, len(want), out.data_ptr(),
+                                            self.stream.cuda_stream))
+            lib.check(_L.ctdk_device_status(self.stream.cuda_stream, None))
+        torch.cuda.current_stream().wait_stream(self.stream)
+        return out
+
+    def step(self, token: int) -> torch.Tensor:
+        """Feeds one chosen token; returns a copy of the logits it leaves behind."""
+        with torch.cuda.stream(self.stream):
+            lib.check(_L.ctdk_decode_step(self._h, int(token), self.stream.cuda_stream))
+            lib.check(_L.ctdk_device_status(self.stream.cuda_stream, None))
+        return self.last_logits().clone()
+
+    def reset(self) -> None:
+        lib.check(_L.ctdk_decode_reset(self._h, self.stream.cuda_stream))
+
     def last_logits(self) -> torch.Tensor:
         p = C.c_void_p()
         lib.check(_L.ctdk_decode_logits(self._h, C.byref(p)))
         base = self.workspace.data_ptr()
         off = p.value - base
-        return self.workspace[off:off + 4 * self.cfg.vocab_size].view(torch.float32)
+        return self.workspace[off:off + 4 * self.vocab].view(torch.float32)
+
+
+class Decoder(DecoderBase):
+    """Greedy KV-cache generation, batch 1, as ctd_generate with temperature <= 0
+    (tools/ctd_generate/main.cpp:94-184): prefill the prompt, then one token per step."""
+
+    def __init__(self, cfg: ModelConfig, max_seq_len: int, device="cuda:0", params: torch.Tensor | None = None):
+        self.cfg, self.max_seq_len, self.vocab = cfg, max_seq_len, cfg.vocab_size
+        self.device = torch.device(device)
+        self.layout = model_layout(cfg)
+        self.params = params if params is not None else torch.zeros(self.layout.total, dtype=torch.float32,
+                                                                    device=self.device)
+        ws = _L.ctdk_decode_workspace_bytes(C.byref(cfg), max_seq_len)
+        if ws < 0:
+            raise lib.CtdkError(-1, lib.last_error())
+        self.workspace = torch.zeros(ws, dtype=torch.uint8, device=self.device)
+        self._h = C.c_void_p()
+        lib.check(_L.ctdk_decode_create(C.byref(cfg), self.params.data_ptr(), self.workspace.data_ptr(), ws,
+                                        max_seq_len, C.byref(self._h)))
+        self.stream = torch.cuda.Stream(device=self.device)
+
+    def named_parameters(self) -> dict:
+        lo = self.layout
+        return {n: self.params[o:o + k].view(s) for n, s, o, k in zip(lo.names, lo.shapes, lo.offsets, lo.numels)}
+
+    def load_parameters(self, tensors: dict) -> None:
+        for n, v in self.named_parameters().items():
+            src = tensors[n]
+            src = torch.from_numpy(np.ascontiguousarray(src)) if isinstance(src, np.ndarray) else src
+            v.copy_(src.to(torch.float32))
+
+
+class HybridModel:
+    """A layer-list model (ctdk_hybrid_*): config is the parsed config.json, shapes maps tensor names to
+    shapes (or to arrays). dtype "bf16" or "fp32"."""
+
+    def __init__(self, config: dict, shapes: dict, dtype: str = "bf16"):
+        self.config, self.dtype = config, dtype
+        head = {n: {"shape": list(getattr(s, "shape", s))} for n, s in shapes.items()}
+        self._h = C.c_void_p()
+        lib.check(_L.ctdk_hybrid_open(json.dumps(config).encode(), json.dumps(head).encode(), {"fp32": 0, "bf16": 1}[dtype],
+                                      C.byref(self._h)))
+        self.vocab = int(_L.ctdk_hybrid_vocab(self._h))
+        self.arena_bytes = int(_L.ctdk_hybrid_arena_bytes(self._h))
+        self.tensors = []
+        for i in range(_L.ctdk_hybrid_num_tensors(self._h)):
+            t = TensorInfo()
+            lib.check(_L.ctdk_hybrid_tensor(self._h, i, C.byref(t)))
+            self.tensors.append(t)
+
+    @classmethod
+    def from_folder(cls, path, dtype: str = "bf16"):
+        """(model, weights) of a folder with config.json and model.safetensors."""
+        path = Path(path)
+        weights = load_safetensors(path / "model.safetensors")
+        return cls(json.loads((path / "config.json").read_text()), weights, dtype), weights
+
+    def __del__(self):
+        h = getattr(self, "_h", None)
+        if h and _L is not None:
+            _L.ctdk_hybrid_close(h)
+            self._h = None
+
+    def views(self, arena: torch.Tensor) -> dict:
+        """Views of the parameter arena by tensor name, [rows, cols] (vectors [cols])."""
+        out = {}
+        for t in self.tensors:
+            dt = torch.bfloat16 if t.is_matrix and self.dtype == "bf16" else torch.float32
+            size = t.rows * t.ld * (2 if dt == torch.bfloat16 else 4)
+            v = arena[t.offset:t.offset + size].view(dt).view(t.rows, t.ld)[:, :t.cols]
+            out[t.name.decode()] = v
+        return out
+
+
+class HybridDecoder(DecoderBase):
+    """Decoder of a layer-list model; portions of up to max_portion rows run at once."""
+
+    def __init__(self, model: HybridModel, max_seq_len: int, max_portion: int = 4096, device="cuda:0",
+                 params: torch.Tensor | None = None):
+        self.cfg = self.model = model
+        self.max_seq_len, self.vocab = max_seq_len, model.vocab
+        self.device = torch.device(device)
+        self.params = params if params is not None else torch.zeros(model.arena_bytes, dtype=torch.uint8, device=self.device)
+        ws = _L.ctdk_hybrid_workspace_bytes(model._h, max_seq_len, max_portion)
+        if ws < 0:
+            raise lib.CtdkError(-1, lib.last_error())
+        self.workspace = torch.empty(ws, dtype=torch.uint8, device=self.device)
+        self._h = C.c_void_p()
+        lib.check(_L.ctdk_hybrid_decode_create(model._h, self.params.data_ptr(), self.workspace.data_ptr(), ws, max_seq_len,
+                                               max_portion, C.byref(self._h)))
+        self.stream = torch.cuda.Stream(device=self.device)
+
+    def named_parameters(self) -> dict:
+        return self.model.views(self.params)
+
+    def load_parameters(self, tensors: dict) -> None:
+        for n, v in self.named_parameters().items():
+            src = tensors[n]
+            src = torch.from_numpy(np.ascontiguousarray(src)) if isinstance(src, np.ndarray) else src
+            v.copy_(src.to(torch.float32).reshape(v.shape))
+
+    def trace_layers(self, out: torch.Tensor | None) -> None:
+        """out [layers, rows, width] (fp32, device) receives the residual stream of the next portions."""
+        lib.check(_L.ctdk_hybrid_trace_layers(self._h, out.data_ptr() if out is not None else None))

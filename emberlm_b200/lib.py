@@ -52,6 +52,7 @@ _p, _i, _l, _f = C.c_void_p, C.c_int, C.c_int64, C.c_float
 _SIGS = {
     "ctdk_reserve_sms": [_i],
     "ctdk_gemm": [_p, _p, _p, _l, _l, _l, _l, _l, _l, _i, _i, _i, _i, _p, _p],
+    "ctdk_gemm_bf16": [_p, _p, _p, _l, _l, _l, _l, _l, _l, _p],
     "ctdk_gemm_ws": [_p, _p, _p, _l, _l, _l, _l, _l, _l, _i, _i, _i, _i, _p, _p, _l, _p],
     "ctdk_attn_fwd_p": [_p, _p, _p, _l, _l, _i, _i, _i, _i, _p],
     "ctdk_attn_bwd_p": [_p, _p, _p, _p, _p, _p, _l, _l, _i, _i, _i, _i, _p],

@@ -6,7 +6,8 @@ state `*.opt.safetensors`), byte-compatible with emberlm's src/core/safetensors.
   The reference emits header keys in alphabetical order (an ordered JSON object,
   safetensors.cpp:100-115) while data offsets follow the caller's tensor order, and pads the
   header with spaces to a multiple of 8 bytes (safetensors.cpp:118-119). It reads F32 / I64 /
-  I32 and ignores "__metadata__" (safetensors.cpp:55-66); it writes F32 only.
+  I32 and ignores "__metadata__" (safetensors.cpp:55-66); it writes F32 only. BF16 tensors are read too,
+  as fp32 arrays of the same values.
 """
 from __future__ import annotations
 
@@ -53,6 +54,11 @@ def load_safetensors(path) -> dict:
         if name == "__metadata__":
             continue
         dt = spec["dtype"]
+        if dt == "BF16":
+            b, e = spec["data_offsets"]
+            raw = np.frombuffer(data, dtype=np.uint16, count=(e - b) // 2, offset=origin + b)
+            out[name] = (raw.astype(np.uint32) << 16).view(np.float32).reshape(tuple(spec["shape"]))
+            continue
         if dt not in _DTYPES:
             raise RuntimeError(f"safetensors: {name} has dtype {dt} which is not supported on the read path")
         b, e = spec["data_offsets"]

@@ -75,6 +75,11 @@ int ctdk_gemm(const float* A, const float* B, float* C, int64_t M, int64_t N, in
               int64_t lda, int64_t ldb, int64_t ldc, int transa, int transb, int precision,
               int epilogue, const float* aux, void* stream);
 
+/* C[M,N] (fp32, ldc) = A[M,K] B[N,K]^T with bfloat16 operands in memory (lda, ldb in elements, multiples
+ * of 8; 16-byte aligned pointers; N >= 8) and fp32 accumulation: the products of a bfloat16 model. */
+int ctdk_gemm_bf16(const void* A, const void* B, float* C, int64_t M, int64_t N, int64_t K, int64_t lda,
+                   int64_t ldb, int64_t ldc, void* stream);
+
 /* Same as ctdk_gemm with a caller-provided workspace, which CTDK_GEMM_3XTF32 needs to run on the
  * tensor cores: both operands are split into a TF32-exact high part and an fp32 remainder and
  * C = A_hi B_hi + A_hi B_lo + A_lo B_hi is accumulated in three tensor-core passes (relative
@@ -525,7 +530,13 @@ int ctdk_sample(const float* logits, int64_t B, int64_t V, float temperature, in
  *   step    : feeds ONE token chosen by the caller (a sampler, a forced token) at the next
  *             position and leaves the logits of that position behind; not to be mixed with
  *             greedy after the same prefill;
- *   logits  : device pointer to the [vocab] logits of the last processed position.
+ *   logits  : device pointer to the [vocab] logits of the last processed position;
+ *   extend  : appends a portion of T >= 1 given tokens at the next position (after create or reset:
+ *             position 0), on the cache and state that earlier calls left, wherever the portion was
+ *             cut. The logits of its rows want[0, n_want) (host int32) go to want_logits
+ *             [n_want, vocab] (device); n_want < 0 leaves those of the last row behind for
+ *             greedy / step. Not after greedy;
+ *   reset   : an empty sequence again; what it held in the cache or state is given back.
  * ------------------------------------------------------------------------------------ */
 int64_t ctdk_decode_workspace_bytes(const ctdk_model_config* cfg, int64_t max_seq);
 int ctdk_decode_create(const ctdk_model_config* cfg, const float* params, void* workspace,
@@ -535,6 +546,47 @@ int ctdk_decode_prefill(void* decoder, const int64_t* ids, int64_t T, void* stre
 int ctdk_decode_greedy(void* decoder, int64_t n_new, int64_t* out_tokens, void* stream);
 int ctdk_decode_step(void* decoder, int64_t token, void* stream);
 int ctdk_decode_logits(void* decoder, const float** logits);
+int ctdk_decode_extend(void* decoder, const int64_t* ids, int64_t T, const int32_t* want, int64_t n_want,
+                       float* want_logits, void* stream);
+int ctdk_decode_reset(void* decoder, void* stream);
+
+/* ------------------------------------------------------------------------------------
+ * Layer-list decoders ("hybrid" family). The model is described by its config.json: a list of layers,
+ * each with one or two mixer branches (chunked attention with tied keys and values, lightning linear
+ * attention, the delta rule with per-channel decay) and an optional clamped GLU, RMS norms before and
+ * after every sublayer, an untied head. A handle from ctdk_hybrid_open owns the parsed description
+ * (host memory only); it names every tensor and where it lies in the parameter arena, and makes
+ * decoders that all ctdk_decode_* calls above accept.
+ *   config_json   text of config.json;
+ *   tensors_json  JSON object name -> {"shape": [...]} (a safetensors header qualifies): the sizes that
+ *                 the config leaves to the tensors (low-rank widths) and a check of all shapes;
+ *   dtype         CTDK_DTYPE_BF16: matrices and matrix-product inputs in bfloat16, 32-bit sums, and
+ *                 32-bit norms, scores, recurrences, residual; CTDK_DTYPE_F32: everything in fp32.
+ * Arena: matrices are [rows, ld] in the model's dtype (ld >= cols, a multiple of 8, the padding zero),
+ * everything else fp32 [rows, cols]; the caller zero-fills it before loading. max_portion bounds the
+ * rows a prompt pass takes at once (longer portions are cut inside the call).
+ * ------------------------------------------------------------------------------------ */
+#define CTDK_DTYPE_F32 0
+#define CTDK_DTYPE_BF16 1
+typedef struct {
+  char name[96];
+  int64_t rows, cols, ld;   /* elements */
+  int64_t offset;           /* bytes from the start of the arena */
+  int is_matrix;            /* 1: stored in the model's dtype; 0: fp32 */
+} ctdk_tensor_info;
+int ctdk_hybrid_open(const char* config_json, const char* tensors_json, int dtype, void** model);
+int ctdk_hybrid_close(void* model);
+int64_t ctdk_hybrid_num_tensors(void* model);
+int ctdk_hybrid_tensor(void* model, int64_t i, ctdk_tensor_info* out);
+int64_t ctdk_hybrid_arena_bytes(void* model);
+int64_t ctdk_hybrid_vocab(void* model);
+int64_t ctdk_hybrid_workspace_bytes(void* model, int64_t max_seq, int64_t max_portion);
+int ctdk_hybrid_decode_create(void* model, const void* params, void* workspace, int64_t workspace_bytes,
+                              int64_t max_seq, int64_t max_portion, void** decoder);
+/* Copies the residual stream [rows, width] of the last portion's rows to `out` (device, fp32) after
+ * every layer: out[layer][row][width]. NULL switches it off. For tests and debugging; portions of at
+ * most max_portion rows. */
+int ctdk_hybrid_trace_layers(void* decoder, float* out);
 
 #ifdef __cplusplus
 }

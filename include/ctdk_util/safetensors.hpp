@@ -3,8 +3,9 @@
 //   8-byte little-endian header length | JSON header | raw little-endian tensor data
 //   header: {"name": {"dtype": "F32", "shape": [...], "data_offsets": [begin, end]}, ...}
 // The writer emits header keys in alphabetical order, data in the caller's order, and pads the
-// header with spaces to a multiple of 8 bytes (safetensors.cpp:100-119). The reader accepts F32
-// tensors and skips "__metadata__"; other dtypes are reported as unsupported when requested.
+// header with spaces to a multiple of 8 bytes (safetensors.cpp:100-119). The reader skips
+// "__metadata__" and hands out F32 tensors, or the raw 16-bit values of BF16 tensors; other dtypes are
+// reported as unsupported when requested.
 #pragma once
 
 #include <cstdint>
@@ -48,6 +49,7 @@ class File {
     origin_ = 8 + hlen;
     const minijson::Value h = minijson::parse(text);
     if (!h.is_object()) throw std::runtime_error("safetensors: header is not an object: " + path);
+    header_ = text;
     for (const auto& kv : *h.obj) {
       if (kv.first == "__metadata__") continue;
       Entry e;
@@ -63,12 +65,24 @@ class File {
   }
 
   const std::map<std::string, Entry>& entries() const { return entries_; }
+  const std::string& header_text() const { return header_; }
   uint64_t data_origin() const { return origin_; }   // file offset of the data section
   bool has(const std::string& name) const { return entries_.count(name) != 0; }
   const Entry& entry(const std::string& name) const {
     auto it = entries_.find(name);
     if (it == entries_.end()) throw std::runtime_error("safetensors: missing tensor " + name + " in " + path_);
     return it->second;
+  }
+  // Reads a BF16 tensor of exactly `numel` elements as raw 16-bit values.
+  void read_bf16(const std::string& name, uint16_t* dst, int64_t numel) {
+    const Entry& e = entry(name);
+    if (e.dtype != "BF16") throw std::runtime_error("safetensors: " + name + " has dtype " + e.dtype + ", BF16 expected");
+    if (e.numel() != numel || static_cast<int64_t>(e.end - e.begin) != numel * 2)
+      throw std::runtime_error("safetensors: shape mismatch for " + name);
+    in_.clear();
+    in_.seekg(static_cast<std::streamoff>(origin_ + e.begin), std::ios::beg);
+    if (!in_.read(reinterpret_cast<char*>(dst), static_cast<std::streamsize>(numel * 2)))
+      throw std::runtime_error("safetensors: short read on " + name);
   }
   // Reads an F32 tensor of exactly `numel` elements into dst.
   void read_f32(const std::string& name, float* dst, int64_t numel) {
@@ -85,6 +99,7 @@ class File {
  private:
   std::string path_;
   std::ifstream in_;
+  std::string header_;
   uint64_t origin_ = 0;
   std::map<std::string, Entry> entries_;
 };

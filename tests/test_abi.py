@@ -18,9 +18,10 @@ def test_ctypes_signature_table_covers_header():
                "ctdk_prof_collect", "ctdk_gemm_3xtf32_workspace_floats", "ctdk_sample_workspace_bytes"}
     # engine / trainer / decoder entry points are bound in emberlm_b200/engine.py
     engine = {n for n in lib.declared_symbols()
-              if n.startswith(("ctdk_engine_", "ctdk_model_", "ctdk_decode_", "ctdk_trainer_", "ctdk_dp_", "ctdk_batch_"))}
+              if n.startswith(("ctdk_engine_", "ctdk_model_", "ctdk_decode_", "ctdk_trainer_", "ctdk_dp_", "ctdk_batch_",
+                            "ctdk_hybrid_"))}
     from emberlm_b200 import engine as E
-    assert all(getattr(E._L, n).argtypes is not None for n in engine if n.startswith(("ctdk_trainer_", "ctdk_dp_", "ctdk_batch_")))
+    assert all(getattr(E._L, n).argtypes is not None for n in engine if n.startswith(("ctdk_trainer_", "ctdk_dp_", "ctdk_batch_", "ctdk_hybrid_")))
     assert set(lib.declared_symbols()) - special - engine - set(lib._SIGS) == set()
 
 
