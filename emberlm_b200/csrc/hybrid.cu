@@ -7,6 +7,7 @@
 // last inputs (slot = position mod taps). Position 0 starts from nothing whatever these buffers hold,
 // so a reset costs no device work.
 #include <algorithm>
+#include <cmath>
 #include <new>
 #include <vector>
 
@@ -33,7 +34,8 @@ struct BranchBuffers {
   void* cache = nullptr;        // attention
   int64_t chunk = 0;            // cache rows: the chunk, or max_seq when that is smaller
   int rope = -1;                // index of the rotation table
-  float* decay = nullptr;       // lightning
+  float* decay = nullptr;       // lightning: per head; then its powers 0 .. 64 per head
+  float* powers = nullptr;
   float* state = nullptr;
   float* ring = nullptr;
 };
@@ -44,6 +46,8 @@ struct RopeTable {
   float2* table = nullptr;
   double* freqs = nullptr;
 };
+
+constexpr int64_t kChunkedRows = 16;   // shorter portions run the recurrences token by token
 
 int padded_head(int dim, bool tensor_cores) {
   if (!tensor_cores) return (dim + 3) / 4 * 4;
@@ -62,6 +66,8 @@ struct HybridDecoder : DecoderBase {
   // prompt-pass buffers, rows = max_portion
   float *x, *proj, *packed, *attn_out, *o32, *y1, *y2, *gu, *dq, *dk, *dv, *dlog, *dbeta, *dz, *dgate;
   T *h, *mixed, *mixed2, *act, *low_a, *low_g;
+  float *chunk_state, *cw, *ckh, *cqt, *cu, *cscores, *cdecay;
+  __nv_bfloat16 *qb, *kb, *vb;
   int32_t* want_dev;
   // token-pass buffers
   float *tx[2], *tproj, *tout[2], *tgate, *ty1, *ty2, *tgu, *tpart;
@@ -76,6 +82,8 @@ struct HybridDecoder : DecoderBase {
   const U* at(int64_t off) const { return reinterpret_cast<const U*>(params + off); }
   const float* vec(int64_t off) const { return at<float>(off); }
   bool tensor_core_attention(const Branch& b) const { return m.dtype == CTDK_DTYPE_BF16 && b.dim <= 128; }
+
+  bool chunked_lightning(const Branch& b) const { return m.dtype == CTDK_DTYPE_BF16 && lightning_chunked_ok(b.dim, b.vdim); }
 
   int carve(Bump& b);
   int build_phases();
@@ -97,6 +105,8 @@ template <typename T>
 int HybridDecoder<T>::carve(Bump& b) {
   const int64_t R = max_portion, W = m.width;
   int64_t n_in = 8, mix = 8, heads_out = 8, packed_n = 0, attn_n = 0, ff = 8, parts = 0, arrives = 0;
+  int64_t ck_n = 0, cv_n = 0, cs_n = 0, cd_n = 0;
+  int64_t chunk_n = 0, qk_tiles = 0, v_tiles = 0;
   int64_t qk = 0, dv_n = 0, dlog_n = 0, db_n = 0, rank = 8, rank_g = 8, gate_n = 0;
   bufs.assign(m.layers.size(), {});
   ropes.clear();
@@ -133,12 +143,29 @@ int HybridDecoder<T>::carve(Bump& b) {
         bb.state = b.floats(static_cast<int64_t>(br.heads) * br.dim * br.vdim);
         if (br.kind == BranchKind::kLightning) {
           bb.decay = b.floats(br.heads);
+          bb.powers = b.floats(static_cast<int64_t>(br.heads) * (kLightningChunk + 1));
+          if (chunked_lightning(br)) {
+            const int64_t tiles = ((R + kLightningChunk - 1) / kLightningChunk) * br.heads;
+            const int64_t dk = lightning_tile(br.dim), dv = lightning_tile(br.vdim);
+            chunk_n = std::max(chunk_n, tiles * dk * dv);
+            qk_tiles = std::max(qk_tiles, tiles * kLightningChunk * dk);
+            v_tiles = std::max(v_tiles, tiles * kLightningChunk * dv);
+          }
         } else {
           bb.ring = b.floats(static_cast<int64_t>(br.taps) * (2 * br.kv_heads * br.dim + out_n));
           qk = std::max<int64_t>(qk, static_cast<int64_t>(br.kv_heads) * br.dim);
           dv_n = std::max<int64_t>(dv_n, out_n);
           dlog_n = std::max<int64_t>(dlog_n, pad8(static_cast<int64_t>(br.heads) * br.dim));
           gate_n = std::max<int64_t>(gate_n, pad8(out_n));
+          if (delta_chunked_ok(br.dim, br.vdim)) {
+            const int64_t tiles = ((R + kDeltaChunk - 1) / kDeltaChunk) * br.heads;
+            const int64_t tk = lightning_tile(br.dim), tv = lightning_tile(br.vdim);
+            chunk_n = std::max(chunk_n, tiles * tk * tv);
+            ck_n = std::max(ck_n, tiles * kDeltaChunk * tk);
+            cv_n = std::max(cv_n, tiles * kDeltaChunk * tv);
+            cs_n = std::max(cs_n, tiles * kDeltaChunk * kDeltaChunk);
+            cd_n = std::max(cd_n, tiles * tk);
+          }
           db_n = std::max<int64_t>(db_n, br.heads);
           rank = std::max<int64_t>(rank, pad8(br.rank_a));
           rank_g = std::max<int64_t>(rank_g, pad8(br.rank_g));
@@ -168,6 +195,16 @@ int HybridDecoder<T>::carve(Bump& b) {
   dbeta = b.floats(R * db_n);
   low_a = typed(R * rank);
   low_g = typed(R * rank_g);
+  chunk_state = b.floats(chunk_n);
+  cw = b.floats(ck_n);
+  ckh = b.floats(ck_n);
+  cqt = b.floats(ck_n);
+  cu = b.floats(cv_n);
+  cscores = b.floats(cs_n);
+  cdecay = b.floats(cd_n);
+  qb = static_cast<__nv_bfloat16*>(b.bytes(qk_tiles * 2));
+  kb = static_cast<__nv_bfloat16*>(b.bytes(qk_tiles * 2));
+  vb = static_cast<__nv_bfloat16*>(b.bytes(v_tiles * 2));
   want_dev = static_cast<int32_t*>(b.bytes(R * 4));
 
   tx[0] = b.floats(W);
@@ -358,10 +395,18 @@ int HybridDecoder<T>::build_phases() {
 template <typename T>
 int HybridDecoder<T>::upload(cudaStream_t s) {
   auto copy = [&](void* dst, const void* src, size_t n) { return cudaMemcpyAsync(dst, src, n, cudaMemcpyHostToDevice, s) == cudaSuccess; };
+  std::vector<std::vector<float>> powers;
   bool ok = copy(phases_dev, phases.data(), phases.size() * sizeof(TokenPhase));
   for (size_t l = 0; l < m.layers.size(); ++l)
     for (size_t b = 0; b < bufs[l].size(); ++b)
-      if (bufs[l][b].decay != nullptr) ok = ok && copy(bufs[l][b].decay, m.layers[l].branches[b].decay.data(), m.layers[l].branches[b].decay.size() * 4);
+      if (bufs[l][b].decay != nullptr) {
+        const std::vector<float>& d = m.layers[l].branches[b].decay;
+        powers.emplace_back();
+        for (const float x : d)
+          for (int i = 0; i <= kLightningChunk; ++i) powers.back().push_back(static_cast<float>(std::pow(static_cast<double>(x), i)));
+        ok = ok && copy(bufs[l][b].powers, powers.back().data(), powers.back().size() * 4);
+        ok = ok && copy(bufs[l][b].decay, d.data(), d.size() * 4);
+      }
   std::vector<std::vector<double>> freqs;
   for (RopeTable& r : ropes) {
     std::vector<double> f(r.spec.dims / 2);
@@ -408,21 +453,42 @@ int HybridDecoder<T>::mixer_attention(const Branch& b, const BranchBuffers& bb, 
 template <typename T>
 int HybridDecoder<T>::mixer_lightning(const Branch& b, const BranchBuffers& bb, int64_t n, int64_t pos, float* y, int64_t ldp,
                                       cudaStream_t s) {
-  ScanArgs a;
-  a.q = proj + b.col_q;
-  a.k = proj + b.col_k;
-  a.v = proj + b.col_v;
-  a.ldq = a.ldk = a.ldv = ldp;
-  a.decay = bb.decay;
-  a.silu = 1;
-  a.state = bb.state;
-  a.out = o32;
-  a.H = a.G = b.heads;
-  a.dim = b.dim;
-  a.vdim = b.vdim;
-  a.rows = n;
-  a.resume = pos > 0;
-  DTRY(recurrent_scan(a, false, s));
+  if (chunked_lightning(b) && n >= kChunkedRows) {
+    LightningArgs a;
+    a.q = proj + b.col_q;
+    a.k = proj + b.col_k;
+    a.v = proj + b.col_v;
+    a.ldp = ldp;
+    a.powers = bb.powers;
+    a.state = bb.state;
+    a.chunk_state = chunk_state;
+    a.out = o32;
+    a.qb = qb;
+    a.kb = kb;
+    a.vb = vb;
+    a.H = b.heads;
+    a.dim = b.dim;
+    a.vdim = b.vdim;
+    a.rows = n;
+    a.resume = pos > 0;
+    DTRY(lightning_chunked(a, s));
+  } else {
+    ScanArgs a;
+    a.q = proj + b.col_q;
+    a.k = proj + b.col_k;
+    a.v = proj + b.col_v;
+    a.ldq = a.ldk = a.ldv = ldp;
+    a.decay = bb.decay;
+    a.silu = 1;
+    a.state = bb.state;
+    a.out = o32;
+    a.H = a.G = b.heads;
+    a.dim = b.dim;
+    a.vdim = b.vdim;
+    a.rows = n;
+    a.resume = pos > 0;
+    DTRY(recurrent_scan(a, false, s));
+  }
   const int cols = b.heads * b.vdim;
   DTRY(gated_norm_rows(o32, vec(b.w_norm), proj + b.col_g, ldp, mixed, b.ld_o, n, cols, m.eps, s));
   return gemm_rows(mixed, at<T>(b.w_o), y, n, m.width, cols, b.ld_o, b.ld_o, m.width, s);
@@ -465,23 +531,48 @@ int HybridDecoder<T>::mixer_delta(const Branch& b, const BranchBuffers& bb, int6
   p.pos = pos;
   DTRY(delta_prep(p, s));
   DTRY(delta_ring_store(p, s));
-  ScanArgs a;
-  a.q = dq;
-  a.k = dk;
-  a.v = dv;
-  a.ldq = a.ldk = static_cast<int64_t>(b.kv_heads) * b.dim;
-  a.ldv = static_cast<int64_t>(b.heads) * b.vdim;
-  a.logg = dlog;
-  a.beta = dbeta;
-  a.state = bb.state;
-  a.out = o32;
-  a.H = b.heads;
-  a.G = b.kv_heads;
-  a.dim = b.dim;
-  a.vdim = b.vdim;
-  a.rows = n;
-  a.resume = pos > 0;
-  DTRY(recurrent_scan(a, true, s));
+  if (delta_chunked_ok(b.dim, b.vdim) && n >= kChunkedRows) {
+    DeltaChunkArgs a;
+    a.q = dq;
+    a.k = dk;
+    a.v = dv;
+    a.logg = dlog;
+    a.beta = dbeta;
+    a.state = bb.state;
+    a.out = o32;
+    a.w = cw;
+    a.kh = ckh;
+    a.qt = cqt;
+    a.u = cu;
+    a.scores = cscores;
+    a.decay = cdecay;
+    a.chunk_state = chunk_state;
+    a.H = b.heads;
+    a.G = b.kv_heads;
+    a.dim = b.dim;
+    a.vdim = b.vdim;
+    a.rows = n;
+    a.resume = pos > 0;
+    DTRY(delta_chunked(a, s));
+  } else {
+    ScanArgs a;
+    a.q = dq;
+    a.k = dk;
+    a.v = dv;
+    a.ldq = a.ldk = static_cast<int64_t>(b.kv_heads) * b.dim;
+    a.ldv = static_cast<int64_t>(b.heads) * b.vdim;
+    a.logg = dlog;
+    a.beta = dbeta;
+    a.state = bb.state;
+    a.out = o32;
+    a.H = b.heads;
+    a.G = b.kv_heads;
+    a.dim = b.dim;
+    a.vdim = b.vdim;
+    a.rows = n;
+    a.resume = pos > 0;
+    DTRY(recurrent_scan(a, true, s));
+  }
   DTRY(gated_head_norm_rows(o32, vec(b.w_norm), dgate, ldg, mixed, b.ld_o, n, b.heads, b.vdim, m.eps, s));
   return gemm_rows(mixed, at<T>(b.w_o), y, n, m.width, static_cast<int64_t>(b.heads) * b.vdim, b.ld_o, b.ld_o, m.width, s);
 }

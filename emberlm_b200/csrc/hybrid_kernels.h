@@ -90,6 +90,39 @@ struct ScanArgs {
 };
 int recurrent_scan(const ScanArgs& a, bool delta, cudaStream_t s);
 
+// Chunk-parallel lightning attention (bfloat16 models): q, k, v are columns of the projection (before
+// silu), powers[h][i] = decay_h^i for i in [0, 64]. Scratch: chunk_state [chunks][H][dk][dv] floats,
+// qb / kb [chunks][H][64][dk], vb [chunks][H][64][dv] with dk, dv the tile sizes of lightning_tile().
+constexpr int kLightningChunk = 64;
+struct LightningArgs {
+  const float *q = nullptr, *k = nullptr, *v = nullptr;
+  int64_t ldp = 0;
+  const float* powers = nullptr;
+  float *state = nullptr, *chunk_state = nullptr, *out = nullptr;
+  __nv_bfloat16 *qb = nullptr, *kb = nullptr, *vb = nullptr;
+  int H = 0, dim = 0, vdim = 0;
+  int64_t rows = 0;
+  int resume = 0;
+};
+// Chunk-parallel delta rule: inputs as for recurrent_scan (q, k [rows][G * dim], v [rows][H * vdim], logg
+// [rows][H * dim], beta [rows][H], dense). Scratch per (chunk, head), dk / dv the tile sizes: w, kh, qt
+// [64][dk], u [64][dv], scores [64][64], decay [dk], chunk_state [dk][dv].
+constexpr int kDeltaChunk = 64;
+struct DeltaChunkArgs {
+  const float *q = nullptr, *k = nullptr, *v = nullptr, *logg = nullptr, *beta = nullptr;
+  float *state = nullptr, *out = nullptr;
+  float *w = nullptr, *kh = nullptr, *qt = nullptr, *u = nullptr, *scores = nullptr, *decay = nullptr, *chunk_state = nullptr;
+  int H = 0, G = 0, dim = 0, vdim = 0;
+  int64_t rows = 0;
+  int resume = 0;
+};
+bool delta_chunked_ok(int dim, int vdim);
+int delta_chunked(const DeltaChunkArgs& a, cudaStream_t s);
+
+bool lightning_chunked_ok(int dim, int vdim);
+inline int lightning_tile(int d) { return d <= 64 ? 64 : 128; }
+int lightning_chunked(const LightningArgs& a, cudaStream_t s);
+
 // rms over all H * vdim columns, * w * sigmoid(gate)
 template <typename T>
 int gated_norm_rows(const float* o, const float* w, const float* gate, int64_t ldg, T* dst, int64_t ld, int64_t rows, int n, float eps,

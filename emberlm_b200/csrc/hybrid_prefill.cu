@@ -363,6 +363,80 @@ __global__ void __launch_bounds__(256) delta_prep_kernel(const DeltaPrepArgs a) 
   }
 }
 
+// The same for four taps with a sliding window: one warp per (unit, run of kRun rows), so that a
+// projection row is read once. E = ceil(max(dim, vdim) / 32) channels per lane.
+constexpr int kRun = 8;
+template <int E>
+__global__ void __launch_bounds__(256) delta_prep4_kernel(const DeltaPrepArgs a) {
+  pdl_launch();
+  pdl_wait();
+  const int lane = threadIdx.x & 31;
+  const int units = 2 * a.G + 2 * a.H, qk = a.G * a.dim, ring_ld = 2 * qk + a.H * a.vdim;
+  const int64_t runs = (a.rows + kRun - 1) / kRun, n = runs * units, nw = static_cast<int64_t>(gridDim.x) * 8;
+  const float qscale = rsqrtf(static_cast<float>(a.dim));
+  for (int64_t i = (static_cast<int64_t>(blockIdx.x) * 256 + threadIdx.x) >> 5; i < n; i += nw) {
+    const int u = static_cast<int>(i % units);
+    const int64_t t0 = i / units * kRun, t1 = t0 + kRun < a.rows ? t0 + kRun : a.rows;
+    if (u >= 2 * a.G + a.H) {   // decays and beta
+      const int head = u - 2 * a.G - a.H;
+      const float amp = -expf(a.a_log[head]);
+      for (int64_t t = t0; t < t1; ++t)
+        for (int d = lane; d < a.dim; d += 32) {
+          const int c = head * a.dim + d;
+          a.logg[t * a.H * a.dim + c] = amp * softplus_f(a.z[t * a.ldz + c] + a.dt_bias[c]);
+        }
+      if (t0 + lane < t1) a.beta[(t0 + lane) * a.H + head] = sigmoid_f(a.proj[(t0 + lane) * a.ldp + a.col_b + head]);
+      continue;
+    }
+    const int kind = u < a.G ? 0 : (u < 2 * a.G ? 1 : 2);
+    const int head = kind == 0 ? u : (kind == 1 ? u - a.G : u - 2 * a.G);
+    const int width = kind == 2 ? a.vdim : a.dim;
+    const int col = (kind == 0 ? a.col_q : (kind == 1 ? a.col_k : a.col_v)) + head * width;
+    const int ring_c = (kind == 0 ? 0 : (kind == 1 ? qk : 2 * qk)) + head * width;
+    const float* taps = (kind == 0 ? a.conv_q : (kind == 1 ? a.conv_k : a.conv_v)) + static_cast<int64_t>(head) * width * 4;
+    float4 w[E];
+    float x0[E], x1[E], x2[E];   // inputs three, two and one rows back
+    auto before = [&](int64_t t, int d) {
+      if (t >= 0) return a.proj[t * a.ldp + col + d];
+      const int64_t p = a.pos + t;
+      return p < 0 ? 0.0f : a.ring[(p & 3) * ring_ld + ring_c + d];
+    };
+#pragma unroll
+    for (int e = 0; e < E; ++e) {
+      const int d = lane + 32 * e;
+      w[e] = make_float4(0.f, 0.f, 0.f, 0.f);
+      x0[e] = x1[e] = x2[e] = 0.0f;
+      if (d < width) {
+        w[e] = *reinterpret_cast<const float4*>(taps + static_cast<int64_t>(d) * 4);
+        x0[e] = before(t0 - 3, d);
+        x1[e] = before(t0 - 2, d);
+        x2[e] = before(t0 - 1, d);
+      }
+    }
+    for (int64_t t = t0; t < t1; ++t) {
+      float y[E], ss = 0.0f;
+#pragma unroll
+      for (int e = 0; e < E; ++e) {
+        const int d = lane + 32 * e;
+        const float x = d < width ? a.proj[t * a.ldp + col + d] : 0.0f;
+        y[e] = silu_f(fmaf(w[e].w, x, fmaf(w[e].z, x2[e], fmaf(w[e].y, x1[e], w[e].x * x0[e]))));
+        ss += y[e] * y[e];
+        x0[e] = x1[e];
+        x1[e] = x2[e];
+        x2[e] = x;
+      }
+      float sc = 1.0f;
+      if (kind < 2) sc = rsqrtf(warp_sum(ss) + 1e-6f) * (kind == 0 ? qscale : 1.0f);
+      float* dst = kind == 2 ? a.v + t * a.H * a.vdim + head * width : (kind == 0 ? a.q : a.k) + t * qk + head * width;
+#pragma unroll
+      for (int e = 0; e < E; ++e) {
+        const int d = lane + 32 * e;
+        if (d < width) dst[d] = y[e] * sc;
+      }
+    }
+  }
+}
+
 __global__ void __launch_bounds__(256) delta_ring_store_kernel(const DeltaPrepArgs a) {
   pdl_launch();
   pdl_wait();
@@ -448,6 +522,13 @@ int gated_head_norm_rows(const float* o, const float* w, const float* gate, int6
   LAUNCH("hybrid head norm", gated_head_norm_kernel<T>, row_grid(rows * H, 8), 0, o, w, gate, ldg, dst, ld, rows, H, vdim, eps);
 }
 int delta_prep(const DeltaPrepArgs& a, cudaStream_t s) {
+  const int wide = a.dim > a.vdim ? a.dim : a.vdim;
+  if (a.taps == 4 && wide <= 128) {
+    const int grid = row_grid((a.rows + kRun - 1) / kRun * (2 * a.G + 2 * a.H), 8);
+    if (wide <= 32) LAUNCH("delta prep", delta_prep4_kernel<1>, grid, 0, a);
+    if (wide <= 64) LAUNCH("delta prep", delta_prep4_kernel<2>, grid, 0, a);
+    LAUNCH("delta prep", delta_prep4_kernel<4>, grid, 0, a);
+  }
   LAUNCH("delta prep", delta_prep_kernel, row_grid(a.rows * (2 * a.G + 2 * a.H), 8), 0, a);
 }
 int delta_ring_store(const DeltaPrepArgs& a, cudaStream_t s) {
