@@ -69,7 +69,7 @@ struct LocalCfg {
 
 // grid (chunks, heads), 512 threads.
 template <int DK, int DV>
-__global__ void __launch_bounds__(512) delta_local_kernel(const DeltaChunkArgs a) {
+__global__ void __launch_bounds__(512, 1) delta_local_kernel(const DeltaChunkArgs a) {
   using Cfg = LocalCfg<DK, DV>;
   constexpr int LD = Cfg::LD, LV = Cfg::LV;
   extern __shared__ __align__(16) float sm[];
@@ -89,18 +89,30 @@ __global__ void __launch_bounds__(512) delta_local_kernel(const DeltaChunkArgs a
   const int64_t t0 = static_cast<int64_t>(c) * C, tile = static_cast<int64_t>(c) * a.H + h;
   const int n = static_cast<int>(a.rows - t0 < C ? a.rows - t0 : C);
 
-  for (int i = tid; i < C * DK; i += 512) {
-    const int r = i / DK, d = i % DK;
-    float q = 0.0f, k = 0.0f, g = 0.0f;
-    if (r < n && d < a.dim) {
-      const int64_t at = (t0 + r) * a.G * a.dim + grp * a.dim + d;
-      q = a.q[at];
-      k = a.k[at];
-      g = a.logg[((t0 + r) * a.H + h) * a.dim + d] * kLog2e;
-    }
-    q_s[r * LD + d] = q;
-    k_s[r * LD + d] = k;
-    b_s[r * LD + d] = g;
+  // four columns per thread and turn; head sizes that are not multiples of four load one by one
+  auto fetch = [](const float* p, int left, bool vec) {
+    float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (left <= 0) return x;
+    if (vec) return ld4(p);
+    x.x = p[0];
+    if (left > 1) x.y = p[1];
+    if (left > 2) x.z = p[2];
+    if (left > 3) x.w = p[3];
+    return x;
+  };
+  const bool vec_k = a.dim % 4 == 0, vec_v = a.vdim % 4 == 0;
+  constexpr int KT = C * DK / 2048, VT = C * DV / 2048;   // turns
+#pragma unroll
+  for (int u = 0; u < KT; ++u) {
+    const int i = (tid + u * 512) * 4, r = i / DK, d = i % DK;
+    const int left = r < n ? a.dim - d : 0;
+    const int64_t at = (t0 + r) * a.G * a.dim + grp * a.dim + d;
+    const float4 q = fetch(a.q + at, left, vec_k), k = fetch(a.k + at, left, vec_k);
+    float4 g = fetch(a.logg + ((t0 + r) * a.H + h) * a.dim + d, left, vec_k);
+    g = make_float4(g.x * kLog2e, g.y * kLog2e, g.z * kLog2e, g.w * kLog2e);
+    store4(q_s + r * LD + d, q);
+    store4(k_s + r * LD + d, k);
+    store4(b_s + r * LD + d, g);
   }
   if (tid < C) be[tid] = tid < n ? a.beta[(t0 + tid) * a.H + h] : 0.0f;
   for (int i = tid; i < C * LT; i += 512) L_s[i] = X_s[i] = 0.0f;
@@ -125,15 +137,17 @@ __global__ void __launch_bounds__(512) delta_local_kernel(const DeltaChunkArgs a
   // pairs in different 16-row blocks
   for (int I = 1; I < 4; ++I) {
     const float* ref = b_s + (16 * I - 1) * LD;
-    for (int i = tid; i < 16 * DK; i += 512) {
+    for (int i = tid * 4; i < 16 * (I + 1) * DK; i += 2048) {   // rows before the block, then its own
       const int r = i / DK, d = i % DK;
-      const float e = ex2(b_s[(16 * I + r) * LD + d] - ref[d]);
-      kr[r * LD + d] = k_s[(16 * I + r) * LD + d] * e;
-      qr[r * LD + d] = q_s[(16 * I + r) * LD + d] * e;
-    }
-    for (int i = tid; i < 16 * I * DK; i += 512) {
-      const int r = i / DK, d = i % DK;
-      kx[r * LD + d] = k_s[r * LD + d] * ex2(ref[d] - b_s[r * LD + d]);
+      const float4 z = ld4(ref + d), b = ld4(b_s + r * LD + d), k = ld4(k_s + r * LD + d);
+      if (r < 16 * I) {
+        store4(kx + r * LD + d, make_float4(k.x * ex2(z.x - b.x), k.y * ex2(z.y - b.y), k.z * ex2(z.z - b.z), k.w * ex2(z.w - b.w)));
+      } else {
+        const float4 q = ld4(q_s + r * LD + d);
+        const float4 e = make_float4(ex2(b.x - z.x), ex2(b.y - z.y), ex2(b.z - z.z), ex2(b.w - z.w));
+        store4(kr + (r - 16 * I) * LD + d, make_float4(k.x * e.x, k.y * e.y, k.z * e.z, k.w * e.w));
+        store4(qr + (r - 16 * I) * LD + d, make_float4(q.x * e.x, q.y * e.y, q.z * e.z, q.w * e.w));
+      }
     }
     __syncthreads();
     const int cols = 16 * I;
@@ -157,14 +171,18 @@ __global__ void __launch_bounds__(512) delta_local_kernel(const DeltaChunkArgs a
     __syncthreads();
   }
   {   // pairs inside a block: four columns per item, two threads share the channels
-    const int half = tid & 1, item = tid >> 1, jq = item & 3, i = item >> 2, blk = i & ~15;
+    // A warp takes four neighbouring rows i and only the column steps u that reach below their diagonal;
+    // the row groups are dealt so that every scheduler gets long and short ones.
+    const int half = tid & 1, jq = (tid >> 1) & 3, w = tid >> 5;
+    const int blk = w >> 2 << 4, ig = ((w >> 2) + w) & 3, i = blk + 4 * ig + ((tid >> 3) & 3);
     float ak[4] = {0, 0, 0, 0}, aq[4] = {0, 0, 0, 0};
-    if (blk + jq <= i) {
+    {
 #pragma unroll 2
       for (int d = half * 4; d < DK; d += 8) {
         const float4 bi = ld4(b_s + i * LD + d), ki = ld4(k_s + i * LD + d), qi = ld4(q_s + i * LD + d);
 #pragma unroll
         for (int u = 0; u < 4; ++u) {
+          if (u > ig) break;
           const int j = blk + jq + 4 * u;
           const float4 bj = ld4(b_s + j * LD + d), kj = ld4(k_s + j * LD + d);
           const float e0 = kj.x * ex2(bi.x - bj.x), e1 = kj.y * ex2(bi.y - bj.y), e2 = kj.z * ex2(bi.z - bj.z),
@@ -222,19 +240,29 @@ __global__ void __launch_bounds__(512) delta_local_kernel(const DeltaChunkArgs a
     __syncthreads();
   }
   for (int p = tid; p < C * C; p += 512) X_s[(p / C) * LT + p % C] *= be[p % C];
-  // what the state and output kernels multiply with
-  for (int i = tid; i < C * DK; i += 512) {
-    const int r = i / DK, d = i % DK;
-    const float b = b_s[r * LD + d], k = k_s[r * LD + d];
-    a.kh[tile * (C * DK) + i] = k * ex2(b_s[(C - 1) * LD + d] - b);
-    a.qt[tile * (C * DK) + i] = q_s[r * LD + d] * ex2(b);
-    k_s[r * LD + d] = k * ex2(b);
-    if (r == 0) a.decay[tile * DK + d] = ex2(b_s[(C - 1) * LD + d]);
+  // what the state and output kernels multiply with; the values replace q
+  float4 val[VT];
+#pragma unroll
+  for (int u = 0; u < VT; ++u) {
+    const int i = (tid + u * 512) * 4, r = i / DV, d = i % DV;
+    val[u] = fetch(a.v + (t0 + r) * a.H * a.vdim + h * a.vdim + d, r < n ? a.vdim - d : 0, vec_v);
+  }
+#pragma unroll
+  for (int u = 0; u < KT; ++u) {
+    const int i = (tid + u * 512) * 4, r = i / DK, d = i % DK;
+    const float4 b = ld4(b_s + r * LD + d), k = ld4(k_s + r * LD + d), q = ld4(q_s + r * LD + d), z = ld4(b_s + (C - 1) * LD + d);
+    const float4 e = make_float4(ex2(b.x), ex2(b.y), ex2(b.z), ex2(b.w));
+    store4(a.kh + tile * (C * DK) + i,
+           make_float4(k.x * ex2(z.x - b.x), k.y * ex2(z.y - b.y), k.z * ex2(z.z - b.z), k.w * ex2(z.w - b.w)));
+    store4(a.qt + tile * (C * DK) + i, make_float4(q.x * e.x, q.y * e.y, q.z * e.z, q.w * e.w));
+    store4(k_s + r * LD + d, make_float4(k.x * e.x, k.y * e.y, k.z * e.z, k.w * e.w));
+    if (r == C - 1) store4(a.decay + tile * DK + d, e);
   }
   __syncthreads();
-  for (int i = tid; i < C * DV; i += 512) {
-    const int r = i / DV, d = i % DV;
-    q_s[r * LV + d] = (r < n && d < a.vdim) ? a.v[(t0 + r) * a.H * a.vdim + h * a.vdim + d] : 0.0f;
+#pragma unroll
+  for (int u = 0; u < VT; ++u) {
+    const int i = (tid + u * 512) * 4, r = i / DV, d = i % DV;
+    store4(q_s + r * LV + d, val[u]);
   }
   __syncthreads();
   for (int it = tid; it < 16 * (DK / 4); it += 512) {
@@ -265,9 +293,10 @@ struct StateCfg {
   static constexpr int kFloats = 2 * kStage + DK * LN + C * LN;
 };
 
-// grid (DV / 16, heads), 256 threads: U = T V - W S and the state, chunk after chunk.
+// grid (DV / 16, heads), 512 threads: U = T V - W S and the state, chunk after chunk.
+constexpr int kStateThreads = 512;
 template <int DK, int DV>
-__global__ void __launch_bounds__(256) delta_state_kernel(const DeltaChunkArgs a, int chunks) {
+__global__ void __launch_bounds__(kStateThreads, 1) delta_state_kernel(const DeltaChunkArgs a, int chunks) {
   using Cfg = StateCfg<DK>;
   constexpr int LD = Cfg::LD;
   extern __shared__ __align__(16) float sm[];
@@ -281,26 +310,26 @@ __global__ void __launch_bounds__(256) delta_state_kernel(const DeltaChunkArgs a
     const int64_t tile = static_cast<int64_t>(c) * a.H + h;
     const float* w = a.w + tile * (C * DK);
     const float* kh = a.kh + tile * (C * DK);
-    for (int i = tid; i < C * (DK / 4); i += 256) {
+    for (int i = tid; i < C * (DK / 4); i += kStateThreads) {
       const int r = i / (DK / 4), p = i % (DK / 4) * 4;
       cp_async16(st + r * LD + p, w + r * DK + p);
       cp_async16(st + (C + r) * LD + p, kh + r * DK + p);
     }
     float* us = st + 2 * C * LD;
-    {
+    if (tid < C * 4) {
       const int r = tid >> 2, p = (tid & 3) * 4;
       cp_async16(us + r * LN + p, a.u + tile * (C * DV) + r * DV + c0 + p);
     }
     if (tid < DK / 4) cp_async16(us + C * LN + tid * 4, a.decay + tile * DK + tid * 4);
     cp_async_commit();
   };
-  // a thread owns state rows k0 .. k0 + 3, columns s0, s0 + 1
-  const int k0 = tid / 8 * 4, s0 = (tid & 7) * 2;
+  // a thread owns state rows k0, k0 + 1, columns s0, s0 + 1
+  const int k0 = tid / 8 * 2, s0 = (tid & 7) * 2;
   const bool owner = k0 < DK;
-  float S[4][2] = {};
+  float S[2][2] = {};
   if (owner) {
 #pragma unroll
-    for (int e = 0; e < 4; ++e)
+    for (int e = 0; e < 2; ++e)
 #pragma unroll
       for (int f = 0; f < 2; ++f) {
         const int r = k0 + e, col = c0 + s0 + f;
@@ -309,7 +338,8 @@ __global__ void __launch_bounds__(256) delta_state_kernel(const DeltaChunkArgs a
       }
   }
   load(0);
-  const int ur = tid >> 2, uc = (tid & 3) * 4;
+  // for U: row ur, columns uc .. uc + 3, and half of the key channels (neighbouring lanes add up)
+  const int ur = tid >> 3, uc = ((tid >> 1) & 3) * 4, kh2 = (tid & 1) * 4;
   for (int c = 0; c < chunks; ++c) {
     const int64_t tile = static_cast<int64_t>(c) * a.H + h;
     if (c + 1 < chunks) {
@@ -325,47 +355,51 @@ __global__ void __launch_bounds__(256) delta_state_kernel(const DeltaChunkArgs a
     const float* dec = Uv + C * LN;
     if (owner)
 #pragma unroll
-      for (int e = 0; e < 4; ++e)
+      for (int e = 0; e < 2; ++e)
         *reinterpret_cast<float2*>(a.chunk_state + tile * (DK * DV) + (k0 + e) * DV + c0 + s0) = make_float2(S[e][0], S[e][1]);
     float u[4] = {}, u2[4] = {};
-#pragma unroll 4
-    for (int k = 0; k < DK; k += 4) {
+#pragma unroll 8
+    for (int k = kh2; k < DK; k += 8) {
       const float4 w = ld4(W + ur * LD + k);
       axpy4(w.x, ld4(S_s + k * LN + uc), u);
       axpy4(w.y, ld4(S_s + (k + 1) * LN + uc), u2);
       axpy4(w.z, ld4(S_s + (k + 2) * LN + uc), u);
       axpy4(w.w, ld4(S_s + (k + 3) * LN + uc), u2);
     }
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      u[e] += u2[e];
+      u[e] += __shfl_xor_sync(0xffffffffu, u[e], 1);
+    }
     const float4 v = ld4(Uv + ur * LN + uc);
-    const float4 res = make_float4(v.x - (u[0] + u2[0]), v.y - (u[1] + u2[1]), v.z - (u[2] + u2[2]), v.w - (u[3] + u2[3]));
-    *reinterpret_cast<float4*>(U_s + ur * LN + uc) = res;
-    *reinterpret_cast<float4*>(a.u + tile * (C * DV) + ur * DV + c0 + uc) = res;
+    const float4 res = make_float4(v.x - u[0], v.y - u[1], v.z - u[2], v.w - u[3]);
+    if (kh2 == 0) store4(U_s + ur * LN + uc, res);
+    else store4(a.u + tile * (C * DV) + ur * DV + c0 + uc, res);
     __syncthreads();
     if (owner) {
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
+      for (int e = 0; e < 2; ++e) {
         const float d = dec[k0 + e];
         S[e][0] *= d;
         S[e][1] *= d;
       }
 #pragma unroll 8
       for (int j = 0; j < C; ++j) {
-        const float4 k = ld4(Kh + j * LD + k0);
+        const float2 k = *reinterpret_cast<const float2*>(Kh + j * LD + k0);
         const float2 x = *reinterpret_cast<const float2*>(U_s + j * LN + s0);
-#pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          S[e][0] = fmaf(lane4(k, e), x.x, S[e][0]);
-          S[e][1] = fmaf(lane4(k, e), x.y, S[e][1]);
-        }
+        S[0][0] = fmaf(k.x, x.x, S[0][0]);
+        S[0][1] = fmaf(k.x, x.y, S[0][1]);
+        S[1][0] = fmaf(k.y, x.x, S[1][0]);
+        S[1][1] = fmaf(k.y, x.y, S[1][1]);
       }
 #pragma unroll
-      for (int e = 0; e < 4; ++e) *reinterpret_cast<float2*>(S_s + (k0 + e) * LN + s0) = make_float2(S[e][0], S[e][1]);
+      for (int e = 0; e < 2; ++e) *reinterpret_cast<float2*>(S_s + (k0 + e) * LN + s0) = make_float2(S[e][0], S[e][1]);
     }
     __syncthreads();   // nobody reads this stage or the old state any more
   }
   if (owner) {
 #pragma unroll
-    for (int e = 0; e < 4; ++e)
+    for (int e = 0; e < 2; ++e)
 #pragma unroll
       for (int f = 0; f < 2; ++f) {
         const int r = k0 + e, col = c0 + s0 + f;
@@ -428,7 +462,7 @@ int launch(const DeltaChunkArgs& a, cudaStream_t s) {
   if (e == cudaSuccess)
     e = cudaFuncSetAttribute(delta_out_kernel<DK, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(m3));
   if (e == cudaSuccess) e = launch_pdl(delta_local_kernel<DK, DV>, dim3(chunks, a.H), dim3(512), m1, s, a);
-  if (e == cudaSuccess) e = launch_pdl(delta_state_kernel<DK, DV>, dim3(DV / NB, a.H), dim3(256), m2, s, a, chunks);
+  if (e == cudaSuccess) e = launch_pdl(delta_state_kernel<DK, DV>, dim3(DV / NB, a.H), dim3(kStateThreads), m2, s, a, chunks);
   if (e == cudaSuccess) e = launch_pdl(delta_out_kernel<DK, DV>, dim3(chunks, a.H, DV / 64), dim3(256), m3, s, a);
   if (e != cudaSuccess) return fail(CTDK_ELAUNCH, "delta chunks: %s", cudaGetErrorString(e));
   check_launch("delta chunks");

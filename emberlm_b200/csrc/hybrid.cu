@@ -623,7 +623,7 @@ int HybridDecoder<T>::run_rows(const int64_t* ids, int64_t n, int64_t pos, int64
     if (L.ff > 0) {
       DTRY(sandwich(vec(L.norm2)));
       DTRY(gemm_rows(h, at<T>(L.w_gu), gu, n, 2 * L.ffp, m.width, m.ldw, m.ldw, 2 * L.ffp, s));
-      DTRY(clamped_glu_rows(gu, act, n, L.ff, L.ffp, L.limit, s));
+      DTRY(clamped_glu_rows(gu, act, n, L.ffp, L.limit, s));
       DTRY(gemm_rows(act, at<T>(L.w_down), y1, n, m.width, L.ff, L.ffp, L.ld_down, m.width, s));
       pending(vec(L.norm2b), nullptr, nullptr, nullptr);
     }

@@ -35,7 +35,7 @@ int norm_rows(const NormArgs<T>& a, int64_t rows, cudaStream_t s);
 
 // act = g sigmoid(1.702 g) (u + 1), g = min(gate, limit), u = clamp(up, +-limit); gu rows hold ffp gate then ffp up columns.
 template <typename T>
-int clamped_glu_rows(const float* gu, T* act, int64_t rows, int ff, int ffp, float limit, cudaStream_t s);
+int clamped_glu_rows(const float* gu, T* act, int64_t rows, int ffp, float limit, cudaStream_t s);
 
 // cos / sin of position * frequency (both in double) for positions [0, n): table[n][pairs].
 int rope_table_f64(float2* table, int64_t n, const double* freqs_dev, int pairs, cudaStream_t s);
@@ -153,12 +153,23 @@ template <typename T>
 int cast_columns(const float* src, int64_t lds, T* dst, int64_t ldd, int64_t rows, int cols, cudaStream_t s);
 
 #ifdef __CUDACC__
-__device__ __forceinline__ float sigmoid_f(float x) { return 1.0f / (1.0f + expf(-x)); }
-__device__ __forceinline__ float silu_f(float x) { return x / (1.0f + expf(-x)); }
+__device__ __forceinline__ float sigmoid_f(float x) { return __fdividef(1.0f, 1.0f + expf(-x)); }
+__device__ __forceinline__ float silu_f(float x) { return x * sigmoid_f(x); }
 __device__ __forceinline__ float softplus_f(float x) { return x > 20.0f ? x : log1pf(expf(x)); }
 __device__ __forceinline__ float clamped_glu_f(float gate, float up, float limit) {
   const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
   return g * sigmoid_f(1.702f * g) * (u + 1.0f);
+}
+__device__ __forceinline__ float4 load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 load4(const __nv_bfloat16* p) {
+  const uint2 u = *reinterpret_cast<const uint2*>(p);
+  return make_float4(__uint_as_float(u.x << 16), __uint_as_float(u.x & 0xffff0000u), __uint_as_float(u.y << 16),
+                     __uint_as_float(u.y & 0xffff0000u));
+}
+__device__ __forceinline__ void store4(float* p, const float4& v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void store4(__nv_bfloat16* p, const float4& v) {
+  const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+  *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
 }
 __device__ __forceinline__ float to_f(float v) { return v; }
 __device__ __forceinline__ float to_f(__nv_bfloat16 v) { return __bfloat162float(v); }

@@ -104,20 +104,17 @@ __global__ void __launch_bounds__(256) norm_rows_kernel(const NormArgs<T> a, int
 
 template <typename T>
 __global__ void __launch_bounds__(256)
-    clamped_glu_kernel(const float* __restrict__ gu, T* __restrict__ act, int64_t n, int ff, int ffp, float limit) {
+    clamped_glu_kernel(const float* __restrict__ gu, T* __restrict__ act, int64_t rows, int ffp, float limit) {
   pdl_launch();
   pdl_wait();
-  const int64_t stride = static_cast<int64_t>(gridDim.x) * 256 * 4;
-  for (int64_t i = (static_cast<int64_t>(blockIdx.x) * 256 + threadIdx.x) * 4; i < n; i += stride) {
-    const int64_t r = i / ffp;
-    const int c = static_cast<int>(i - r * ffp);
-    const float4 g = *reinterpret_cast<const float4*>(gu + r * 2 * ffp + c);
-    const float4 u = *reinterpret_cast<const float4*>(gu + r * 2 * ffp + ffp + c);
-    T* d = act + r * ffp + c;
-    d[0] = from_f<T>(clamped_glu_f(g.x, u.x, limit));
-    d[1] = from_f<T>(clamped_glu_f(g.y, u.y, limit));
-    d[2] = from_f<T>(clamped_glu_f(g.z, u.z, limit));
-    d[3] = from_f<T>(clamped_glu_f(g.w, u.w, limit));
+  for (int64_t r = blockIdx.x; r < rows; r += gridDim.x) {
+    const float* g_row = gu + r * 2 * ffp;
+#pragma unroll 4
+    for (int c = threadIdx.x * 4; c < ffp; c += 1024) {
+      const float4 g = load4(g_row + c), u = load4(g_row + ffp + c);
+      store4(act + r * ffp + c, make_float4(clamped_glu_f(g.x, u.x, limit), clamped_glu_f(g.y, u.y, limit),
+                                            clamped_glu_f(g.z, u.z, limit), clamped_glu_f(g.w, u.w, limit)));
+    }
   }
 }
 
@@ -161,6 +158,50 @@ __global__ void __launch_bounds__(256) attn_pack_kernel(const AttnArgs<T> a, int
       o = make_float2(u * cs.x - v * cs.y, v * cs.x + u * cs.y);
     }
     *reinterpret_cast<float2*>(dst + hh * a.Dp) = o;
+  }
+}
+
+// The same for head sizes that are multiples of four: four columns per thread, a row per CTA turn.
+template <typename T>
+__global__ void __launch_bounds__(256) attn_pack4_kernel(const AttnArgs<T> a, int64_t first, int64_t rows) {
+  pdl_launch();
+  pdl_wait();
+  const int P = a.Dp / 4, heads = a.H + a.G, RS = (a.H + 2 * a.G) * a.Dp, n = heads * P;
+  for (int64_t r = blockIdx.x; r < rows; r += gridDim.x) {
+    const bool fresh = r >= first;
+    const float* row = a.proj + (r - first) * a.ldp;
+    const float2* table = a.table + (r % a.chunk) * a.rot_pairs;
+    float* out = a.packed + r * RS;
+#pragma unroll 2
+    for (int i = threadIdx.x; i < n; i += 256) {
+      const int hh = i / P, d = (i % P) * 4;
+      const bool is_q = hh < a.H;
+      const int head = is_q ? hh : hh - a.H;
+      float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (d < a.dim) {
+        if (fresh) {
+          x = load4(row + (is_q ? a.col_q : a.col_k) + head * a.dim + d);
+          const float4 b = load4((is_q ? a.b_q : a.b_k) + head * a.dim + d);
+          x.x += b.x;
+          x.y += b.y;
+          x.z += b.z;
+          x.w += b.w;
+        } else if (!is_q) {
+          x = load4(a.cache + (static_cast<int64_t>(head) * a.chunk + r) * a.dim + d);
+        }
+      }
+      if (!is_q) store4(out + (a.H + a.G + head) * a.Dp + d, x);
+      const int p = d >> 1;
+      if (p < a.rot_pairs) {
+        const float2 cs = table[p];
+        x = make_float4(x.x * cs.x - x.y * cs.y, x.y * cs.x + x.x * cs.y, x.z, x.w);
+      }
+      if (p + 1 < a.rot_pairs) {
+        const float2 cs = table[p + 1];
+        x = make_float4(x.x, x.y, x.z * cs.x - x.w * cs.y, x.w * cs.x + x.z * cs.y);
+      }
+      store4(out + hh * a.Dp + d, x);
+    }
   }
 }
 
@@ -249,6 +290,24 @@ __global__ void __launch_bounds__(256) attn_gate_kernel(const AttnArgs<T> a, T* 
     const int64_t t = i / cols;
     const int h = c / a.dim, d = c % a.dim;
     dst[t * ld + c] = from_f<T>(a.out[(first + t) * a.H * a.Dp + h * a.Dp + d] * sigmoid_f(a.proj[t * a.ldp + a.col_g + h]));
+  }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256) attn_gate4_kernel(const AttnArgs<T> a, T* dst, int64_t ld, int64_t first, int64_t rows) {
+  pdl_launch();
+  pdl_wait();
+  const int P = a.dim / 4, n = a.H * P;
+  for (int64_t t = blockIdx.x; t < rows - first; t += gridDim.x) {
+    const float* o = a.out + (first + t) * a.H * a.Dp;
+    const float* g = a.proj + t * a.ldp + a.col_g;
+#pragma unroll 2
+    for (int i = threadIdx.x; i < n; i += 256) {
+      const int h = i / P, d = (i % P) * 4;
+      const float4 v = load4(o + h * a.Dp + d);
+      const float s = sigmoid_f(g[h]);
+      store4(dst + t * ld + h * a.dim + d, make_float4(v.x * s, v.y * s, v.z * s, v.w * s));
+    }
   }
 }
 
@@ -380,11 +439,16 @@ __global__ void __launch_bounds__(256) delta_prep4_kernel(const DeltaPrepArgs a)
     if (u >= 2 * a.G + a.H) {   // decays and beta
       const int head = u - 2 * a.G - a.H;
       const float amp = -expf(a.a_log[head]);
-      for (int64_t t = t0; t < t1; ++t)
-        for (int d = lane; d < a.dim; d += 32) {
-          const int c = head * a.dim + d;
-          a.logg[t * a.H * a.dim + c] = amp * softplus_f(a.z[t * a.ldz + c] + a.dt_bias[c]);
-        }
+      for (int d = lane; d < a.dim; d += 32) {
+        const int c = head * a.dim + d;
+        const float bias = a.dt_bias[c];
+        float z[kRun];
+#pragma unroll
+        for (int r = 0; r < kRun; ++r) z[r] = t0 + r < t1 ? a.z[(t0 + r) * a.ldz + c] : 0.0f;
+#pragma unroll
+        for (int r = 0; r < kRun; ++r)
+          if (t0 + r < t1) a.logg[(t0 + r) * a.H * a.dim + c] = amp * softplus_f(z[r] + bias);
+      }
       if (t0 + lane < t1) a.beta[(t0 + lane) * a.H + head] = sigmoid_f(a.proj[(t0 + lane) * a.ldp + a.col_b + head]);
       continue;
     }
@@ -413,12 +477,22 @@ __global__ void __launch_bounds__(256) delta_prep4_kernel(const DeltaPrepArgs a)
         x2[e] = before(t0 - 1, d);
       }
     }
-    for (int64_t t = t0; t < t1; ++t) {
-      float y[E], ss = 0.0f;
+    float rows_x[kRun][E];   // the whole run requested up front
+#pragma unroll
+    for (int r = 0; r < kRun; ++r)
 #pragma unroll
       for (int e = 0; e < E; ++e) {
         const int d = lane + 32 * e;
-        const float x = d < width ? a.proj[t * a.ldp + col + d] : 0.0f;
+        rows_x[r][e] = (d < width && t0 + r < t1) ? a.proj[(t0 + r) * a.ldp + col + d] : 0.0f;
+      }
+#pragma unroll
+    for (int r = 0; r < kRun; ++r) {
+      const int64_t t = t0 + r;
+      if (t >= t1) break;
+      float y[E], ss = 0.0f;
+#pragma unroll
+      for (int e = 0; e < E; ++e) {
+        const float x = rows_x[r][e];
         y[e] = silu_f(fmaf(w[e].w, x, fmaf(w[e].z, x2[e], fmaf(w[e].y, x1[e], w[e].x * x0[e]))));
         ss += y[e] * y[e];
         x0[e] = x1[e];
@@ -484,8 +558,8 @@ int norm_rows(const NormArgs<T>& a, int64_t rows, cudaStream_t s) {
   LAUNCH("hybrid norm", norm_rows_kernel<T>, row_grid(rows), smem, a, rows);
 }
 template <typename T>
-int clamped_glu_rows(const float* gu, T* act, int64_t rows, int ff, int ffp, float limit, cudaStream_t s) {
-  LAUNCH("hybrid glu", clamped_glu_kernel<T>, row_grid(rows * ffp, 1024), 0, gu, act, rows * ffp, ff, ffp, limit);
+int clamped_glu_rows(const float* gu, T* act, int64_t rows, int ffp, float limit, cudaStream_t s) {
+  LAUNCH("hybrid glu", clamped_glu_kernel<T>, row_grid(rows), 0, gu, act, rows, ffp, limit);
 }
 int rope_table_f64(float2* table, int64_t n, const double* freqs_dev, int pairs, cudaStream_t s) {
   rope_table_f64_kernel<<<ceil_div(n * pairs, 256), 256, 0, s>>>(table, n, freqs_dev, pairs);
@@ -493,6 +567,7 @@ int rope_table_f64(float2* table, int64_t n, const double* freqs_dev, int pairs,
 }
 template <typename T>
 int attn_pack(const AttnArgs<T>& a, int64_t first, int64_t rows, cudaStream_t s) {
+  if (a.dim % 4 == 0) LAUNCH("hybrid attention pack", attn_pack4_kernel<T>, row_grid(rows), 0, a, first, rows);
   LAUNCH("hybrid attention pack", attn_pack_kernel<T>, row_grid(rows * (a.H + a.G) * (a.Dp / 2), 256), 0, a, first, rows);
 }
 template <typename T>
@@ -509,6 +584,7 @@ int attn_chunked_fp32(const float* packed, float* out, int64_t first, int64_t ro
 }
 template <typename T>
 int attn_gate(const AttnArgs<T>& a, T* dst, int64_t ld, int64_t first, int64_t rows, cudaStream_t s) {
+  if (a.dim % 4 == 0) LAUNCH("hybrid attention gate", attn_gate4_kernel<T>, row_grid(rows - first), 0, a, dst, ld, first, rows);
   LAUNCH("hybrid attention gate", attn_gate_kernel<T>, row_grid((rows - first) * a.H * a.dim, 256), 0, a, dst, ld, first, rows);
 }
 template <typename T>
@@ -541,7 +617,7 @@ int cast_columns(const float* src, int64_t lds, T* dst, int64_t ldd, int64_t row
 
 #define INSTANTIATE(T)                                                                                                              \
   template int norm_rows<T>(const NormArgs<T>&, int64_t, cudaStream_t);                                                             \
-  template int clamped_glu_rows<T>(const float*, T*, int64_t, int, int, float, cudaStream_t);                                       \
+  template int clamped_glu_rows<T>(const float*, T*, int64_t, int, float, cudaStream_t);                                            \
   template int attn_pack<T>(const AttnArgs<T>&, int64_t, int64_t, cudaStream_t);                                                    \
   template int attn_store<T>(const AttnArgs<T>&, int64_t, int64_t, cudaStream_t);                                                   \
   template int attn_gate<T>(const AttnArgs<T>&, T*, int64_t, int64_t, int64_t, cudaStream_t);                                       \

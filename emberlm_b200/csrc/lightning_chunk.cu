@@ -37,28 +37,45 @@ __global__ void __launch_bounds__(256) lightning_local_kernel(const LightningArg
   if (threadIdx.x <= C) pw[threadIdx.x] = a.powers[h * (C + 1) + threadIdx.x];
   __syncthreads();
   const int64_t tile = static_cast<int64_t>(c) * a.H + h;
-  for (int i = threadIdx.x; i < C * DK; i += 256) {
-    const int j = i / DK, d = i % DK;
-    float q = 0.0f, k = 0.0f;
-    if (j < n && d < a.dim) {
-      q = silu_f(a.q[(t0 + j) * a.ldp + h * a.dim + d]);
-      k = silu_f(a.k[(t0 + j) * a.ldp + h * a.dim + d]);
-    }
-    const __nv_bfloat16 kb = __float2bfloat16(k);
-    ks[j * LK + d] = kb;
-    a.kb[tile * (C * DK) + i] = kb;
-    a.qb[tile * (C * DK) + i] = __float2bfloat16(q);
+  // four columns per thread and turn; head sizes that are not multiples of four load one by one
+  const bool vec_k = a.dim % 4 == 0, vec_v = a.vdim % 4 == 0;
+  auto fetch = [&](const float* base, int j, int d, int width, bool vec) {
+    float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (j >= n || d >= width) return x;
+    const float* p = base + (t0 + j) * a.ldp + h * width + d;
+    if (vec) return load4(p);
+    x.x = p[0];
+    if (d + 1 < width) x.y = p[1];
+    if (d + 2 < width) x.z = p[2];
+    if (d + 3 < width) x.w = p[3];
+    return x;
+  };
+  auto act = [](const float4& x) { return make_float4(silu_f(x.x), silu_f(x.y), silu_f(x.z), silu_f(x.w)); };
+  constexpr int QT = C * DK / 1024, VT = C * DV / 1024;   // turns
+#pragma unroll 4
+  for (int u = 0; u < QT; ++u) {
+    const int i = (threadIdx.x + u * 256) * 4, j = i / DK, d = i % DK;
+    const float4 q = act(fetch(a.q, j, d, a.dim, vec_k)), k = act(fetch(a.k, j, d, a.dim, vec_k));
+    store4(ks + j * LK + d, k);
+    store4(a.kb + tile * (C * DK) + i, k);
+    store4(a.qb + tile * (C * DK) + i, q);
   }
-  for (int i = threadIdx.x; i < C * DV; i += 256) {
-    const int j = i / DV, d = i % DV;
-    float v = 0.0f;
-    if (j < n && d < a.vdim) v = silu_f(a.v[(t0 + j) * a.ldp + h * a.vdim + d]);
-    const __nv_bfloat16 vb = __float2bfloat16(v);
-    a.vb[tile * (C * DV) + i] = vb;
-    const float s = j < n ? __bfloat162float(vb) * pw[n - 1 - j] : 0.0f;
-    const __nv_bfloat16 hi = __float2bfloat16(s);
-    vh[j * LV + d] = hi;
-    vl[j * LV + d] = __float2bfloat16(s - __bfloat162float(hi));
+#pragma unroll 4
+  for (int u = 0; u < VT; ++u) {
+    const int i = (threadIdx.x + u * 256) * 4, j = i / DV, d = i % DV;
+    const float4 v = act(fetch(a.v, j, d, a.vdim, vec_v));
+    __nv_bfloat16* dst = a.vb + tile * (C * DV) + i;
+    store4(dst, v);
+    const float w = j < n ? pw[n - 1 - j] : 0.0f;
+    float s[4] = {v.x, v.y, v.z, v.w}, hi[4], lo[4];
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      s[e] = __bfloat162float(__float2bfloat16(s[e])) * w;   // the stored value, decayed
+      hi[e] = __bfloat162float(__float2bfloat16(s[e]));
+      lo[e] = s[e] - hi[e];
+    }
+    store4(vh + j * LV + d, make_float4(hi[0], hi[1], hi[2], hi[3]));
+    store4(vl + j * LV + d, make_float4(lo[0], lo[1], lo[2], lo[3]));
   }
   __syncthreads();
   constexpr int MG = DK / 32, NG = 8 / MG, COLS = DV / NG, NT = COLS / 8;
