@@ -1,5 +1,4 @@
-// Delta rule with one decay per key channel over long portions, parallel over chunks of 64 tokens; fp32
-// arithmetic throughout. Inside a chunk let b_i be the running sum of the log decays (per channel,
+// Delta rule with one decay per key channel over long portions, parallel over chunks of 64 tokens. Inside a chunk let b_i be the running sum of the log decays (per channel,
 // inclusive) and S the state in front of it. Unrolling
 //   S <- diag(g) S;  u_i = beta_i (v_i - S^T k_i);  S <- S + k_i u_i^T;  o_i = S^T q_i
 // gives, with A_ij = sum_c k_ic k_jc e^(b_ic - b_jc) (j < i) and B_ij the same with q_i (j <= i),
@@ -12,6 +11,13 @@
 // Exponents are differences b_i - b_j with j <= i only, never positive: between 16-row blocks both
 // factors are taken relative to the running sum in front of the later block, inside a block the
 // difference is formed per pair. Strong decays underflow to zero and nothing overflows.
+//
+// delta_local is fp32 arithmetic throughout. The other two exist twice: in fp32, and (split, for
+// bfloat16 models) on the tensor cores with every factor - W, K e^.., Q e^.., U, B and the fp32 state -
+// split into a bfloat16 sum of two terms, x y = xh yh + xh yl + xl yh: 16 mantissa bits of each factor,
+// fp32 sums, the state itself kept in fp32. Shared memory feeds an fp32 tile product at half the FMA
+// rate at best (a 128-bit load per warp occupies it for four cycles, whatever it broadcasts), which made
+// the serial state kernel five times slower than the split form.
 #include "hybrid_kernels.h"
 #include "mma_bf16.cuh"
 
@@ -60,6 +66,21 @@ __device__ __forceinline__ void tile_product(const float* M, int ldm, const floa
   }
 }
 
+// Two bfloat16 planes [2][rows][cols] in the bytes of an fp32 tile.
+__device__ __forceinline__ void store_split(float* tile, int plane, int i, const float4& v) {
+  __nv_bfloat16* p = reinterpret_cast<__nv_bfloat16*>(tile);
+  uint32_t h0, l0, h1, l1;
+  split_bf16x2(v.x, v.y, h0, l0);
+  split_bf16x2(v.z, v.w, h1, l1);
+  *reinterpret_cast<uint2*>(p + i) = make_uint2(h0, h1);
+  *reinterpret_cast<uint2*>(p + plane + i) = make_uint2(l0, l1);
+}
+template <bool SPLIT>
+__device__ __forceinline__ void put4(float* tile, int plane, int i, const float4& v) {
+  if (SPLIT) store_split(tile, plane, i, v);
+  else store4(tile + i, v);
+}
+
 template <int DK, int DV>
 struct LocalCfg {
   static constexpr int LD = DK + 4, LV = DV + 4;
@@ -68,7 +89,7 @@ struct LocalCfg {
 };
 
 // grid (chunks, heads), 512 threads.
-template <int DK, int DV>
+template <int DK, int DV, bool SPLIT>
 __global__ void __launch_bounds__(512, 1) delta_local_kernel(const DeltaChunkArgs a) {
   using Cfg = LocalCfg<DK, DV>;
   constexpr int LD = Cfg::LD, LV = Cfg::LV;
@@ -252,9 +273,9 @@ __global__ void __launch_bounds__(512, 1) delta_local_kernel(const DeltaChunkArg
     const int i = (tid + u * 512) * 4, r = i / DK, d = i % DK;
     const float4 b = ld4(b_s + r * LD + d), k = ld4(k_s + r * LD + d), q = ld4(q_s + r * LD + d), z = ld4(b_s + (C - 1) * LD + d);
     const float4 e = make_float4(ex2(b.x), ex2(b.y), ex2(b.z), ex2(b.w));
-    store4(a.kh + tile * (C * DK) + i,
-           make_float4(k.x * ex2(z.x - b.x), k.y * ex2(z.y - b.y), k.z * ex2(z.z - b.z), k.w * ex2(z.w - b.w)));
-    store4(a.qt + tile * (C * DK) + i, make_float4(q.x * e.x, q.y * e.y, q.z * e.z, q.w * e.w));
+    put4<SPLIT>(a.kh + tile * (C * DK), C * DK, i,
+                make_float4(k.x * ex2(z.x - b.x), k.y * ex2(z.y - b.y), k.z * ex2(z.z - b.z), k.w * ex2(z.w - b.w)));
+    put4<SPLIT>(a.qt + tile * (C * DK), C * DK, i, make_float4(q.x * e.x, q.y * e.y, q.z * e.z, q.w * e.w));
     store4(k_s + r * LD + d, make_float4(k.x * e.x, k.y * e.y, k.z * e.z, k.w * e.w));
     if (r == C - 1) store4(a.decay + tile * DK + d, e);
   }
@@ -271,7 +292,7 @@ __global__ void __launch_bounds__(512, 1) delta_local_kernel(const DeltaChunkArg
     tile_product(X_s, LT, k_s, LD, r0, c0, r0 + 4, acc);
 #pragma unroll
     for (int r = 0; r < 4; ++r)
-      *reinterpret_cast<float4*>(a.w + tile * (C * DK) + (r0 + r) * DK + c0) = make_float4(acc[r][0], acc[r][1], acc[r][2], acc[r][3]);
+      put4<SPLIT>(a.w + tile * (C * DK), C * DK, (r0 + r) * DK + c0, make_float4(acc[r][0], acc[r][1], acc[r][2], acc[r][3]));
   }
   for (int it = tid; it < 16 * (DV / 4); it += 512) {
     const int r0 = it / (DV / 4) * 4, c0 = it % (DV / 4) * 4;
@@ -451,17 +472,277 @@ __global__ void __launch_bounds__(256) delta_out_kernel(const DeltaChunkArgs a) 
       if (r0 + r < n && n0 + c0 + e < a.vdim) a.out[(t0 + r0 + r) * a.H * a.vdim + h * a.vdim + n0 + c0 + e] = acc[r][e];
 }
 
+// ---- split form ----
+constexpr int LNB = NB + 8;   // bfloat16 pitch of the 16-column tiles
+
+template <int DK>
+struct SplitStateCfg {
+  static constexpr int LK = DK + 8;
+  static constexpr int kStage = 4 * C * LK * 2 + C * LN * 4 + DK * 4;   // W high / low, K high / low, T V, decay (bytes)
+  static constexpr int kBytes = 2 * kStage + 2 * DK * LNB * 2 + 2 * C * LNB * 2;
+};
+
+// grid (DV / 16, heads), 256 threads. A warp owns one (16-row, 8-column) tile of U and 16 rows of the
+// state, which stays in its accumulators.
+template <int DK, int DV>
+__global__ void __launch_bounds__(256, 1) delta_state_split_kernel(const DeltaChunkArgs a, int chunks) {
+  using Cfg = SplitStateCfg<DK>;
+  constexpr int LK = Cfg::LK;
+  extern __shared__ __align__(16) unsigned char raw[];
+  __nv_bfloat16* Sh = reinterpret_cast<__nv_bfloat16*>(raw + 2 * Cfg::kStage);   // [DK][LNB]
+  __nv_bfloat16* Sl = Sh + DK * LNB;
+  __nv_bfloat16* Uh = Sl + DK * LNB;   // [C][LNB]
+  __nv_bfloat16* Ul = Uh + C * LNB;
+  pdl_launch();
+  pdl_wait();
+  const int h = blockIdx.y, c0 = blockIdx.x * NB, tid = threadIdx.x, lane = tid & 31, wid = tid >> 5;
+  auto load = [&](int c) {
+    unsigned char* st = raw + (c & 1) * Cfg::kStage;
+    __nv_bfloat16* ops = reinterpret_cast<__nv_bfloat16*>(st);   // four planes [C][LK]
+    const int64_t tile = static_cast<int64_t>(c) * a.H + h;
+    const __nv_bfloat16* w = reinterpret_cast<const __nv_bfloat16*>(a.w + tile * (C * DK));
+    const __nv_bfloat16* kh = reinterpret_cast<const __nv_bfloat16*>(a.kh + tile * (C * DK));
+#pragma unroll
+    for (int i = tid; i < 2 * C * (DK / 8); i += 256) {   // both planes are contiguous rows
+      const int r = i / (DK / 8), p = i % (DK / 8) * 8;
+      cp_async16(ops + r * LK + p, w + r * DK + p);
+      cp_async16(ops + (2 * C + r) * LK + p, kh + r * DK + p);
+    }
+    float* us = reinterpret_cast<float*>(st + 4 * C * LK * 2);
+    const int r = tid >> 2, p = (tid & 3) * 4;
+    cp_async16(us + r * LN + p, a.u + tile * (C * DV) + r * DV + c0 + p);
+    if (tid < DK / 4) cp_async16(us + C * LN + tid * 4, a.decay + tile * DK + tid * 4);
+    cp_async_commit();
+  };
+  // accumulator element e of column tile t: row wid * 16 + lane / 4 + (e / 2) * 8, column t * 8 + (lane % 4) * 2 + e % 2
+  const int sr = wid * 16 + (lane >> 2), sc = (lane & 3) * 2;
+  const bool owner = wid * 16 < DK;
+  float S[2][4];
+#pragma unroll
+  for (int t = 0; t < 2; ++t)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int r = sr + (e >> 1) * 8, col = c0 + t * 8 + sc + (e & 1);
+      S[t][e] = (a.resume && owner && r < a.dim && col < a.vdim) ? a.state[(static_cast<int64_t>(h) * a.dim + r) * a.vdim + col] : 0.0f;
+    }
+  load(0);
+  for (int c = 0; c < chunks; ++c) {
+    const int64_t tile = static_cast<int64_t>(c) * a.H + h;
+    if (owner) {   // the state in front of the chunk: for this chunk's products, and for the output kernel
+      __nv_bfloat16* g = reinterpret_cast<__nv_bfloat16*>(a.chunk_state + tile * (DK * DV));
+#pragma unroll
+      for (int t = 0; t < 2; ++t)
+#pragma unroll
+        for (int f = 0; f < 2; ++f) {
+          const int r = sr + f * 8, col = t * 8 + sc;
+          uint32_t hi, lo;
+          split_bf16x2(S[t][2 * f], S[t][2 * f + 1], hi, lo);
+          *reinterpret_cast<uint32_t*>(Sh + r * LNB + col) = hi;
+          *reinterpret_cast<uint32_t*>(Sl + r * LNB + col) = lo;
+          *reinterpret_cast<uint32_t*>(g + r * (2 * DV) + c0 + col) = hi;
+          *reinterpret_cast<uint32_t*>(g + r * (2 * DV) + DV + c0 + col) = lo;
+        }
+    }
+    if (c + 1 < chunks) {
+      load(c + 1);
+      cp_async_wait<1>();
+    } else {
+      cp_async_wait<0>();
+    }
+    __syncthreads();   // operands and state have landed
+    const unsigned char* st = raw + (c & 1) * Cfg::kStage;
+    const __nv_bfloat16* Wh = reinterpret_cast<const __nv_bfloat16*>(st);
+    const __nv_bfloat16* Wl = Wh + C * LK;
+    const __nv_bfloat16* Kh = Wl + C * LK;
+    const __nv_bfloat16* Kl = Kh + C * LK;
+    const float* Uv = reinterpret_cast<const float*>(st + 4 * C * LK * 2);
+    const float* dec = Uv + C * LN;
+    {
+      const int m0 = (wid & 3) * 16, nt = wid >> 2;
+      float p[3][4] = {};
+#pragma unroll
+      for (int k0 = 0; k0 < DK; k0 += 16) {
+        uint32_t ah[4], al[4], bh[4], bl[4];
+        ldsm_a(ah, Wh, LK, m0, k0, lane);
+        ldsm_a(al, Wl, LK, m0, k0, lane);
+        ldsm_b_trans(bh, Sh, LNB, k0, 0, lane);
+        ldsm_b_trans(bl, Sl, LNB, k0, 0, lane);
+        const uint32_t h0 = nt ? bh[2] : bh[0], h1 = nt ? bh[3] : bh[1], l0 = nt ? bl[2] : bl[0], l1 = nt ? bl[3] : bl[1];
+        mma_bf16(p[0], ah, h0, h1);
+        mma_bf16(p[1], ah, l0, l1);
+        mma_bf16(p[2], al, h0, h1);
+      }
+      __nv_bfloat16* gu = reinterpret_cast<__nv_bfloat16*>(a.us + tile * (C * DV));
+#pragma unroll
+      for (int f = 0; f < 2; ++f) {
+        const int r = m0 + (lane >> 2) + f * 8, col = nt * 8 + sc;
+        const float2 v = *reinterpret_cast<const float2*>(Uv + r * LN + col);
+        const float x = v.x - (p[0][2 * f] + (p[1][2 * f] + p[2][2 * f])), y = v.y - (p[0][2 * f + 1] + (p[1][2 * f + 1] + p[2][2 * f + 1]));
+        uint32_t hi, lo;
+        split_bf16x2(x, y, hi, lo);
+        *reinterpret_cast<uint32_t*>(Uh + r * LNB + col) = hi;
+        *reinterpret_cast<uint32_t*>(Ul + r * LNB + col) = lo;
+        *reinterpret_cast<uint32_t*>(gu + r * DV + c0 + col) = hi;
+        *reinterpret_cast<uint32_t*>(gu + C * DV + r * DV + c0 + col) = lo;
+      }
+    }
+    __syncthreads();
+    if (owner) {
+      float q[2][2][4] = {};   // the cross terms, summed apart from the state
+#pragma unroll
+      for (int t = 0; t < 2; ++t)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) S[t][e] *= dec[sr + (e >> 1) * 8];
+#pragma unroll
+      for (int k0 = 0; k0 < C; k0 += 16) {
+        uint32_t ah[4], al[4], bh[4], bl[4];
+        ldsm_a_trans(ah, Kh, LK, wid * 16, k0, lane);
+        ldsm_a_trans(al, Kl, LK, wid * 16, k0, lane);
+        ldsm_b_trans(bh, Uh, LNB, k0, 0, lane);
+        ldsm_b_trans(bl, Ul, LNB, k0, 0, lane);
+#pragma unroll
+        for (int t = 0; t < 2; ++t) {
+          mma_bf16(S[t], ah, bh[2 * t], bh[2 * t + 1]);
+          mma_bf16(q[0][t], ah, bl[2 * t], bl[2 * t + 1]);
+          mma_bf16(q[1][t], al, bh[2 * t], bh[2 * t + 1]);
+        }
+      }
+#pragma unroll
+      for (int t = 0; t < 2; ++t)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) S[t][e] += q[0][t][e] + q[1][t][e];
+    }
+    __syncthreads();   // nobody reads this stage, the old state or U any more
+  }
+  if (owner) {
+#pragma unroll
+    for (int t = 0; t < 2; ++t)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int r = sr + (e >> 1) * 8, col = c0 + t * 8 + sc + (e & 1);
+        if (r < a.dim && col < a.vdim) a.state[(static_cast<int64_t>(h) * a.dim + r) * a.vdim + col] = S[t][e];
+      }
+  }
+}
+
+template <int DK>
+struct SplitOutCfg {
+  static constexpr int LK = DK + 8, LB = 64 + 8;
+  static constexpr int kBytes = (2 * C * LK + 2 * DK * LB + 2 * C * LB) * 2;
+};
+
+// grid (chunks, heads, DV / 64), 128 threads: a warp owns 16 rows and 64 columns.
+template <int DK, int DV>
+__global__ void __launch_bounds__(128) delta_out_split_kernel(const DeltaChunkArgs a) {
+  using Cfg = SplitOutCfg<DK>;
+  constexpr int LK = Cfg::LK, LB = Cfg::LB;
+  extern __shared__ __align__(16) unsigned char raw[];
+  __nv_bfloat16* Q = reinterpret_cast<__nv_bfloat16*>(raw);   // [2][C][LK]
+  __nv_bfloat16* S = Q + 2 * C * LK;                          // [2][DK][LB]
+  __nv_bfloat16* U = S + 2 * DK * LB;                         // [2][C][LB]
+  pdl_launch();
+  pdl_wait();
+  const int c = blockIdx.x, h = blockIdx.y, n0 = blockIdx.z * 64, tid = threadIdx.x, lane = tid & 31, wid = tid >> 5;
+  const int64_t t0 = static_cast<int64_t>(c) * C, tile = static_cast<int64_t>(c) * a.H + h;
+  auto copy = [&](__nv_bfloat16* dst, int ld, const __nv_bfloat16* src, int lds, int rows, int cols) {
+    const int per = cols / 8;
+    for (int i = tid; i < rows * per; i += 128) cp_async16(dst + i / per * ld + i % per * 8, src + static_cast<int64_t>(i / per) * lds + i % per * 8);
+  };
+  const __nv_bfloat16* gs = reinterpret_cast<const __nv_bfloat16*>(a.chunk_state + tile * (DK * DV));
+  copy(Q, LK, reinterpret_cast<const __nv_bfloat16*>(a.qt + tile * (C * DK)), DK, 2 * C, DK);
+  copy(S, LB, gs + n0, 2 * DV, DK, 64);
+  copy(S + DK * LB, LB, gs + DV + n0, 2 * DV, DK, 64);
+  copy(U, LB, reinterpret_cast<const __nv_bfloat16*>(a.us + tile * (C * DV)) + n0, DV, 2 * C, 64);
+  cp_async_commit();
+  const int m0 = wid * 16, r0 = m0 + (lane >> 2);
+  const float* B = a.scores + tile * (C * C);
+  float2 sc[C / 16][4];   // scores of the warp's rows, in the order of an A fragment
+#pragma unroll
+  for (int kk = 0; kk < C / 16; ++kk)
+#pragma unroll
+    for (int e = 0; e < 4; ++e)
+      sc[kk][e] = kk * 16 < m0 + 16 ? *reinterpret_cast<const float2*>(B + (r0 + (e & 1) * 8) * C + kk * 16 + (e >> 1) * 8 + (lane & 3) * 2)
+                                    : make_float2(0.0f, 0.0f);
+  cp_async_wait_all();
+  __syncthreads();
+  float o[8][4] = {};
+#pragma unroll 2
+  for (int k0 = 0; k0 < DK; k0 += 16) {
+    uint32_t ah[4], al[4], bh[4], bl[4];
+    ldsm_a(ah, Q, LK, m0, k0, lane);
+    ldsm_a(al, Q + C * LK, LK, m0, k0, lane);
+#pragma unroll
+    for (int t = 0; t < 8; t += 2) {
+      ldsm_b_trans(bh, S, LB, k0, t * 8, lane);
+      ldsm_b_trans(bl, S + DK * LB, LB, k0, t * 8, lane);
+#pragma unroll
+      for (int f = 0; f < 2; ++f) {
+        mma_bf16(o[t + f], ah, bh[2 * f], bh[2 * f + 1]);
+        mma_bf16(o[t + f], ah, bl[2 * f], bl[2 * f + 1]);
+        mma_bf16(o[t + f], al, bh[2 * f], bh[2 * f + 1]);
+      }
+    }
+  }
+#pragma unroll
+  for (int kk = 0; kk < C / 16; ++kk) {
+    if (kk * 16 >= m0 + 16) break;
+    uint32_t ah[4], al[4], bh[4], bl[4];
+#pragma unroll
+    for (int e = 0; e < 4; ++e) split_bf16x2(sc[kk][e].x, sc[kk][e].y, ah[e], al[e]);
+#pragma unroll
+    for (int t = 0; t < 8; t += 2) {
+      ldsm_b_trans(bh, U, LB, kk * 16, t * 8, lane);
+      ldsm_b_trans(bl, U + C * LB, LB, kk * 16, t * 8, lane);
+#pragma unroll
+      for (int f = 0; f < 2; ++f) {
+        mma_bf16(o[t + f], ah, bh[2 * f], bh[2 * f + 1]);
+        mma_bf16(o[t + f], ah, bl[2 * f], bl[2 * f + 1]);
+        mma_bf16(o[t + f], al, bh[2 * f], bh[2 * f + 1]);
+      }
+    }
+  }
+  const int n = static_cast<int>(a.rows - t0 < C ? a.rows - t0 : C);
+  const int64_t ldo = static_cast<int64_t>(a.H) * a.vdim;
+  float* out = a.out + t0 * ldo + h * a.vdim;
+#pragma unroll
+  for (int t = 0; t < 8; ++t)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int i = r0 + (e >> 1) * 8, col = n0 + t * 8 + (lane & 3) * 2 + (e & 1);
+      if (i < n && col < a.vdim) out[i * ldo + col] = o[t][e];
+    }
+}
+
+template <int DK, int DV>
+int launch_split(const DeltaChunkArgs& a, cudaStream_t s) {
+  const int chunks = static_cast<int>((a.rows + C - 1) / C);
+  constexpr size_t m1 = LocalCfg<DK, DV>::kFloats * 4, m2 = SplitStateCfg<DK>::kBytes, m3 = SplitOutCfg<DK>::kBytes;
+  static_assert(m1 <= 227 * 1024 && m2 <= 227 * 1024, "shared memory");
+  cudaError_t e = cudaFuncSetAttribute(delta_local_kernel<DK, DV, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(m1));
+  if (e == cudaSuccess)
+    e = cudaFuncSetAttribute(delta_state_split_kernel<DK, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(m2));
+  if (e == cudaSuccess)
+    e = cudaFuncSetAttribute(delta_out_split_kernel<DK, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(m3));
+  if (e == cudaSuccess) e = launch_pdl(delta_local_kernel<DK, DV, true>, dim3(chunks, a.H), dim3(512), m1, s, a);
+  if (e == cudaSuccess) e = launch_pdl(delta_state_split_kernel<DK, DV>, dim3(DV / NB, a.H), dim3(256), m2, s, a, chunks);
+  if (e == cudaSuccess) e = launch_pdl(delta_out_split_kernel<DK, DV>, dim3(chunks, a.H, DV / 64), dim3(128), m3, s, a);
+  if (e != cudaSuccess) return fail(CTDK_ELAUNCH, "delta chunks: %s", cudaGetErrorString(e));
+  check_launch("delta chunks");
+  check_launch("delta chunks");
+  return check_launch("delta chunks");
+}
+
 template <int DK, int DV>
 int launch(const DeltaChunkArgs& a, cudaStream_t s) {
   const int chunks = static_cast<int>((a.rows + C - 1) / C);
   constexpr size_t m1 = LocalCfg<DK, DV>::kFloats * 4, m2 = StateCfg<DK>::kFloats * 4, m3 = OutCfg<DK>::kFloats * 4;
   static_assert(m1 <= 227 * 1024 && m2 <= 227 * 1024, "shared memory");
-  cudaError_t e = cudaFuncSetAttribute(delta_local_kernel<DK, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(m1));
+  cudaError_t e = cudaFuncSetAttribute(delta_local_kernel<DK, DV, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(m1));
   if (e == cudaSuccess)
     e = cudaFuncSetAttribute(delta_state_kernel<DK, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(m2));
   if (e == cudaSuccess)
     e = cudaFuncSetAttribute(delta_out_kernel<DK, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(m3));
-  if (e == cudaSuccess) e = launch_pdl(delta_local_kernel<DK, DV>, dim3(chunks, a.H), dim3(512), m1, s, a);
+  if (e == cudaSuccess) e = launch_pdl(delta_local_kernel<DK, DV, false>, dim3(chunks, a.H), dim3(512), m1, s, a);
   if (e == cudaSuccess) e = launch_pdl(delta_state_kernel<DK, DV>, dim3(DV / NB, a.H), dim3(kStateThreads), m2, s, a, chunks);
   if (e == cudaSuccess) e = launch_pdl(delta_out_kernel<DK, DV>, dim3(chunks, a.H, DV / 64), dim3(256), m3, s, a);
   if (e != cudaSuccess) return fail(CTDK_ELAUNCH, "delta chunks: %s", cudaGetErrorString(e));
@@ -477,6 +758,10 @@ bool delta_chunked_ok(int dim, int vdim) { return dim <= 128 && vdim <= 128; }
 int delta_chunked(const DeltaChunkArgs& a, cudaStream_t s) {
   CTDK_REQUIRE(delta_chunked_ok(a.dim, a.vdim) && a.H <= 65535, "delta chunks: head sizes above 128");
   const int dk = lightning_tile(a.dim), dv = lightning_tile(a.vdim);
+  if (a.split) {
+    if (dk == 64) return dv == 64 ? launch_split<64, 64>(a, s) : launch_split<64, 128>(a, s);
+    return dv == 64 ? launch_split<128, 64>(a, s) : launch_split<128, 128>(a, s);
+  }
   if (dk == 64) return dv == 64 ? launch<64, 64>(a, s) : launch<64, 128>(a, s);
   return dv == 64 ? launch<128, 64>(a, s) : launch<128, 128>(a, s);
 }

@@ -66,7 +66,7 @@ struct HybridDecoder : DecoderBase {
   // prompt-pass buffers, rows = max_portion
   float *x, *proj, *packed, *attn_out, *o32, *y1, *y2, *gu, *dq, *dk, *dv, *dlog, *dbeta, *dz, *dgate;
   T *h, *mixed, *mixed2, *act, *low_a, *low_g;
-  float *chunk_state, *cw, *ckh, *cqt, *cu, *cscores, *cdecay;
+  float *chunk_state, *cw, *ckh, *cqt, *cu, *cus, *cscores, *cdecay;
   __nv_bfloat16 *qb, *kb, *vb;
   int32_t* want_dev;
   // token-pass buffers
@@ -200,6 +200,7 @@ int HybridDecoder<T>::carve(Bump& b) {
   ckh = b.floats(ck_n);
   cqt = b.floats(ck_n);
   cu = b.floats(cv_n);
+  cus = b.floats(cv_n);
   cscores = b.floats(cs_n);
   cdecay = b.floats(cd_n);
   qb = static_cast<__nv_bfloat16*>(b.bytes(qk_tiles * 2));
@@ -544,6 +545,8 @@ int HybridDecoder<T>::mixer_delta(const Branch& b, const BranchBuffers& bb, int6
     a.kh = ckh;
     a.qt = cqt;
     a.u = cu;
+    a.us = cus;
+    a.split = m.dtype == CTDK_DTYPE_BF16 ? 1 : 0;
     a.scores = cscores;
     a.decay = cdecay;
     a.chunk_state = chunk_state;

@@ -106,15 +106,16 @@ struct LightningArgs {
 };
 // Chunk-parallel delta rule: inputs as for recurrent_scan (q, k [rows][G * dim], v [rows][H * vdim], logg
 // [rows][H * dim], beta [rows][H], dense). Scratch per (chunk, head), dk / dv the tile sizes: w, kh, qt
-// [64][dk], u [64][dv], scores [64][64], decay [dk], chunk_state [dk][dv].
+// [64][dk], u and us [64][dv], scores [64][64], decay [dk], chunk_state [dk][dv]. split: the products after
+// the per-chunk kernel run on the tensor cores with factors of two bfloat16 terms (delta_chunk.cu).
 constexpr int kDeltaChunk = 64;
 struct DeltaChunkArgs {
   const float *q = nullptr, *k = nullptr, *v = nullptr, *logg = nullptr, *beta = nullptr;
   float *state = nullptr, *out = nullptr;
-  float *w = nullptr, *kh = nullptr, *qt = nullptr, *u = nullptr, *scores = nullptr, *decay = nullptr, *chunk_state = nullptr;
+  float *w = nullptr, *kh = nullptr, *qt = nullptr, *u = nullptr, *us = nullptr, *scores = nullptr, *decay = nullptr, *chunk_state = nullptr;
   int H = 0, G = 0, dim = 0, vdim = 0;
   int64_t rows = 0;
-  int resume = 0;
+  int resume = 0, split = 0;
 };
 bool delta_chunked_ok(int dim, int vdim);
 int delta_chunked(const DeltaChunkArgs& a, cudaStream_t s);
