@@ -178,8 +178,10 @@ def test_far_memory_of_the_recurrences_is_carried(dtype):
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("a_log,dt", [(4.0, 3.0), (-9.0, -4.0), (1.5, 0.0)])
 def test_delta_rule_with_strong_and_weak_decays(a_log, dt, dtype):
-    """Decays that wipe a channel within a token (e^-160) or hardly move it: nothing overflows."""
-    cfg = hc.model(40, 48, [hc.delta(2, 1, 64, 40, 4), hc.delta(1, 1, 20, 20, 3)])
+    """Decays that wipe a channel within a token (e^-160) or hardly move it: nothing overflows. A wiped state
+    leaves o = (q . k) u, which the norm over the head divides by |q . k|: the large eps keeps tokens whose
+    q and k happen to be orthogonal from magnifying their own rounding."""
+    cfg = hc.model(40, 48, [hc.delta(2, 1, 64, 40, 4), hc.delta(1, 1, 20, 20, 3)], eps=1e-2)
     w = hc.weights(cfg, 81)
     for i in (0, 1):
         w[f"l{i}.mix.A_log"] = hc.bf16(w[f"l{i}.mix.A_log"] + a_log)
