@@ -499,6 +499,27 @@ def run_decode(args) -> dict:
             "last_tokens": toks[-4:].tolist()}
 
 
+def run_serving(args) -> dict:
+    """Prefill and greedy decode, batch 1, of the layer-list design Zutalix in bfloat16 beside the preset
+    decoder closest to it at equal width, depth, feed-forward width and vocabulary (random weights). A
+    "step" is one prompt of 4096 tokens plus 128 greedy tokens; value = prompt tokens/s of the larger
+    Zutalix; `models` holds every figure."""
+    from emberlm_b200 import serve_bench
+    import torch
+    torch.cuda.set_device(0)
+    rows = []
+    for size in sorted(serve_bench.SIZES):
+        rows += serve_bench.run(size, steps=args.steps, warmup=max(args.warmup, 3), sampler=lambda: ClockSampler(0))
+    main_row = next(r for r in reversed(rows) if r["model"].startswith("zutalix"))
+    return {"metric": "prefill tokens/s (batch 1, 4096-token prompt)", "value": main_row["prefill_tokens_per_s"], "unit": "tokens/s",
+            "n_gpus": 1, "steps": args.steps, "warmup": max(args.warmup, 3),
+            "ms_per_step": main_row["prefill_ms"] + main_row["token_ms"] * main_row["new_tokens"], "higher_is_better": True,
+            "scaling": "replicas only", "vs_baseline": None, "dtype": "bf16", "data": "synthetic", "impl": "ours",
+            "config": {"workload": "zutalix_serving", "model": main_row["model"], "prompt_len": main_row["prompt_len"],
+                       "new_tokens": main_row["new_tokens"], "l2": "weights larger than L2"},
+            "clocks": main_row["clocks"], "gpu_launches": main_row["gpu_launches"], "models": rows}
+
+
 def run_decode_reference(args) -> dict:
     """The reference's own generator (tools/ctd_generate/main.cpp:104-184, built unmodified as
     oracle/_ref/ref_ctd_generate) on the same workload: same random weights written as a safetensors
@@ -572,7 +593,7 @@ def main():
     ap.add_argument("--steps", type=int, default=10)
     ap.add_argument("--warmup", type=int, default=3)
     ap.add_argument("--impl", choices=["ours", "reference"], default="ours")
-    ap.add_argument("--workload", choices=sorted(WORKLOADS) + ["qwen3_0_6b_decode"], default=DEFAULT_WORKLOAD)
+    ap.add_argument("--workload", choices=sorted(WORKLOADS) + ["qwen3_0_6b_decode", "zutalix_serving"], default=DEFAULT_WORKLOAD)
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--precision", choices=["tf32", "3xtf32"], default="tf32",
                     help="3xtf32: every contraction splits its operands into TF32 high and low parts (near-fp32 results)")
@@ -582,7 +603,9 @@ def main():
     args = ap.parse_args()
     if args.warmup < 3 and args.impl == "ours":
         print(f"note: --warmup {args.warmup} < 3; timing rules ask for at least 3", file=sys.stderr)
-    if args.workload == "qwen3_0_6b_decode":
+    if args.workload == "zutalix_serving":
+        out = run_serving(args) if args.impl == "ours" else {"impl": "reference", "unavailable": "the reference has no such model"}
+    elif args.workload == "qwen3_0_6b_decode":
         out = run_decode(args) if args.impl == "ours" else run_decode_reference(args)
     else:
         out = run_reference(args) if args.impl == "reference" else run_ours(args)

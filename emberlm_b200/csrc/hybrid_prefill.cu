@@ -424,9 +424,9 @@ __global__ void __launch_bounds__(256) delta_prep_kernel(const DeltaPrepArgs a) 
 
 // The same for four taps with a sliding window: one warp per (unit, run of kRun rows), so that a
 // projection row is read once. E = ceil(max(dim, vdim) / 32) channels per lane.
-constexpr int kRun = 8;
+constexpr int kRun = 8, kAhead = 4;
 template <int E>
-__global__ void __launch_bounds__(256) delta_prep4_kernel(const DeltaPrepArgs a) {
+__global__ void __launch_bounds__(256, 3) delta_prep4_kernel(const DeltaPrepArgs a) {
   pdl_launch();
   pdl_wait();
   const int lane = threadIdx.x & 31;
@@ -477,35 +477,38 @@ __global__ void __launch_bounds__(256) delta_prep4_kernel(const DeltaPrepArgs a)
         x2[e] = before(t0 - 1, d);
       }
     }
-    float rows_x[kRun][E];   // the whole run requested up front
+#pragma unroll 1
+    for (int64_t tb = t0; tb < t1; tb += kAhead) {
+      float rows_x[kAhead][E];   // requested together
 #pragma unroll
-    for (int r = 0; r < kRun; ++r)
+      for (int r = 0; r < kAhead; ++r)
 #pragma unroll
-      for (int e = 0; e < E; ++e) {
-        const int d = lane + 32 * e;
-        rows_x[r][e] = (d < width && t0 + r < t1) ? a.proj[(t0 + r) * a.ldp + col + d] : 0.0f;
-      }
+        for (int e = 0; e < E; ++e) {
+          const int d = lane + 32 * e;
+          rows_x[r][e] = (d < width && tb + r < t1) ? a.proj[(tb + r) * a.ldp + col + d] : 0.0f;
+        }
 #pragma unroll
-    for (int r = 0; r < kRun; ++r) {
-      const int64_t t = t0 + r;
-      if (t >= t1) break;
-      float y[E], ss = 0.0f;
+      for (int r = 0; r < kAhead; ++r) {
+        const int64_t t = tb + r;
+        if (t >= t1) break;
+        float y[E], ss = 0.0f;
 #pragma unroll
-      for (int e = 0; e < E; ++e) {
-        const float x = rows_x[r][e];
-        y[e] = silu_f(fmaf(w[e].w, x, fmaf(w[e].z, x2[e], fmaf(w[e].y, x1[e], w[e].x * x0[e]))));
-        ss += y[e] * y[e];
-        x0[e] = x1[e];
-        x1[e] = x2[e];
-        x2[e] = x;
-      }
-      float sc = 1.0f;
-      if (kind < 2) sc = rsqrtf(warp_sum(ss) + 1e-6f) * (kind == 0 ? qscale : 1.0f);
-      float* dst = kind == 2 ? a.v + t * a.H * a.vdim + head * width : (kind == 0 ? a.q : a.k) + t * qk + head * width;
+        for (int e = 0; e < E; ++e) {
+          const float x = rows_x[r][e];
+          y[e] = silu_f(fmaf(w[e].w, x, fmaf(w[e].z, x2[e], fmaf(w[e].y, x1[e], w[e].x * x0[e]))));
+          ss += y[e] * y[e];
+          x0[e] = x1[e];
+          x1[e] = x2[e];
+          x2[e] = x;
+        }
+        float sc = 1.0f;
+        if (kind < 2) sc = rsqrtf(warp_sum(ss) + 1e-6f) * (kind == 0 ? qscale : 1.0f);
+        float* dst = kind == 2 ? a.v + t * a.H * a.vdim + head * width : (kind == 0 ? a.q : a.k) + t * qk + head * width;
 #pragma unroll
-      for (int e = 0; e < E; ++e) {
-        const int d = lane + 32 * e;
-        if (d < width) dst[d] = y[e] * sc;
+        for (int e = 0; e < E; ++e) {
+          const int d = lane + 32 * e;
+          if (d < width) dst[d] = y[e] * sc;
+        }
       }
     }
   }

@@ -22,7 +22,7 @@ constexpr int kPad = 8;   // bfloat16 columns behind every shared-memory row: co
 
 // grid (chunks, heads), 256 threads.
 template <int DK, int DV>
-__global__ void __launch_bounds__(256) lightning_local_kernel(const LightningArgs a) {
+__global__ void __launch_bounds__(256, 3) lightning_local_kernel(const LightningArgs a) {
   constexpr int LK = DK + kPad, LV = DV + kPad;
   extern __shared__ __align__(16) unsigned char smem[];
   __nv_bfloat16* ks = reinterpret_cast<__nv_bfloat16*>(smem);   // [C][LK]

@@ -89,16 +89,22 @@ def build_preset(size: str, layers: int | None, max_seq: int):
     return dec, sum(dec.layout.numels)
 
 
-def measure(dec, vocab: int, prompt_len: int, new_tokens: int, steps: int, warmup: int) -> dict:
-    """Milliseconds per prefill of prompt_len tokens and per greedy token after it."""
+def measure(dec, vocab: int, prompt_len: int, new_tokens: int, steps: int, warmup: int, sampler=None) -> dict:
+    """Milliseconds per prefill of prompt_len tokens and per greedy token after it. sampler: makes an object
+    with start() / stop() that watches the clocks of the timed steps."""
     L, s = E._L, dec.stream
     gen = torch.Generator(device="cuda").manual_seed(7)
     ids = torch.randint(0, vocab, (prompt_len,), generator=gen, device="cuda")
     out = torch.zeros(new_tokens + 1, dtype=torch.int64, device="cuda")
     torch.cuda.synchronize()
     pre = dcd = 0.0
+    watch, launches = sampler() if sampler else None, 0
     with torch.cuda.stream(s):
         for i in range(warmup + steps):
+            if i == warmup:
+                launches = L.ctdk_launch_count()
+                if watch:
+                    watch.start()
             e = [torch.cuda.Event(enable_timing=True) for _ in range(3)]
             e[0].record(s)
             lib.check(L.ctdk_decode_prefill(dec._h, ids.data_ptr(), prompt_len, s.cuda_stream))
@@ -109,17 +115,19 @@ def measure(dec, vocab: int, prompt_len: int, new_tokens: int, steps: int, warmu
             if i >= warmup:
                 pre += e[0].elapsed_time(e[1])
                 dcd += e[1].elapsed_time(e[2])
-    return {"prefill_ms": pre / steps, "prefill_tokens_per_s": prompt_len * steps / pre * 1e3, "token_ms": dcd / steps / new_tokens,
+    launches = L.ctdk_launch_count() - launches
+    extra = {"clocks": watch.stop()} if watch else {}
+    return {**extra, "gpu_launches": launches, "prefill_ms": pre / steps, "prefill_tokens_per_s": prompt_len * steps / pre * 1e3, "token_ms": dcd / steps / new_tokens,
             "decode_tokens_per_s": new_tokens * steps / dcd * 1e3}
 
 
 def run(size: str, layers: int | None = None, prompt_len: int = 4096, new_tokens: int = 128, steps: int = 5, warmup: int = 3,
-        models=("zutalix", "preset")) -> list[dict]:
+        models=("zutalix", "preset"), sampler=None) -> list[dict]:
     rows = []
     for which in models:
         max_seq = prompt_len + new_tokens + 64
         dec, params = (build_zutalix(size, layers, max_seq, prompt_len) if which == "zutalix" else build_preset(size, layers, max_seq))
-        r = measure(dec, dec.vocab, prompt_len, new_tokens, steps, warmup)
+        r = measure(dec, dec.vocab, prompt_len, new_tokens, steps, warmup, sampler)
         bytes_per = 2 if which == "zutalix" else 4
         rows.append({"model": f"zutalix-{size}" if which == "zutalix" else SIZES[size][0],
                      "dtype": "bf16" if which == "zutalix" else "tf32 prefill, fp32 decode", "params": params, "prompt_len": prompt_len,
