@@ -79,3 +79,23 @@ def test_decode_limits_and_errors():
         dec.generate([], 4)
     with pytest.raises(RuntimeError):
         dec.generate(np.arange(24), 1)                        # prompt must leave room for one token
+
+
+@pytest.mark.parametrize("kw", CASES)
+def test_portions_of_given_tokens(kw):
+    """extend(): a prompt cut anywhere gives the logits of the whole prompt, also after a reset."""
+    from emberlm_b200 import engine as E
+    ocfg, ecfg, params = build(kw, 47)
+    t = np.random.default_rng(8).integers(0, ocfg.vocab_size, size=30)
+    want = om.forward_logits(params, ocfg, t[None, :], acc=np.float64)[0]
+    dec = E.Decoder(ecfg, max_seq_len=32)
+    dec.load_parameters(params)
+    for sizes in ([30], [17, 13], [1, 1, 28], [29, 1]):
+        dec.reset()
+        got, at = [], 0
+        for n in sizes:
+            got.append(dec.extend(t[at:at + n], range(n)).cpu().numpy())
+            at += n
+        assert np.abs(np.concatenate(got) - want).max() <= 5e-3 * max(np.abs(want).max(), 1.0), sizes
+    assert np.abs(dec.step(int(t[0])).cpu().numpy() - om.forward_logits(
+        params, ocfg, np.append(t, t[0])[None, :], acc=np.float64)[0, -1]).max() <= 5e-3 * max(np.abs(want).max(), 1.0)
