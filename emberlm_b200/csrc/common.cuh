@@ -41,6 +41,10 @@ void prof_end(void* token, cudaStream_t s);
 int encode_tensor_map(CUtensorMap* map, const float* base, int rank, const uint64_t* dims,
                       const uint64_t* strides_bytes, const uint32_t* box, bool atom32);
 
+// The same for bfloat16 data, 128-byte swizzle in 16-byte chunks.
+int encode_tensor_map_bf16(CUtensorMap* map, const void* base, int rank, const uint64_t* dims, const uint64_t* strides_bytes,
+                           const uint32_t* box);
+
 inline int ceil_div(int64_t a, int64_t b) { return static_cast<int>((a + b - 1) / b); }
 
 #define CTDK_REQUIRE(cond, ...)                                   \

@@ -52,6 +52,10 @@ struct GemmArgs {
   int vec_ok;  // C (and aux) rows are 16-byte aligned and N%4==0
   int splits;  // K is cut into `splits` ranges; >1: partial tiles are added to C with atomics
   int* status;
+  // Grouped product (bfloat16 form): m-block i multiplies with the n_pitch rows of B that belong to group
+  // tiles[i], and only the first tiles[max_tiles] m-blocks exist. Null: one group.
+  const int32_t* tiles = nullptr;
+  int max_tiles = 0, n_pitch = 0;
 };
 
 // Instruction descriptor: D=F32 (bit 4), A,B format at bits 7 and 10 (kind::tf32: 2 = TF32;
@@ -94,7 +98,8 @@ __global__ void __launch_bounds__(kThreads, 1)
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(final_bar + 1);
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int m_blocks = (args.M + BM - 1) / BM;
+  const bool grouped = BF16 && args.tiles != nullptr;
+  const int m_blocks = grouped ? args.tiles[args.max_tiles] : (args.M + BM - 1) / BM;
   const int n_blocks = (args.N + BN - 1) / BN;
   const int num_tiles = m_blocks * n_blocks;
   const int k_blocks = (args.K + kElems - 1) / kElems;
@@ -133,6 +138,7 @@ __global__ void __launch_bounds__(kThreads, 1)
         int mb, nb;
         tile_coords(unit % num_tiles, m_blocks, n_blocks, mb, nb);
         const int m0 = mb * BM, n0 = nb * BN;
+        const int b_row = grouped ? n0 + args.tiles[mb] * args.n_pitch : n0;
         const int split = unit / num_tiles;
         const int kb0 = static_cast<int>(static_cast<int64_t>(split) * k_blocks / args.splits);
         const int kb1 = static_cast<int>(static_cast<int64_t>(split + 1) * k_blocks / args.splits);
@@ -157,7 +163,7 @@ __global__ void __launch_bounds__(kThreads, 1)
             for (int c = 0; c < BN / 32; ++c)
               tma_load_2d(b_dst + c * kChunkBytes, &tmB, &full[s], n0 + 32 * c, k0);
           } else {
-            tma_load_2d(b_dst, &tmB, &full[s], k0, n0);
+            tma_load_2d(b_dst, &tmB, &full[s], k0, b_row);
           }
           if (++s == C::kStages) {
             s = 0;
@@ -422,7 +428,7 @@ int launch(const CUtensorMap& ta, const CUtensorMap& tb, const GemmArgs& args,
                   C::kSmemBytes, cudaGetErrorString(e));
     attr_set[dev] = true;
   }
-  const int m_blocks = (args.M + BM - 1) / BM, n_blocks = (args.N + BN - 1) / BN;
+  const int m_blocks = args.tiles != nullptr ? args.max_tiles : (args.M + BM - 1) / BM, n_blocks = (args.N + BN - 1) / BN;
   const int tiles = m_blocks * n_blocks * args.splits;
   const int sms = sm_count();
   const int grid = tiles < sms ? tiles : sms;
@@ -703,6 +709,25 @@ int gemm_tcgen05(const float* A, const float* B, float* Cp, int64_t M, int64_t N
   }
 }
 
+int encode_tensor_map_bf16(CUtensorMap* map, const void* base, int rank, const uint64_t* dims, const uint64_t* strides_bytes,
+                           const uint32_t* box) {
+  auto enc = encode_fn();
+  if (enc == nullptr) return fail(CTDK_ELAUNCH, "cuTensorMapEncodeTiled unavailable");
+  cuuint64_t d[5], st[4];
+  cuuint32_t bx[5], es[5];
+  for (int i = 0; i < rank; ++i) {
+    d[i] = dims[i];
+    bx[i] = box[i];
+    es[i] = 1u;
+    if (i + 1 < rank) st[i] = strides_bytes[i];
+  }
+  const CUresult r = enc(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, static_cast<cuuint32_t>(rank), const_cast<void*>(base), d, st, bx, es,
+                         CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+                         CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  if (r != CUDA_SUCCESS) return fail(CTDK_ELAUNCH, "cuTensorMapEncodeTiled failed (%d) for a bfloat16 operand", static_cast<int>(r));
+  return CTDK_OK;
+}
+
 int gemm_tcgen05_2cta_bf16(const CUtensorMap& ta, const CUtensorMap& tb, const CUtensorMap& tc, int tma_out, float* C,
                            int64_t ldc, int M, int N, int K, int vec_ok, int splits, int* status, cudaStream_t stream);
 
@@ -718,17 +743,9 @@ int gemm_bf16_tcgen05(const void* A, const void* B, float* Cp, int64_t M, int64_
   bool use_pair;
   choose_tile(M, N, k_blocks, &bn, &splits, &use_pair);
   auto map_bf16 = [](CUtensorMap* map, const void* base, int64_t inner, int64_t outer, int64_t ld, int box_rows) {
-    auto enc = encode_fn();
-    if (enc == nullptr) return fail(CTDK_ELAUNCH, "cuTensorMapEncodeTiled unavailable");
-    cuuint64_t dims[2] = {static_cast<cuuint64_t>(inner), static_cast<cuuint64_t>(outer)};
-    cuuint64_t strides[1] = {static_cast<cuuint64_t>(ld) * 2};
-    cuuint32_t box[2] = {static_cast<cuuint32_t>(BKH), static_cast<cuuint32_t>(box_rows)};
-    cuuint32_t estr[2] = {1u, 1u};
-    const CUresult r = enc(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(base), dims, strides, box, estr,
-                           CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
-                           CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
-    if (r != CUDA_SUCCESS) return fail(CTDK_ELAUNCH, "cuTensorMapEncodeTiled failed (%d) for a bfloat16 operand", static_cast<int>(r));
-    return CTDK_OK;
+    const uint64_t dims[2] = {static_cast<uint64_t>(inner), static_cast<uint64_t>(outer)}, strides[1] = {static_cast<uint64_t>(ld) * 2};
+    const uint32_t box[2] = {static_cast<uint32_t>(BKH), static_cast<uint32_t>(box_rows)};
+    return encode_tensor_map_bf16(map, base, 2, dims, strides, box);
   };
   CUtensorMap ta, tb;
   int rc = map_bf16(&ta, A, K, M, lda, BM);
@@ -754,6 +771,36 @@ int gemm_bf16_tcgen05(const void* A, const void* B, float* Cp, int64_t M, int64_
                                   splits, st, stream);
   }
   const GemmArgs args{Cp, nullptr, ldc, static_cast<int>(M), static_cast<int>(N), static_cast<int>(K), CTDK_EPI_STORE, vec, splits, st};
+  switch (bn) {
+    case 64: return launch<64, false, false, true>(ta, tb, args, stream);
+    case 128: return launch<128, false, false, true>(ta, tb, args, stream);
+    default: return launch<256, false, false, true>(ta, tb, args, stream);
+  }
+}
+
+// Grouped form: C[m-block i of 128 rows] = A[m-block i] B[tiles[i]]^T for the first tiles[max_tiles] m-blocks;
+// group g's N rows of B start at row g * n_pitch. tiles lies in device memory.
+int gemm_bf16_grouped(const void* A, int64_t lda, const void* B, int64_t ldb, int64_t n_pitch, float* Cp, int64_t ldc, int N, int K, int groups,
+                      const int32_t* tiles, int max_tiles, cudaStream_t stream) {
+  auto a16 = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15u) == 0; };
+  CTDK_REQUIRE(a16(A) && a16(B) && (lda & 7) == 0 && (ldb & 7) == 0, "gemm_bf16_grouped: operands must be 16-byte aligned");
+  CTDK_REQUIRE(N >= 8 && K >= 1 && groups >= 1 && max_tiles >= 1 && n_pitch * groups <= INT32_MAX && n_pitch >= N, "gemm_bf16_grouped: bad shape");
+  const int bn = N >= 256 ? 256 : (N > 64 ? 128 : 64);
+  const int64_t M = static_cast<int64_t>(max_tiles) * BM;
+  CTDK_REQUIRE(M <= INT32_MAX, "gemm_bf16_grouped: too many rows");
+  const uint64_t da[2] = {static_cast<uint64_t>(K), static_cast<uint64_t>(M)}, sa[1] = {static_cast<uint64_t>(lda) * 2};
+  const uint64_t db[2] = {static_cast<uint64_t>(K), static_cast<uint64_t>(n_pitch * groups)}, sb[1] = {static_cast<uint64_t>(ldb) * 2};
+  const uint32_t box_a[2] = {static_cast<uint32_t>(BKH), static_cast<uint32_t>(BM)}, box_b[2] = {static_cast<uint32_t>(BKH), static_cast<uint32_t>(bn)};
+  CUtensorMap ta, tb;
+  int rc = encode_tensor_map_bf16(&ta, A, 2, da, sa, box_a);
+  if (rc == CTDK_OK) rc = encode_tensor_map_bf16(&tb, B, 2, db, sb, box_b);
+  if (rc != CTDK_OK) return rc;
+  int* st = device_status_word();
+  if (st == nullptr) return fail(CTDK_ELAUNCH, "gemm: no status word");
+  GemmArgs args{Cp, nullptr, ldc, static_cast<int>(M), N, K, CTDK_EPI_STORE, (a16(Cp) && (ldc & 3) == 0) ? 1 : 0, 1, st};
+  args.tiles = tiles;
+  args.max_tiles = max_tiles;
+  args.n_pitch = static_cast<int>(n_pitch);
   switch (bn) {
     case 64: return launch<64, false, false, true>(ta, tb, args, stream);
     case 128: return launch<128, false, false, true>(ta, tb, args, stream);

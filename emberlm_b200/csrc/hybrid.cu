@@ -11,98 +11,14 @@
 #include <new>
 #include <vector>
 
-#include "decode_core.h"
-#include "hybrid_kernels.h"
-#include "hybrid_model.h"
-#include "hybrid_token.h"
+#include "hybrid_decoder.h"
 
 namespace ctdk {
 namespace hybrid {
-namespace {
-
-int gemm_rows(const __nv_bfloat16* A, const __nv_bfloat16* W, float* C, int64_t M, int64_t N, int64_t K, int64_t lda, int64_t ldw,
-              int64_t ldc, cudaStream_t s) {
-  return ctdk_gemm_bf16(A, W, C, M, N, K, lda, ldw, ldc, s);
-}
-int gemm_rows(const float* A, const float* W, float* C, int64_t M, int64_t N, int64_t K, int64_t lda, int64_t ldw, int64_t ldc,
-              cudaStream_t s) {
-  return ctdk_gemm(A, W, C, M, N, K, lda, ldw, ldc, 0, 1, CTDK_GEMM_FP32_SIMT, CTDK_EPI_STORE, nullptr, s);
-}
-
-// Device buffers of one branch.
-struct BranchBuffers {
-  void* cache = nullptr;        // attention
-  int64_t chunk = 0;            // cache rows: the chunk, or max_seq when that is smaller
-  int rope = -1;                // index of the rotation table
-  float* decay = nullptr;       // lightning: per head; then its powers 0 .. 64 per head
-  float* powers = nullptr;
-  float* state = nullptr;
-  float* ring = nullptr;
-};
-
-struct RopeTable {
-  RopeSpec spec;
-  int64_t rows = 0;
-  float2* table = nullptr;
-  double* freqs = nullptr;
-};
-
-constexpr int64_t kChunkedRows = 16;   // shorter portions run the recurrences token by token
-
-int padded_head(int dim, bool tensor_cores) {
-  if (!tensor_cores) return (dim + 3) / 4 * 4;
-  return dim <= 64 ? 64 : 128;
-}
-
-template <typename T>
-struct HybridDecoder : DecoderBase {
-  Model m;
-  const char* params = nullptr;
-  int64_t max_portion = 0;
-  std::vector<std::vector<BranchBuffers>> bufs;
-  std::vector<RopeTable> ropes;
-  float* layers_out = nullptr;
-
-  // prompt-pass buffers, rows = max_portion
-  float *x, *proj, *packed, *attn_out, *o32, *y1, *y2, *gu, *dq, *dk, *dv, *dlog, *dbeta, *dz, *dgate;
-  T *h, *mixed, *mixed2, *act, *low_a, *low_g;
-  float *chunk_state, *cw, *ckh, *cqt, *cu, *cus, *cscores, *cdecay;
-  __nv_bfloat16 *qb, *kb, *vb;
-  int32_t* want_dev;
-  // token-pass buffers
-  float *tx[2], *tproj, *tout[2], *tgate, *ty1, *ty2, *tgu, *tpart;
-  unsigned int* sync;
-  int64_t sync_words = 0;
-  TokenPhase* phases_dev;
-  std::vector<TokenPhase> phases;
-  int stage_floats = 0, token_ctas = 0;
-  size_t token_smem = 0;
-
-  template <typename U>
-  const U* at(int64_t off) const { return reinterpret_cast<const U*>(params + off); }
-  const float* vec(int64_t off) const { return at<float>(off); }
-  bool tensor_core_attention(const Branch& b) const { return m.dtype == CTDK_DTYPE_BF16 && b.dim <= 128; }
-
-  bool chunked_lightning(const Branch& b) const { return m.dtype == CTDK_DTYPE_BF16 && lightning_chunked_ok(b.dim, b.vdim); }
-
-  int carve(Bump& b);
-  int build_phases();
-  int upload(cudaStream_t s);
-  int run_rows(const int64_t* ids, int64_t n, int64_t pos, int64_t done, const int32_t* want, int64_t n_want, float* want_logits,
-               bool last, cudaStream_t s);
-  int mixer_attention(const Branch& b, const BranchBuffers& bb, int64_t n, int64_t pos, float* y, int64_t ldp, cudaStream_t s);
-  int mixer_lightning(const Branch& b, const BranchBuffers& bb, int64_t n, int64_t pos, float* y, int64_t ldp, cudaStream_t s);
-  int mixer_delta(const Branch& b, const BranchBuffers& bb, int64_t n, int64_t pos, float* y, int64_t ldp, cudaStream_t s);
-
-  int portion(const int64_t* ids, int64_t n, int64_t pos, const int32_t* want, int64_t n_want, float* want_logits,
-              cudaStream_t s) override;
-  int token_forward(cudaStream_t s) override;
-  int burst(int64_t n, int64_t* out_tokens, cudaStream_t s) override;
-  TokenArgs token_args() const;
-};
 
 template <typename T>
 int HybridDecoder<T>::carve(Bump& b) {
+  if (m.arrangement == Arrangement::kParallel) return carve_parallel(b);
   const int64_t R = max_portion, W = m.width;
   int64_t n_in = 8, mix = 8, heads_out = 8, packed_n = 0, attn_n = 0, ff = 8, parts = 0, arrives = 0;
   int64_t ck_n = 0, cv_n = 0, cs_n = 0, cd_n = 0;
@@ -230,6 +146,7 @@ int HybridDecoder<T>::carve(Bump& b) {
 // The phases of one token (see hybrid_token.cu).
 template <typename T>
 int HybridDecoder<T>::build_phases() {
+  if (m.arrangement == Arrangement::kParallel) return build_parallel_phases();
   phases.clear();
   stage_floats = static_cast<int>(m.ldw);
   int cur = 0;                       // which of tx[] holds the residual
@@ -366,23 +283,31 @@ int HybridDecoder<T>::build_phases() {
   hd.gemv[0] = TokenGemv{at<T>(m.head), logits, vocab, static_cast<int>(m.ldw), 0};
   phases.push_back(hd);
 
+  return finish_phases();
+}
+
+// Prefetch order, shared memory, warps per row.
+template <typename T>
+int HybridDecoder<T>::finish_phases() {
   // every phase asks for the weights of one coming product, the mix phases run the queue one ahead
   const int n = static_cast<int>(phases.size());
   int next = 1;
   for (int i = 0; i < n; ++i) {
     next = std::max(next, i + 1);
-    while (next < n && phases[next].is_mix) ++next;
+    while (next < n && (phases[next].is_mix || (phases[next].n_gemv == 0 && phases[next].extra == nullptr))) ++next;
     if (next < n && next - i <= 3) phases[i].prefetch = next++;
   }
   token_smem = token_smem_bytes(stage_floats, phases.data(), n);
   CTDK_REQUIRE(token_smem <= 200 * 1024, "hybrid decoder: the token pass needs %zu bytes of shared memory", token_smem);
-  int rc = token_grid<T>(token_smem, &token_ctas);
+  int rc = token_grid<T>(token_smem, m.arrangement == Arrangement::kParallel, &token_ctas);
   if (rc != CTDK_OK) return rc;
   for (TokenPhase& p : phases) {
     if (p.is_mix) continue;
-    const int rows = p.gemv[0].rows + (p.n_gemv > 1 ? p.gemv[1].rows : 0);
-    int K = p.gemv[0].K;
-    if (p.n_gemv > 1) K = std::max(K, p.gemv[1].K);
+    int rows = 0, K = 0;
+    for (int i = 0; i < p.n_gemv; ++i) {
+      rows += p.gemv[i].rows;
+      K = std::max(K, p.gemv[i].K);
+    }
     int wpr = 1;
     while (wpr < 8 && static_cast<int64_t>(rows) * wpr * 2 <= static_cast<int64_t>(token_ctas) * 8 &&
            K * static_cast<int>(sizeof(T)) / 16 >= 64 * wpr)
@@ -488,7 +413,7 @@ int HybridDecoder<T>::mixer_lightning(const Branch& b, const BranchBuffers& bb, 
     a.vdim = b.vdim;
     a.rows = n;
     a.resume = pos > 0;
-    DTRY(recurrent_scan(a, false, s));
+    DTRY(recurrent_scan(a, Recurrence::kLightning, s));
   }
   const int cols = b.heads * b.vdim;
   DTRY(gated_norm_rows(o32, vec(b.w_norm), proj + b.col_g, ldp, mixed, b.ld_o, n, cols, m.eps, s));
@@ -574,7 +499,7 @@ int HybridDecoder<T>::mixer_delta(const Branch& b, const BranchBuffers& bb, int6
     a.vdim = b.vdim;
     a.rows = n;
     a.resume = pos > 0;
-    DTRY(recurrent_scan(a, true, s));
+    DTRY(recurrent_scan(a, Recurrence::kDelta, s));
   }
   DTRY(gated_head_norm_rows(o32, vec(b.w_norm), dgate, ldg, mixed, b.ld_o, n, b.heads, b.vdim, m.eps, s));
   return gemm_rows(mixed, at<T>(b.w_o), y, n, m.width, static_cast<int64_t>(b.heads) * b.vdim, b.ld_o, b.ld_o, m.width, s);
@@ -584,6 +509,7 @@ int HybridDecoder<T>::mixer_delta(const Branch& b, const BranchBuffers& bb, int6
 template <typename T>
 int HybridDecoder<T>::run_rows(const int64_t* ids, int64_t n, int64_t pos, int64_t done, const int32_t* want, int64_t n_want,
                                float* want_logits, bool last, cudaStream_t s) {
+  if (m.arrangement == Arrangement::kParallel) return run_parallel_rows(ids, n, pos, done, want, n_want, want_logits, last, s);
   NormArgs<T> na;   // the pending norm: what the next norm_rows adds to the residual
   na.width = m.width;
   na.eps = m.eps;
@@ -638,7 +564,20 @@ int HybridDecoder<T>::run_rows(const int64_t* ids, int64_t n, int64_t pos, int64
     ra.w_pre = vec(m.final_norm);
     DTRY(norm_rows(ra, n, s));
   }
-  // head: wanted rows only
+  return run_head(n, done, want, n_want, want_logits, last, [&](const int32_t* gather, int64_t k) {
+    NormArgs<T> fa = na;
+    fa.x = x;
+    fa.gather = gather;
+    fa.x_out = nullptr;
+    fa.w_pre = vec(m.final_norm);
+    return norm_rows(fa, k, s);
+  }, s);
+}
+
+// The head for the wanted rows among n (see run_rows): `norm` forms h of the gathered rows.
+template <typename T>
+int HybridDecoder<T>::run_head(int64_t n, int64_t done, const int32_t* want, int64_t n_want, float* want_logits, bool last,
+                               const std::function<int(const int32_t*, int64_t)>& norm, cudaStream_t s) {
   std::vector<int32_t> rows;
   std::vector<int64_t> dst;
   if (n_want < 0) {
@@ -659,12 +598,7 @@ int HybridDecoder<T>::run_rows(const int64_t* ids, int64_t n, int64_t pos, int64
     const int64_t k = static_cast<int64_t>(i1 - i0);
     if (cudaMemcpyAsync(want_dev, rows.data() + i0, k * 4, cudaMemcpyHostToDevice, s) != cudaSuccess)
       return fail(CTDK_ELAUNCH, "hybrid decoder: copying the wanted rows failed");
-    NormArgs<T> fa = na;
-    fa.x = x;
-    fa.gather = want_dev;
-    fa.x_out = nullptr;
-    fa.w_pre = vec(m.final_norm);
-    DTRY(norm_rows(fa, k, s));
+    DTRY(norm(want_dev, k));
     DTRY(gemm_rows(h, at<T>(m.head), dst[i0] < 0 ? logits : want_logits + dst[i0] * vocab, k, vocab, m.width, m.ldw, m.ldw, vocab, s));
     i0 = i1;
   }
@@ -691,7 +625,8 @@ TokenArgs HybridDecoder<T>::token_args() const {
   a.eps = m.eps;
   a.embed = at<T>(m.embed);
   a.ld_embed = m.ldw;
-  a.w_embed = vec(m.embed_norm);
+  a.w_embed = m.arrangement == Arrangement::kSandwich ? vec(m.embed_norm) : nullptr;
+  a.embed_scale = m.embed_scale;
   a.vocab = vocab;
   a.cur_token = cur_token;
   a.counters = counters;
@@ -706,7 +641,7 @@ template <typename T>
 int HybridDecoder<T>::token_forward(cudaStream_t s) {
   const TokenArgs a = token_args();
   CTDK_REQUIRE(a.status != nullptr, "hybrid decoder: no status word");
-  return launch_token_kernel<T>(a, token_ctas, token_smem, s);
+  return launch_token_kernel<T>(a, m.arrangement == Arrangement::kParallel, token_ctas, token_smem, s);
 }
 
 template <typename T>
@@ -716,8 +651,10 @@ int HybridDecoder<T>::burst(int64_t n, int64_t* out_tokens, cudaStream_t s) {
   a.out_tokens = out_tokens;
   a.out_offset = static_cast<int>(generated);
   a.n_tokens = static_cast<int>(n);
-  return launch_token_kernel<T>(a, token_ctas, token_smem, s);
+  return launch_token_kernel<T>(a, m.arrangement == Arrangement::kParallel, token_ctas, token_smem, s);
 }
+
+namespace {
 
 int check_sizes(const Model* m, int64_t max_seq, int64_t max_portion) {
   CTDK_REQUIRE(m != nullptr && max_seq > 0 && max_seq < (1 << 24) && max_portion > 0, "hybrid decoder: bad arguments");

@@ -74,13 +74,17 @@ int attn_gate(const AttnArgs<T>& a, T* dst, int64_t ld, int64_t first, int64_t r
 // ---- recurrences ----
 // State S[H][dim][vdim] (fp32). q / k / v / g are [rows] x heads with the given row pitches; head h reads
 // q, k of group h / (H / G). silu != 0: q, k, v pass silu on load. resume == 0: the stored state is
-// ignored (a new sequence). Delta: logg [rows][H * dim] log decays, beta [rows][H]; otherwise decay[H].
+// ignored (a new sequence). Lightning: decay[H]. Delta: logg [rows][H * dim] log decays, beta [rows][H].
+// Wkv: decays e^(-e^(z + w0)) from z [rows][ldz] and w0 [H * dim], bonus [H * dim].
+enum class Recurrence { kLightning, kDelta, kWkv };
 struct ScanArgs {
   const float *q = nullptr, *k = nullptr, *v = nullptr;
   int64_t ldq = 0, ldk = 0, ldv = 0;
   const float* logg = nullptr;
   const float* beta = nullptr;
   const float* decay = nullptr;
+  const float *z = nullptr, *w0 = nullptr, *bonus = nullptr;
+  int64_t ldz = 0;
   int silu = 0;
   float* state = nullptr;
   float* out = nullptr;   // [rows][H * vdim]
@@ -88,7 +92,7 @@ struct ScanArgs {
   int64_t rows = 0;
   int resume = 0;
 };
-int recurrent_scan(const ScanArgs& a, bool delta, cudaStream_t s);
+int recurrent_scan(const ScanArgs& a, Recurrence kind, cudaStream_t s);
 
 // Chunk-parallel lightning attention (bfloat16 models): q, k, v are columns of the projection (before
 // silu), powers[h][i] = decay_h^i for i in [0, 64]. Scratch: chunk_state [chunks][H][dk][dv] floats,

@@ -114,6 +114,13 @@ RopeSpec parse_rope(const Value& v, int dim) {
   return r;
 }
 
+// null and a missing key mean the same
+bool given(const Value& v, const char* key) { return v.contains(key) && v.at(key).kind != Value::kNull; }
+
+int count_or_zero(const Value& v, const char* key) {
+  return given(v, key) && v.at(key).number() != 0.0 ? positive(v, key) : 0;
+}
+
 void check_groups(const Branch& b) {
   if (b.heads % b.kv_heads != 0) bad("heads must be a multiple of kv_heads");
 }
@@ -160,6 +167,43 @@ Branch parse_channel_delta(const Value& v) {
   return b;
 }
 
+// Keys and values read out of one latent per position; the rotated part is rotate-half over rot_dim.
+Branch parse_latent(const Value& v) {
+  Branch b;
+  b.kind = BranchKind::kLatent;
+  b.heads = b.kv_heads = positive(v, "heads");
+  b.dim = positive(v, "dim");
+  b.vdim = positive(v, "vdim");
+  b.rot_dim = positive(v, "rot_dim");
+  b.kv_rank = positive(v, "kv_rank");
+  b.q_rank = positive(v, "q_rank");
+  b.scale = static_cast<float>(v.at("scale").number());
+  b.rope = parse_rope(v.at("rot"), b.rot_dim);
+  if (b.rope.dims != b.rot_dim) bad("latent attention rotates all of rot_dim");
+  if (b.kv_rank > 1024 || b.vdim > 1024 || b.dim + b.rot_dim > 1024) bad("latent attention sizes too large");
+  return b;
+}
+
+Branch parse_wkv(const Value& v) {
+  Branch b;
+  b.kind = BranchKind::kWkv;
+  b.heads = b.kv_heads = positive(v, "heads");
+  b.dim = b.vdim = positive(v, "dim");
+  if (b.dim > 256) bad("recurrent key size above 256");
+  return b;
+}
+
+void place_latent(Branch& b, Layout& lay, const std::string& p) {
+  b.col_q = lay.stacked(p + "dq", b.q_rank);
+  b.col_k = lay.stacked(p + "dkv", b.kv_rank + b.rot_dim);
+  b.col_g = lay.stacked(p + "g", b.heads);
+}
+void place_wkv(Branch& b, Layout& lay, const std::string& p) {
+  b.rank_w = static_cast<int>(lay.shape(p + "w1").at(0));
+  const int64_t n = static_cast<int64_t>(b.heads) * b.dim;
+  const char* names[Branch::kMixes] = {"r", "k", "v", "g", "w1"};
+  for (int i = 0; i < Branch::kMixes; ++i) b.col_mix[i] = lay.stacked(p + names[i], i < 4 ? n : b.rank_w);
+}
 void place_attention(Branch& b, Layout& lay, const std::string& p) {
   b.col_q = lay.stacked(p + "q", b.heads * b.dim);
   b.col_k = lay.stacked(p + "k", b.kv_heads * b.dim);
@@ -188,6 +232,24 @@ void place_rest(Branch& b, Layout& lay, const std::string& p, int width) {
     b.b_k = lay.vec(p + "k.b", b.kv_heads * b.dim);
   } else if (b.kind == BranchKind::kLightning) {
     b.w_norm = lay.vec(p + "norm", b.heads * b.vdim);
+  } else if (b.kind == BranchKind::kLatent) {
+    b.q_norm = lay.vec(p + "dq.norm", b.q_rank);
+    b.kv_norm = lay.vec(p + "dkv.norm", b.kv_rank);
+    b.w_uq = lay.matrix(p + "uq", static_cast<int64_t>(b.heads) * (b.dim + b.rot_dim), b.q_rank);
+    b.ld_uq = pad8(b.q_rank);
+    lay.begin_stack(b.kv_rank);
+    lay.stacked(p + "uk", static_cast<int64_t>(b.heads) * b.dim);
+    b.row_uv = lay.stacked(p + "uv", static_cast<int64_t>(b.heads) * b.vdim);
+    b.n_ukv = lay.end_stack(&b.w_ukv);
+    b.ld_ukv = pad8(b.kv_rank);
+  } else if (b.kind == BranchKind::kWkv) {
+    const char* names[Branch::kMixes] = {"r", "k", "v", "g", "w"};
+    for (int i = 0; i < Branch::kMixes; ++i) b.mu[i] = lay.vec(p + "mu." + names[i], width);
+    b.w_w2 = lay.matrix(p + "w2", static_cast<int64_t>(b.heads) * b.dim, b.rank_w);
+    b.ld_w2 = pad8(b.rank_w);
+    b.w0 = lay.vec(p + "w0", static_cast<int64_t>(b.heads) * b.dim);
+    b.bonus = lay.table(p + "u", b.heads, b.dim);
+    b.w_norm = lay.vec(p + "norm", static_cast<int64_t>(b.heads) * b.dim);
   } else {
     b.conv_q = lay.table(p + "q.conv", b.kv_heads * b.dim, b.taps);
     b.conv_k = lay.table(p + "k.conv", b.kv_heads * b.dim, b.taps);
@@ -206,6 +268,126 @@ void place_rest(Branch& b, Layout& lay, const std::string& p, int width) {
 
 }  // namespace
 
+namespace {
+
+Moe parse_moe(const Value& v) {
+  Moe e;
+  const Value& r = v.at("router");
+  e.experts = positive(r, "experts");
+  e.identity = count_or_zero(r, "identity");
+  e.top = positive(r, "top");
+  if (given(r, "groups")) {
+    e.groups = positive(r.at("groups"), "count");
+    e.keep = positive(r.at("groups"), "keep");
+  }
+  if (e.outputs() % e.groups != 0) bad("router outputs must form equal groups");
+  if (e.keep > e.groups || e.top > e.outputs() / e.groups * e.keep) bad("the router keeps fewer outputs than it chooses");
+  if (e.outputs() > 1024 || e.top > 32) bad("more than 1024 router outputs or 32 chosen ones");
+  e.eff = positive(v.at("expert"), "ff");
+  e.effp = pad8(e.eff);
+  if (given(v, "shared")) {
+    e.sff = positive(v.at("shared"), "ff");
+    e.sffp = pad8(e.sff);
+  }
+  return e;
+}
+
+// One norm, token shift, mixer and feed-forward side by side, each behind its own gate.
+Layer parse_parallel_layer(const Model& m, const Value& lv, Layout& lay, const std::string& p) {
+  const std::string mix = p + "mix.", mlp = p + "mlp.", type = lv.at("type").string();
+  const int W = m.width;
+  Layer L;
+  L.norm1 = lay.vec(p + "norm1", W);
+  L.shift = lay.vec(p + "shift", W);
+  const Value& mv = lv.at("mixer");
+  if (type == "latent_attention") L.branches.push_back(parse_latent(mv));
+  else if (type == "wkv") L.branches.push_back(parse_wkv(mv));
+  else bad("unknown mixer type '" + type + "'");
+  Branch& b = L.branches[0];
+  lay.begin_stack(W);
+  if (b.kind == BranchKind::kLatent) place_latent(b, lay, mix);
+  else place_wkv(b, lay, mix);
+  L.n_in = lay.end_stack(&L.w_in);
+  place_rest(b, lay, mix, W);
+
+  if (given(lv, "mlp")) {
+    const Value& f = lv.at("mlp");
+    const std::string kind = f.at("kind").string();
+    if (kind == "dense") {
+      L.ffn = FeedForward::kGeluGlu;
+      L.ff = positive(f, "ff");
+      L.ffp = pad8(L.ff);
+    } else if (kind == "moe") {
+      L.ffn = FeedForward::kMoe;
+      L.moe = parse_moe(f);
+    } else {
+      bad("unknown feed-forward kind '" + kind + "'");
+    }
+  }
+  Moe& e = L.moe;
+  lay.begin_stack(W);
+  L.col_rg1 = lay.stacked(p + "rg1", W);
+  if (L.ffn != FeedForward::kNone) L.col_rg2 = lay.stacked(p + "rg2", W);
+  if (L.ffn == FeedForward::kGeluGlu || e.sff > 0) {
+    const std::string q = L.ffn == FeedForward::kGeluGlu ? mlp : mlp + "shared.";
+    const int ff = L.ffn == FeedForward::kGeluGlu ? L.ff : e.sff;
+    L.col_gu = lay.stacked(q + "gate", ff);
+    lay.stacked(q + "up", ff);
+  }
+  if (L.ffn == FeedForward::kMoe) {
+    L.col_router = lay.stacked(mlp + "router", e.outputs());
+    if (e.sff > 0) L.col_sg = lay.stacked(mlp + "shared.sg", 1);
+  }
+  L.n_side = lay.end_stack(&L.w_side);
+  L.b_rg1 = lay.vec(p + "rg1.b", W);
+  if (L.ffn != FeedForward::kNone) L.b_rg2 = lay.vec(p + "rg2.b", W);
+  if (L.ffn == FeedForward::kGeluGlu) {
+    L.w_down = lay.matrix(mlp + "down", W, L.ff);
+    L.ld_down = L.ffp;
+  } else if (L.ffn == FeedForward::kMoe) {
+    e.correction = lay.vec(mlp + "correction", e.outputs());
+    lay.begin_stack(W);
+    for (int i = 0; i < e.experts; ++i) {
+      lay.stacked(mlp + "e" + std::to_string(i) + ".gate", e.eff);
+      lay.stacked(mlp + "e" + std::to_string(i) + ".up", e.eff);
+    }
+    lay.end_stack(&e.w_gu);
+    lay.begin_stack(e.eff);
+    for (int i = 0; i < e.experts; ++i) lay.stacked(mlp + "e" + std::to_string(i) + ".down", W);
+    lay.end_stack(&e.w_down);
+    e.ld_down = e.effp;
+    if (e.sff > 0) {
+      e.w_sdown = lay.matrix(mlp + "shared.down", W, e.sff);
+      e.ld_sdown = e.sffp;
+    }
+  }
+  return L;
+}
+
+void parse_parallel_model(const Value& c, Layout& lay, Model& m) {
+  m.arrangement = Arrangement::kParallel;
+  m.norm_groups = positive(c.at("norm"), "groups");
+  if (m.width % m.norm_groups != 0) bad("norm.groups must divide the width");
+  m.embed_scale = static_cast<float>(c.at("embedding").at("scale").number());
+  m.embed = lay.matrix("embed", m.vocab, m.width);
+  const minijson::Array& layers = c.at("layers").array();
+  std::vector<int> source;   // whose weights a layer uses; every layer has a cache and state of its own
+  for (size_t i = 0; i < layers.size(); ++i) {
+    const double j = given(layers[i], "weights_of") ? layers[i].at("weights_of").number() : static_cast<double>(i);
+    if (!(j >= 0.0 && j < static_cast<double>(layers.size())) || j != std::floor(j)) bad("'weights_of' must name a layer");
+    source.push_back(static_cast<int>(j));
+  }
+  m.layers.resize(layers.size());
+  for (size_t i = 0; i < layers.size(); ++i)
+    if (source[i] == static_cast<int>(i)) m.layers[i] = parse_parallel_layer(m, layers[i], lay, "l" + std::to_string(i) + ".");
+  for (size_t i = 0; i < layers.size(); ++i) {
+    if (source[source[i]] != source[i]) bad("'weights_of' must name a layer with weights of its own");
+    if (source[i] != static_cast<int>(i)) m.layers[i] = m.layers[source[i]];
+  }
+}
+
+}  // namespace
+
 double RopeSpec::frequency(int i) const {
   const double f = std::pow(base, -2.0 * i / dims);
   if (!scaled) return f;
@@ -220,7 +402,7 @@ void parse_model(const std::string& config_json, const std::string& tensors_json
   const Value c = minijson::parse(config_json);
   const Value shapes = minijson::parse(tensors_json);
   const std::string arch = c.at("architecture").string();
-  if (arch != "Zutalix") bad("unknown architecture '" + arch + "'");
+  if (arch != "Zutalix" && arch != "Detatar") bad("unknown architecture '" + arch + "'");
   if (dtype != CTDK_DTYPE_F32 && dtype != CTDK_DTYPE_BF16) bad("unknown dtype");
   Model& m = *out;
   m = Model();
@@ -231,6 +413,12 @@ void parse_model(const std::string& config_json, const std::string& tensors_json
   m.ldw = pad8(m.width);
   m.eps = static_cast<float>(c.at("norm").at("eps").number());
   Layout lay(&m, shapes);
+  if (arch == "Detatar") {
+    parse_parallel_model(c, lay, m);
+    m.final_norm = lay.vec("final.norm", m.width);
+    m.head = lay.matrix("head", m.vocab, m.width);
+    return;
+  }
   m.embed = lay.matrix("embed", m.vocab, m.width);
   m.embed_norm = lay.vec("embed.norm", m.width);
   int i = 0;
@@ -263,6 +451,7 @@ void parse_model(const std::string& config_json, const std::string& tensors_json
     if (lv.contains("mlp") && lv.at("mlp").kind != Value::kNull) {
       const Value& f = lv.at("mlp");
       if (f.at("kind").string() != "dense") bad("unknown feed-forward kind '" + f.at("kind").string() + "'");
+      L.ffn = FeedForward::kClampedGlu;
       L.ff = positive(f, "ff");
       L.ffp = pad8(L.ff);
       L.limit = static_cast<float>(f.at("limit").number());

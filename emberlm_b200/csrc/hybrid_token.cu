@@ -10,6 +10,8 @@
 #include "decode_core.h"
 #include "hybrid_kernels.h"
 #include "hybrid_token.h"
+#include "moe_route.cuh"
+#include "parallel_kernels.h"
 
 namespace ctdk {
 namespace hybrid {
@@ -34,6 +36,12 @@ struct Chunk<float> {
     acc = fmaf(w.z, v.z, acc);
     return fmaf(w.w, v.w, acc);
   }
+  __device__ __forceinline__ void unpack(float (&o)[4]) const {
+    o[0] = w.x;
+    o[1] = w.y;
+    o[2] = w.z;
+    o[3] = w.w;
+  }
 };
 template <>
 struct Chunk<__nv_bfloat16> {
@@ -50,6 +58,14 @@ struct Chunk<__nv_bfloat16> {
     acc = fmaf(__uint_as_float(w.z & 0xffff0000u), b.y, acc);
     acc = fmaf(__uint_as_float(w.w << 16), b.z, acc);
     return fmaf(__uint_as_float(w.w & 0xffff0000u), b.w, acc);
+  }
+  __device__ __forceinline__ void unpack(float (&o)[8]) const {
+    const uint32_t u[4] = {w.x, w.y, w.z, w.w};
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      o[2 * i] = __uint_as_float(u[i] << 16);
+      o[2 * i + 1] = __uint_as_float(u[i] & 0xffff0000u);
+    }
   }
 };
 
@@ -475,10 +491,476 @@ __device__ void delta_item(const TokenPhase& ph, const TokenBranch& br, int item
   if (wid == 0 && live) br.out[h * br.vdim + c] = o;
 }
 
+// ---- parallel arrangement ----
+
+// Experts of the token, chosen by every CTA for itself.
+struct Routed {
+  int32_t index[32];
+  float weight[32];
+};
+
+// The staged rows of ShiftNormArgs for one token. A thread keeps to its own columns.
+template <typename T>
+__device__ void stage_shift_norm(const TokenArgs& a, const TokenPhase& ph, int64_t tok, int pos, float* sm) {
+  const TokenShift& f = ph.shift;
+  const int W = a.width, gs = W / f.groups, lane = threadIdx.x & 31, wid = threadIdx.x >> 5;
+  const int g0 = wid / f.wpg, gstep = kWarps / f.wpg, wj = wid % f.wpg;
+  const bool active = g0 < gstep, writer = blockIdx.x == 0;
+  const T* e = ph.first_token ? static_cast<const T*>(a.embed) + tok * a.ld_embed : nullptr;
+  float *xs = sm, *part = sm + f.red;
+  __syncthreads();   // the scratch may still be read as part of an earlier phase
+  for (int g = g0; active && g < f.groups; g += gstep) {
+    float ss = 0.0f;
+    for (int c = g * gs + wj * 32 + lane; c < (g + 1) * gs; c += 32 * f.wpg) {
+      float x;
+      if (e != nullptr) {
+        x = to_f(e[c]) * a.embed_scale;
+      } else {
+        x = ldg_f(f.y1 + c) * sigmoid_f(ldg_f(f.z1 + c) + f.b1[c]);
+        if (f.y2 != nullptr) x += ldg_f(f.y2 + c) * sigmoid_f(ldg_f(f.z2 + c) + f.b2[c]);
+        x += ldg_f(f.x + c);
+      }
+      if (writer && f.x_out != nullptr) f.x_out[c] = x;
+      xs[c] = x;
+      ss += x * x;
+    }
+    ss = warp_sum(ss);
+    if (lane == 0) part[g * f.wpg + wj] = ss;
+  }
+  __syncthreads();
+  const float* prev = f.state != nullptr ? f.state + ((pos + 1) & 1) * 2 * W : nullptr;
+  float* next = f.state != nullptr ? f.state + (pos & 1) * 2 * W : nullptr;
+  for (int g = g0; active && g < f.groups; g += gstep) {
+    float ss = 0.0f;
+    for (int k = 0; k < f.wpg; ++k) ss += part[g * f.wpg + k];
+    const float sc = rsqrtf(ss / static_cast<float>(gs) + a.eps);
+    for (int c = g * gs + wj * 32 + lane; c < (g + 1) * gs; c += 32 * f.wpg) {
+      const float h = xs[c] * sc * f.w[c];
+      xs[c] = h;
+      if (f.shift == nullptr) continue;
+      const float m = fmaf((pos > 0 ? ldg_f(prev + c) : 0.0f) - h, f.shift[c], h);
+      sm[f.ld + c] = m;
+      if (writer) {
+        f.h_out[c] = h;
+        next[c] = h;
+        if (f.n_mix > 0) next[W + c] = m;
+      }
+      if (f.n_mix == 0) continue;
+      const float d = (pos > 0 ? ldg_f(prev + W + c) : 0.0f) - m;
+#pragma unroll
+      for (int i = 0; i < kTokenMixes; ++i) sm[(2 + i) * f.ld + c] = fmaf(d, f.mu[i][c], m);
+    }
+  }
+  const int rows = f.shift == nullptr ? 1 : 2 + f.n_mix, pad = f.ld - W;
+  for (int i = threadIdx.x; i < rows * pad; i += kThreads) sm[i / pad * f.ld + W + i % pad] = 0.0f;
+  __syncthreads();
+}
+
+template <typename T>
+__device__ void stage_list(const TokenArgs& a, const TokenPhase& ph, int64_t tok, int pos, float* sm, float* red, Routed& routed) {
+  const int lane = threadIdx.x & 31, wid = threadIdx.x >> 5;
+  for (int i = 0; i < ph.n_ops; ++i) {
+    const StageOp& op = ph.op[i];
+    float* xs = sm + op.at;
+    if (op.kind == kOpShiftNorm) {
+      stage_shift_norm<T>(a, ph, tok, pos, sm);
+    } else if (op.kind == kOpRmsNorm) {
+      float ss[1] = {0.0f};
+      for (int c = threadIdx.x; c < op.n; c += kThreads) {
+        const float v = ldg_f(op.src + c);
+        xs[c] = v;
+        ss[0] += v * v;
+      }
+      block_sum<1>(ss, red);
+      const float sc = rsqrtf(ss[0] / static_cast<float>(op.n) + a.eps);
+      for (int c = threadIdx.x; c < op.ld; c += kThreads) xs[c] = c < op.n ? xs[c] * sc * op.w[c] : 0.0f;
+    } else if (op.kind == kOpCopy) {
+      for (int c = threadIdx.x; c < op.ld; c += kThreads) xs[c] = c < op.n ? ldg_f(op.src + c) : 0.0f;
+    } else if (op.kind == kOpRoute) {
+      if (wid == 0) {   // logits, then the scratch of the choice, at `at`
+        for (int c = lane; c < op.n; c += 32) xs[c] = ldg_f(op.src + c);
+        __syncwarp();
+        route_token(xs, op.w, op.n, ph.route_groups, ph.route_keep, ph.route_top, xs + op.n, routed.index, routed.weight);
+      }
+      __syncthreads();
+    } else if (op.kind == kOpGelu) {
+      for (int c = threadIdx.x; c < op.n; c += kThreads) xs[c] = gelu_tanh_f(ldg_f(op.src + c)) * ldg_f(op.src + op.ld + c);
+    } else if (op.kind == kOpShared) {
+      const float g = sigmoid_f(ldg_f(op.src2));
+      for (int c = threadIdx.x; c < op.n; c += kThreads) xs[c] = g * silu_f(ldg_f(op.src + c)) * ldg_f(op.src + op.ld + c);
+    } else if (op.kind == kOpExperts) {
+      const int n = op.n;
+      for (int c = threadIdx.x; c < ph.route_top * n; c += kThreads) {
+        const int k = c / n;
+        const float* g = op.src + 2 * k * n + c % n;
+        xs[c] = routed.index[k] < op.ld ? routed.weight[k] * silu_f(ldg_f(g)) * ldg_f(g + n) : 0.0f;   // ld: number of experts
+      }
+    } else if (op.kind == kOpHeadNorm) {
+      const TokenBranch& br = ph.br[0];
+      for (int h = wid; h < br.H; h += kWarps) {
+        const float* o = op.src + h * br.dim;
+        float ss = 0.0f;
+        for (int d = lane; d < br.dim; d += 32) {
+          const float v = ldg_f(o + d);
+          ss += v * v;
+        }
+        const float sc = rsqrtf(warp_sum(ss) / static_cast<float>(br.dim) + a.eps);
+        for (int d = lane; d < br.dim; d += 32) {
+          const int c = h * br.dim + d;
+          xs[c] = ldg_f(o + d) * sc * op.w[c] * silu_f(ldg_f(op.src2 + c));
+        }
+      }
+      for (int c = op.n + threadIdx.x; c < op.ld; c += kThreads) xs[c] = 0.0f;
+    } else if (blockIdx.x == gridDim.x - 1) {   // kOpLatentStore
+      const TokenBranch& br = ph.br[0];
+      const float* x = ph.proj + br.col_k;
+      T* row = static_cast<T*>(br.cache) + static_cast<int64_t>(pos) * br.ld_cache;
+      float ss[1] = {0.0f};
+      for (int c = threadIdx.x; c < br.kv_rank; c += kThreads) {
+        const float v = ldg_f(x + c);
+        ss[0] += v * v;
+      }
+      block_sum<1>(ss, red);
+      const float sc = rsqrtf(ss[0] / static_cast<float>(br.kv_rank) + a.eps);
+      for (int c = threadIdx.x; c < br.kv_rank; c += kThreads) row[c] = from_f<T>(ldg_f(x + c) * sc * br.kv_norm[c]);
+      const int half = br.rot_dim / 2;
+      for (int p = threadIdx.x; p < half; p += kThreads) {
+        const float u = ldg_f(x + br.kv_rank + p), v = ldg_f(x + br.kv_rank + half + p);
+        const float2 cs = br.table[static_cast<int64_t>(pos) * half + p];
+        row[br.rot_col + p] = from_f<T>(u * cs.x - v * cs.y);
+        row[br.rot_col + half + p] = from_f<T>(v * cs.x + u * cs.y);
+      }
+    }
+  }
+  __syncthreads();
+}
+
+// Row r of a product, this warp's part of it (all lanes get the sum).
+template <typename T>
+__device__ __forceinline__ float gemv_row(const TokenGemv& g, int r, const float* sm, int part, int wpr, const Routed& routed) {
+  const T* W = static_cast<const T*>(g.W);
+  if (g.mode == kGemvPlain) return row_dot<T>(W + static_cast<int64_t>(r) * g.K, sm + g.in, g.K, part, wpr);
+  if (g.mode == kGemvExpertUp) {
+    const int e = routed.index[r / g.per];
+    if (e >= g.experts) return 0.0f;
+    return row_dot<T>(W + (static_cast<int64_t>(e) * g.pitch + r % g.per) * g.K, sm + g.in, g.K, part, wpr);
+  }
+  float v = 0.0f;
+  for (int k = 0; k < g.top; ++k) {
+    const int e = routed.index[k];
+    if (e < g.experts) v += row_dot<T>(W + (static_cast<int64_t>(e) * g.pitch + r) * g.K, sm + g.in + k * g.K, g.K, part, wpr);
+    else if (part == 0) v = fmaf(routed.weight[k], ldg_f(g.h + r), v);
+  }
+  if (g.W2 != nullptr) v += row_dot<T>(static_cast<const T*>(g.W2) + static_cast<int64_t>(r) * g.K2, sm + g.in2, g.K2, part, wpr);
+  return v;
+}
+
+// 32 value columns of one wkv head (as delta_item: a lane per column, key rows dealt to the warps).
+template <typename T>
+__device__ void wkv_item(const TokenPhase& ph, const TokenBranch& br, int item, int pos, float* sm) {
+  const int nb = (br.dim + 31) / 32, h = item / nb, lane = threadIdx.x & 31, wid = threadIdx.x >> 5;
+  const int dim = br.dim, c = (item % nb) * 32 + lane, rw = (br.rank_w + 7) & ~7;
+  float *low = sm, *q = low + rw, *k = q + dim, *g = k + dim, *b = g + dim, *red = b + dim;
+  __syncthreads();
+  for (int i = threadIdx.x; i < rw; i += kThreads) low[i] = i < br.rank_w ? tanhf(ldg_f(ph.proj + br.col_w1 + i)) : 0.0f;
+  __syncthreads();
+  for (int d = threadIdx.x; d < dim; d += kThreads) {
+    const int ch = h * dim + d;
+    q[d] = ldg_f(ph.proj + br.col_r + ch);
+    k[d] = ldg_f(ph.proj + br.col_k + ch);
+    b[d] = br.bonus[ch];
+    g[d] = expf(-expf(short_dot(static_cast<const T*>(br.w_w2) + static_cast<int64_t>(ch) * rw, low, rw) + br.w0[ch]));
+  }
+  const bool live = c < dim;
+  const float v = live ? ldg_f(ph.proj + br.col_v + h * dim + c) : 0.0f;
+  float* S = br.state + static_cast<int64_t>(h) * dim * dim + c;
+  __syncthreads();
+  float o = 0.0f;
+  if (live) {
+#pragma unroll 8
+    for (int r = wid; r < dim; r += kWarps) {
+      const float s0 = pos > 0 ? ldg_f(S + static_cast<int64_t>(r) * dim) : 0.0f, kv = k[r] * v;
+      o = fmaf(fmaf(b[r], kv, s0), q[r], o);
+      S[static_cast<int64_t>(r) * dim] = fmaf(g[r], s0, kv);
+    }
+  }
+  o = column_sum(o, red);
+  if (wid == 0 && live) br.out[h * dim + c] = o;
+}
+
+template <typename T>
+constexpr int kKeyCols = 16 * Chunk<T>::kN;   // latent columns of a key item
+
+// Queries against the cache rows: W_uk^T q for one block of latent columns of a head; the first block also
+// turns the rotated part. Threads: 16 column groups of one 16-byte chunk, 16 groups of key dimensions.
+template <typename T>
+__device__ void latent_keys_item(const TokenPhase& ph, const TokenBranch& br, int item, int pos, float* sm) {
+  constexpr int N = Chunk<T>::kN, COLS = kKeyCols<T>;
+  const int nb = (br.rot_col + COLS - 1) / COLS, h = item / nb, r0 = item % nb * COLS;
+  const int cg = threadIdx.x & 15, dg = threadIdx.x >> 4, col = r0 + cg * N;
+  const float* q = br.q_up + h * (br.dim + br.rot_dim);
+  float acc[N];
+#pragma unroll
+  for (int e = 0; e < N; ++e) acc[e] = 0.0f;
+  if (col < br.ld_ukv) {
+    const T* w = static_cast<const T*>(br.w_ukv) + static_cast<int64_t>(h) * br.dim * br.ld_ukv + col;
+#pragma unroll 8
+    for (int d = dg; d < br.dim; d += 16) {
+      Chunk<T> c;
+      c.load(w + static_cast<int64_t>(d) * br.ld_ukv);
+      const float x = ldg_f(q + d);
+      float f[N];
+      c.unpack(f);
+#pragma unroll
+      for (int e = 0; e < N; ++e) acc[e] = fmaf(x, f[e], acc[e]);
+    }
+  }
+  __syncthreads();
+#pragma unroll
+  for (int e = 0; e < N; ++e) sm[dg * (COLS + 1) + cg * N + e] = acc[e];
+  __syncthreads();
+  float* out = br.q_abs + static_cast<int64_t>(h) * br.ld_cache;
+  for (int c = threadIdx.x; c < COLS; c += kThreads) {
+    float v = 0.0f;
+#pragma unroll
+    for (int g = 0; g < 16; ++g) v += sm[g * (COLS + 1) + c];
+    if (r0 + c < br.kv_rank) out[r0 + c] = v * br.scale;
+  }
+  if (r0 == 0) {
+    const int half = br.rot_dim / 2;
+    for (int p = threadIdx.x; p < half; p += kThreads) {
+      const float u = ldg_f(q + br.dim + p), v = ldg_f(q + br.dim + half + p);
+      const float2 cs = br.table[static_cast<int64_t>(pos) * half + p];
+      out[br.rot_col + p] = (u * cs.x - v * cs.y) * br.scale;
+      out[br.rot_col + half + p] = (v * cs.x + u * cs.y) * br.scale;
+    }
+  }
+}
+
+// Position ranges in use for L cached positions, and their length.
+__device__ __forceinline__ int latent_ranges(int L, int splits, int& per) {
+  int n = (L + kLatentKeys - 1) / kLatentKeys;
+  if (n > splits) n = splits;
+  per = (L + n - 1) / n;
+  return (L + per - 1) / per;
+}
+
+// kLatentHeads query heads over one range of cached positions: running maximum, sum and the weighted sum of
+// the latents per head. Scores: a warp per head, a lane per position. Sums: a thread per pair of columns.
+template <typename T, int PAIRS>
+__device__ void latent_scan_item(const TokenBranch& br, int item, int pos, float* sm) {
+  constexpr int N = Chunk<T>::kN, HB = kLatentHeads, KT = kLatentKeys;
+  const int blk = item / br.splits, sp = item % br.splits;
+  int per;
+  const int n_act = latent_ranges(pos + 1, br.splits, per);
+  if (sp >= n_act) return;
+  const int lane = threadIdx.x & 31, wid = threadIdx.x >> 5, ldc = br.ld_cache;
+  const int j0 = sp * per, j1 = min(pos + 1, j0 + per);
+  const int chunks = ldc / N, pitch = chunks | 1;       // 16-byte chunks per row; odd pitch: conflict-free
+  float* qs = sm;                                       // [HB][ldc]
+  float* ps = qs + HB * ldc;                            // [HB][KT] scores, then weights
+  float* st = ps + HB * KT;                             // [HB] correction of the sums
+  uint4* tile = reinterpret_cast<uint4*>(st + HB);      // [KT][pitch]
+  for (int i = threadIdx.x; i < HB * ldc; i += kThreads) {
+    const int h = blk * HB + i / ldc;
+    qs[i] = h < br.H ? ldg_f(br.q_abs + static_cast<int64_t>(h) * ldc + i % ldc) : 0.0f;
+  }
+  float m = -FLT_MAX, l = 0.0f;   // of head wid
+  float2 acc[PAIRS][HB];
+#pragma unroll
+  for (int p = 0; p < PAIRS; ++p)
+#pragma unroll
+    for (int h = 0; h < HB; ++h) acc[p][h] = make_float2(0.0f, 0.0f);
+  const uint4* cache = reinterpret_cast<const uint4*>(static_cast<const T*>(br.cache));
+  for (int jb = j0; jb < j1; jb += KT) {
+    const int nk = min(KT, j1 - jb);
+    __syncthreads();
+#pragma unroll 4
+    for (int i = threadIdx.x; i < KT * chunks; i += kThreads) {
+      const int r = i / chunks, c = i % chunks;
+      tile[r * pitch + c] = r < nk ? __ldcg(cache + static_cast<int64_t>(jb + r) * chunks + c) : make_uint4(0u, 0u, 0u, 0u);
+    }
+    __syncthreads();
+    {
+      const float* q = qs + wid * ldc;
+      float s0 = 0.0f, s1 = 0.0f;
+#pragma unroll 2
+      for (int c = 0; c < chunks; ++c) {
+        Chunk<T> k;
+        k.w = *reinterpret_cast<const decltype(k.w)*>(tile + lane * pitch + c);
+        if (c & 1) s1 = k.dot(q + c * N, s1);
+        else s0 = k.dot(q + c * N, s0);
+      }
+      const float s = lane < nk ? s0 + s1 : -FLT_MAX;
+      const float mn = fmaxf(m, warp_max(s));
+      const float p = lane < nk ? expf(s - mn) : 0.0f, c = expf(m - mn);
+      l = l * c + warp_sum(p);
+      m = mn;
+      ps[wid * KT + lane] = p;
+      if (lane == 0) st[wid] = c;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int p = 0; p < PAIRS; ++p) {
+      const int col = 2 * (threadIdx.x + p * kThreads);
+      if (col >= br.kv_rank) break;
+#pragma unroll
+      for (int h = 0; h < HB; ++h) {
+        acc[p][h].x *= st[h];
+        acc[p][h].y *= st[h];
+      }
+      const T* row = reinterpret_cast<const T*>(tile) + col;
+#pragma unroll 1
+      for (int j = 0; j < KT; j += 4) {
+        float x[4], y[4];
+#pragma unroll
+        for (int u = 0; u < 4; ++u) {
+          x[u] = to_f(row[(j + u) * pitch * N]);
+          y[u] = to_f(row[(j + u) * pitch * N + 1]);
+        }
+#pragma unroll
+        for (int h = 0; h < HB; ++h) {
+          const float4 w = *reinterpret_cast<const float4*>(ps + h * KT + j);
+          acc[p][h].x = fmaf(w.x, x[0], fmaf(w.y, x[1], fmaf(w.z, x[2], fmaf(w.w, x[3], acc[p][h].x))));
+          acc[p][h].y = fmaf(w.x, y[0], fmaf(w.y, y[1], fmaf(w.z, y[2], fmaf(w.w, y[3], acc[p][h].y))));
+        }
+      }
+    }
+  }
+  const int PS = br.rot_col + kAttnStats;
+  auto part = [&](int h) { return br.part + (static_cast<int64_t>(blk * HB + h) * br.splits + sp) * PS; };
+#pragma unroll
+  for (int p = 0; p < PAIRS; ++p) {
+    const int col = 2 * (threadIdx.x + p * kThreads);
+    if (col >= br.kv_rank) break;
+#pragma unroll
+    for (int h = 0; h < HB; ++h)   // rows end on an even column: rot_col is a multiple of eight
+      if (blk * HB + h < br.H) *reinterpret_cast<float2*>(part(h) + kAttnStats + col) = acc[p][h];
+  }
+  if (lane == 0 && blk * HB + wid < br.H) {
+    part(wid)[0] = m;
+    part(wid)[1] = l;
+  }
+}
+
+// kLatentOutRows value rows of a head: merges the head's ranges, then W_uv times the mean latent, gated.
+template <typename T>
+__device__ void latent_out_item(const TokenPhase& ph, const TokenBranch& br, int item, int pos, float* sm) {
+  const int nb = (br.vdim + kLatentOutRows - 1) / kLatentOutRows, h = item / nb, r0 = item % nb * kLatentOutRows;
+  const int lane = threadIdx.x & 31, wid = threadIdx.x >> 5, PS = br.rot_col + kAttnStats;
+  int per;
+  const int n_act = latent_ranges(pos + 1, br.splits, per);
+  float *o = sm, *w = o + br.rot_col;   // [rot_col] mean latent, [splits] weights of the ranges
+  const float* part = br.part + static_cast<int64_t>(h) * br.splits * PS;
+  __syncthreads();
+  if (wid == 0) {
+    float m = -FLT_MAX;
+    for (int s = lane; s < n_act; s += 32) m = fmaxf(m, ldg_f(part + static_cast<int64_t>(s) * PS));
+    m = warp_max(m);
+    float l = 0.0f;
+    for (int s = lane; s < n_act; s += 32) {
+      const float e = expf(ldg_f(part + static_cast<int64_t>(s) * PS) - m);
+      w[s] = e;
+      l += e * ldg_f(part + static_cast<int64_t>(s) * PS + 1);
+    }
+    l = 1.0f / warp_sum(l);
+    __syncwarp();
+    for (int s = lane; s < n_act; s += 32) w[s] *= l;
+  }
+  __syncthreads();
+  for (int c = threadIdx.x; c < br.rot_col; c += kThreads) {
+    float v = 0.0f;
+    if (c < br.kv_rank)
+#pragma unroll 8
+      for (int s = 0; s < n_act; ++s) v = fmaf(w[s], ldg_f(part + static_cast<int64_t>(s) * PS + kAttnStats + c), v);
+    o[c] = v;
+  }
+  __syncthreads();
+  const float gate = sigmoid_f(ldg_f(ph.proj + br.col_g + h));
+  for (int r = r0 + wid; r < min(br.vdim, r0 + kLatentOutRows); r += kWarps) {
+    const T* row = static_cast<const T*>(br.w_ukv) + (static_cast<int64_t>(br.row_uv) + h * br.vdim + r) * br.ld_ukv;
+    const float v = row_dot<T>(row, o, br.ld_ukv, 0, 1);
+    if (lane == 0) br.out[h * br.vdim + r] = v * gate;
+  }
+}
+
+template <typename T>
+__device__ void list_item(const TokenPhase& ph, int item, int pos, float* sm) {
+  const TokenBranch& br = ph.br[0];
+  if (br.kind == kTokWkv) wkv_item<T>(ph, br, item, pos, sm);
+  else if (br.kind == kTokLatentKeys) latent_keys_item<T>(ph, br, item, pos, sm);
+  else if (br.kind == kTokLatentOut) latent_out_item<T>(ph, br, item, pos, sm);
+  else if (br.kv_rank <= 2 * kThreads) latent_scan_item<T, 1>(br, item, pos, sm);
+  else latent_scan_item<T, 2>(br, item, pos, sm);
+}
+
+// Staging, products, items. The items lie at the front of the grid, so rows start behind them.
+template <typename T>
+__device__ unsigned long long list_phase(const TokenArgs& a, const TokenPhase& ph, int64_t tok, int pos, float* sm, float* red, float* part_red,
+                                         Routed& routed) {
+  const int lane = threadIdx.x & 31, wid = threadIdx.x >> 5;
+  if (ph.n_ops > 0) stage_list<T>(a, ph, tok, pos, sm, red, routed);
+  unsigned long long best = 0ull;
+  int total = 0;
+  for (int i = 0; i < ph.n_gemv; ++i) total += ph.gemv[i].rows;
+  const int items = ph.n_branch > 0 ? ph.br[0].items : 0;
+  int cta = static_cast<int>(blockIdx.x) - items % static_cast<int>(gridDim.x);
+  if (cta < 0) cta += gridDim.x;
+  const int wpr = ph.wpr, groups = kWarps / (wpr > 0 ? wpr : 1), part = wpr > 0 ? wid % wpr : 0;
+  auto find = [&](int n, int& r) {
+    int i = 0;
+    while (n >= ph.gemv[i].rows) n -= ph.gemv[i++].rows;
+    r = n;
+    return i;
+  };
+  auto finish = [&](const TokenGemv& g, int r, float v) {
+    g.y[r] = v;
+    if (ph.is_head) {
+      const unsigned long long k = argmax_key(v, r);
+      best = k > best ? k : best;
+    }
+  };
+  if (wpr == 1) {
+    for (int n = cta * kWarps + wid; n < total; n += gridDim.x * kWarps) {
+      int r;
+      const TokenGemv& g = ph.gemv[find(n, r)];
+      const float v = gemv_row<T>(g, r, sm, 0, 1, routed);
+      if (lane == 0) finish(g, r, v);
+    }
+  } else {
+    for (int nb = cta * groups; nb < total; nb += gridDim.x * groups) {
+      const int n = nb + wid / wpr;
+      int r = 0;
+      float v = 0.0f;
+      const TokenGemv& g = ph.gemv[n < total ? find(n, r) : 0];
+      if (n < total) v = gemv_row<T>(g, r, sm, part, wpr, routed);
+      if (lane == 0) part_red[wid] = v;
+      __syncthreads();
+      if (part == 0 && lane == 0 && n < total) {
+        float t = 0.0f;
+        for (int w = 0; w < wpr; ++w) t += part_red[wid + w];
+        finish(g, r, t);
+      }
+      __syncthreads();
+    }
+  }
+  for (int it = blockIdx.x; it < items; it += gridDim.x) {
+    __syncthreads();
+    list_item<T>(ph, it, pos, sm);
+  }
+  return best;
+}
+
 template <typename T>
 __device__ void prefetch_phase(const TokenPhase& ph) {
+  if (ph.extra != nullptr) {
+    const char* base = static_cast<const char*>(ph.extra);
+    for (int64_t i = static_cast<int64_t>(blockIdx.x) * kThreads + threadIdx.x; i < ph.extra_bytes / 128; i += static_cast<int64_t>(gridDim.x) * kThreads)
+      prefetch_l2(base + i * 128);
+  }
   for (int s = 0; s < ph.n_gemv; ++s) {
     const TokenGemv& g = ph.gemv[s];
+    if (g.mode != kGemvPlain) continue;   // which experts is not known yet
     const char* base = static_cast<const char*>(g.W);
     const int64_t lines = static_cast<int64_t>(g.rows) * g.K * sizeof(T) / 128;
     for (int64_t i = static_cast<int64_t>(blockIdx.x) * kThreads + threadIdx.x; i < lines; i += static_cast<int64_t>(gridDim.x) * kThreads)
@@ -486,7 +968,8 @@ __device__ void prefetch_phase(const TokenPhase& ph) {
   }
 }
 
-template <typename T>
+// LIST: every phase is a kStageList phase (parallel arrangement); otherwise none is.
+template <typename T, bool LIST>
 __global__ void __launch_bounds__(kThreads, 2) hybrid_token_kernel(const __grid_constant__ TokenArgs a) {
   extern __shared__ __align__(16) float sm[];
   __shared__ TokenPhase ph_s[2];
@@ -494,6 +977,7 @@ __global__ void __launch_bounds__(kThreads, 2) hybrid_token_kernel(const __grid_
   __shared__ float part_red[kWarps];
   __shared__ unsigned long long best_s[kWarps];
   __shared__ int s_flag;
+  __shared__ Routed routed;
   const int lane = threadIdx.x & 31, wid = threadIdx.x >> 5;
   unsigned int epoch = 0;
   int pos = a.counters[0];
@@ -510,7 +994,10 @@ __global__ void __launch_bounds__(kThreads, 2) hybrid_token_kernel(const __grid_
     __syncthreads();
     for (int i = 0; i < a.n_phases; ++i) {
       const TokenPhase& ph = ph_s[i & 1];
-      if (ph.is_mix) {
+      unsigned long long best = 0ull;
+      if constexpr (LIST) {
+        best = list_phase<T>(a, ph, tok, pos, sm, red, part_red, routed);
+      } else if (ph.is_mix) {
         int first = 0;
         for (int b = 0; b < ph.n_branch; ++b) {
           const TokenBranch& br = ph.br[b];
@@ -534,7 +1021,6 @@ __global__ void __launch_bounds__(kThreads, 2) hybrid_token_kernel(const __grid_
         }
         const int wpr = ph.wpr, groups = kWarps / wpr, part = wid % wpr;
         const int rows0 = ph.gemv[0].rows, total = rows0 + (ph.n_gemv > 1 ? ph.gemv[1].rows : 0);
-        unsigned long long best = 0ull;
         if (wpr == 1) {
           for (int n = blockIdx.x * kWarps + wid; n < total; n += gridDim.x * kWarps) {
             const TokenGemv& g = ph.gemv[n < rows0 ? 0 : 1];
@@ -570,14 +1056,14 @@ __global__ void __launch_bounds__(kThreads, 2) hybrid_token_kernel(const __grid_
             __syncthreads();
           }
         }
-        if (ph.is_head && a.out_tokens != nullptr) {
-          if (lane == 0) best_s[wid] = best;
-          __syncthreads();
-          if (threadIdx.x == 0) {
+      }
+      if (ph.is_head && a.out_tokens != nullptr) {
+        if (lane == 0) best_s[wid] = best;
+        __syncthreads();
+        if (threadIdx.x == 0) {
 #pragma unroll
-            for (int w = 1; w < kWarps; ++w) best = best_s[w] > best ? best_s[w] : best;
-            atomicMax(&words[t & 1], best);
-          }
+          for (int w = 1; w < kWarps; ++w) best = best_s[w] > best ? best_s[w] : best;
+          atomicMax(&words[t & 1], best);
         }
       }
       if (ph.prefetch >= 0) prefetch_phase<T>(a.phases[ph.prefetch]);
@@ -609,6 +1095,7 @@ size_t token_smem_bytes(int stage_floats, const TokenPhase* phases, int n) {
     for (int b = 0; phases[i].is_mix && b < phases[i].n_branch; ++b) {
       const TokenBranch& br = phases[i].br[b];
       size_t f = 0;
+      if (phases[i].stage == kStageList) continue;   // counted by the caller
       if (br.kind == kTokAttention) {
         const size_t hq = br.H / br.G, kt = br.dim <= 128 ? 32 : (br.dim <= 256 ? 16 : (br.dim <= 512 ? 8 : 4));
         f = 2 * hq * br.dim + 2 * kt * (br.dim + 1) + hq * 35;
@@ -624,13 +1111,14 @@ size_t token_smem_bytes(int stage_floats, const TokenPhase* phases, int n) {
 }
 
 template <typename T>
-int token_grid(size_t smem, int* grid) {
+int token_grid(size_t smem, bool list, int* grid) {
+  auto* kernel = list ? hybrid_token_kernel<T, true> : hybrid_token_kernel<T, false>;
   int dev = 0, coop = 0, per_sm = 0;
   cudaError_t e = cudaGetDevice(&dev);
   if (e == cudaSuccess) e = cudaDeviceGetAttribute(&coop, cudaDevAttrCooperativeLaunch, dev);
   if (e == cudaSuccess)
-    e = cudaFuncSetAttribute(hybrid_token_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
-  if (e == cudaSuccess) e = cudaOccupancyMaxActiveBlocksPerMultiprocessor(&per_sm, hybrid_token_kernel<T>, kThreads, smem);
+    e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
+  if (e == cudaSuccess) e = cudaOccupancyMaxActiveBlocksPerMultiprocessor(&per_sm, kernel, kThreads, smem);
   if (e != cudaSuccess) return fail(CTDK_ELAUNCH, "hybrid token kernel: %s", cudaGetErrorString(e));
   CTDK_REQUIRE(coop != 0 && per_sm >= 1, "hybrid token kernel: no cooperative launch with %zu bytes of shared memory", smem);
   *grid = sm_count() * (per_sm > 2 ? 2 : per_sm);
@@ -638,21 +1126,21 @@ int token_grid(size_t smem, int* grid) {
 }
 
 template <typename T>
-int launch_token_kernel(const TokenArgs& a, int grid, size_t smem, cudaStream_t s) {
+int launch_token_kernel(const TokenArgs& a, bool list, int grid, size_t smem, cudaStream_t s) {
   if (cudaMemsetAsync(a.sync, 0, a.sync_words * sizeof(unsigned int), s) != cudaSuccess)
     return fail(CTDK_ELAUNCH, "hybrid token kernel: clearing the barrier words failed");
   TokenArgs args = a;
   void* params[] = {&args};
-  const cudaError_t e = cudaLaunchCooperativeKernel(reinterpret_cast<const void*>(hybrid_token_kernel<T>), dim3(grid), dim3(kThreads),
+  const cudaError_t e = cudaLaunchCooperativeKernel(list ? reinterpret_cast<const void*>(hybrid_token_kernel<T, true>) : reinterpret_cast<const void*>(hybrid_token_kernel<T, false>), dim3(grid), dim3(kThreads),
                                                     params, smem, s);
   if (e != cudaSuccess) return fail(CTDK_ELAUNCH, "hybrid token kernel: %s", cudaGetErrorString(e));
   return check_launch("hybrid token kernel");
 }
 
-template int token_grid<float>(size_t, int*);
-template int token_grid<__nv_bfloat16>(size_t, int*);
-template int launch_token_kernel<float>(const TokenArgs&, int, size_t, cudaStream_t);
-template int launch_token_kernel<__nv_bfloat16>(const TokenArgs&, int, size_t, cudaStream_t);
+template int token_grid<float>(size_t, bool, int*);
+template int token_grid<__nv_bfloat16>(size_t, bool, int*);
+template int launch_token_kernel<float>(const TokenArgs&, bool, int, size_t, cudaStream_t);
+template int launch_token_kernel<__nv_bfloat16>(const TokenArgs&, bool, int, size_t, cudaStream_t);
 
 }  // namespace hybrid
 }  // namespace ctdk

@@ -1,6 +1,7 @@
 // Linear-attention recurrences token by token, state in registers (fp32 arithmetic throughout):
 //   lightning      S <- decay_h S + k v^T;                         o = S^T q
 //   channel delta  S <- diag(e^logg) S; u = beta (v - S^T k); S <- S + k u^T;  o = S^T q
+//   wkv            o = (S + diag(bonus) k v^T)^T q;  S <- diag(e^(-e^(z + w0))) S + k v^T
 // One CTA owns 32 value columns of a head, one warp four of them; a lane holds every 32nd key row of
 // the warp's columns, so a token costs two warp reductions and no block barrier. Inputs are staged 16
 // tokens at a time. Used for fp32 models and for short portions; long bfloat16 prompts take the
@@ -29,10 +30,11 @@ __device__ __forceinline__ float warp_sum4(const float (&v)[4]) {
   return r;
 }
 
-template <int RPL, bool DELTA>
+template <int RPL, Recurrence KIND>
 __global__ void __launch_bounds__(256) recurrent_scan_kernel(const ScanArgs a) {
+  constexpr bool DELTA = KIND == Recurrence::kDelta, WKV = KIND == Recurrence::kWkv, GATED = DELTA || WKV;
   constexpr int DK = 32 * RPL, kTile = RPL > 4 ? kMaxTile / 2 : kMaxTile;
-  __shared__ float q_s[kTile][DK], k_s[kTile][DK], g_s[DELTA ? kTile : 1][DELTA ? DK : 1], v_s[kTile][32], b_s[kTile];
+  __shared__ float q_s[kTile][DK], k_s[kTile][DK], g_s[GATED ? kTile : 1][GATED ? DK : 1], v_s[kTile][32], b_s[kTile];
   pdl_launch();
   pdl_wait();
   const int lane = threadIdx.x & 31, wid = threadIdx.x >> 5;
@@ -47,7 +49,10 @@ __global__ void __launch_bounds__(256) recurrent_scan_kernel(const ScanArgs a) {
     for (int j = 0; j < 4; ++j)
       S[i][j] = (a.resume && r < a.dim && cw + j < a.vdim) ? st[static_cast<int64_t>(r) * a.vdim + cw + j] : 0.0f;
   }
-  const float dec = DELTA ? 1.0f : a.decay[h];
+  const float dec = GATED ? 1.0f : a.decay[h];
+  float bonus[RPL];
+#pragma unroll
+  for (int i = 0; i < RPL; ++i) bonus[i] = WKV && lane + 32 * i < a.dim ? a.bonus[h * a.dim + lane + 32 * i] : 0.0f;
   for (int64_t t0 = 0; t0 < a.rows; t0 += kTile) {
     const int nt = static_cast<int>(a.rows - t0 < kTile ? a.rows - t0 : kTile);
     __syncthreads();
@@ -62,10 +67,11 @@ __global__ void __launch_bounds__(256) recurrent_scan_kernel(const ScanArgs a) {
           k = silu_f(k);
         }
         if (DELTA) g = expf(a.logg[((t0 + t) * a.H + h) * a.dim + d]);
+        if (WKV) g = expf(-expf(a.z[(t0 + t) * a.ldz + h * a.dim + d] + a.w0[h * a.dim + d]));
       }
       q_s[t][d] = q;
       k_s[t][d] = k;
-      if (DELTA) g_s[t][d] = g;
+      if (GATED) g_s[t][d] = g;
     }
     for (int i = threadIdx.x; i < nt * 32; i += 256) {
       const int t = i >> 5, c = c0 + (i & 31);
@@ -99,10 +105,13 @@ __global__ void __launch_bounds__(256) recurrent_scan_kernel(const ScanArgs a) {
 #pragma unroll
       for (int i = 0; i < RPL; ++i) {
         const float k = k_s[t][lane + 32 * i], q = q_s[t][lane + 32 * i];
+        const float keep = WKV ? g_s[WKV ? t : 0][WKV ? lane + 32 * i : 0] : dec;
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
-          S[i][j] = DELTA ? fmaf(k, u[j], S[i][j]) : fmaf(dec, S[i][j], k * u[j]);
-          o[j] = fmaf(S[i][j], q, o[j]);
+          const float kv = k * u[j];
+          if (WKV) o[j] = fmaf(fmaf(bonus[i], kv, S[i][j]), q, o[j]);
+          S[i][j] = DELTA ? fmaf(k, u[j], S[i][j]) : fmaf(keep, S[i][j], kv);
+          if (!WKV) o[j] = fmaf(S[i][j], q, o[j]);
         }
       }
       const float r = warp_sum4(o);
@@ -120,23 +129,25 @@ __global__ void __launch_bounds__(256) recurrent_scan_kernel(const ScanArgs a) {
 }
 
 template <int RPL>
-int launch_scan(const ScanArgs& a, bool delta, cudaStream_t s) {
+int launch_scan(const ScanArgs& a, Recurrence kind, cudaStream_t s) {
   const dim3 grid((a.vdim + 31) / 32, a.H);
-  const cudaError_t e = delta ? launch_pdl(recurrent_scan_kernel<RPL, true>, grid, dim3(256), 0, s, a)
-                              : launch_pdl(recurrent_scan_kernel<RPL, false>, grid, dim3(256), 0, s, a);
+  auto* kernel = kind == Recurrence::kDelta ? recurrent_scan_kernel<RPL, Recurrence::kDelta>
+                 : kind == Recurrence::kWkv ? recurrent_scan_kernel<RPL, Recurrence::kWkv>
+                                            : recurrent_scan_kernel<RPL, Recurrence::kLightning>;
+  const cudaError_t e = launch_pdl(kernel, grid, dim3(256), 0, s, a);
   if (e != cudaSuccess) return fail(CTDK_ELAUNCH, "recurrent scan: %s", cudaGetErrorString(e));
   return check_launch("recurrent scan");
 }
 
 }  // namespace
 
-int recurrent_scan(const ScanArgs& a, bool delta, cudaStream_t s) {
+int recurrent_scan(const ScanArgs& a, Recurrence kind, cudaStream_t s) {
   CTDK_REQUIRE(a.dim >= 1 && a.dim <= 256 && a.H <= 65535, "recurrent scan: key size must be at most 256");
-  if (a.dim <= 32) return launch_scan<1>(a, delta, s);
-  if (a.dim <= 64) return launch_scan<2>(a, delta, s);
-  if (a.dim <= 96) return launch_scan<3>(a, delta, s);
-  if (a.dim <= 128) return launch_scan<4>(a, delta, s);
-  return launch_scan<8>(a, delta, s);
+  if (a.dim <= 32) return launch_scan<1>(a, kind, s);
+  if (a.dim <= 64) return launch_scan<2>(a, kind, s);
+  if (a.dim <= 96) return launch_scan<3>(a, kind, s);
+  if (a.dim <= 128) return launch_scan<4>(a, kind, s);
+  return launch_scan<8>(a, kind, s);
 }
 
 }  // namespace hybrid
