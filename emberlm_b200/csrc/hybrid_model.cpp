@@ -235,7 +235,9 @@ void place_rest(Branch& b, Layout& lay, const std::string& p, int width) {
   } else if (b.kind == BranchKind::kLatent) {
     b.q_norm = lay.vec(p + "dq.norm", b.q_rank);
     b.kv_norm = lay.vec(p + "dkv.norm", b.kv_rank);
-    b.w_uq = lay.matrix(p + "uq", static_cast<int64_t>(b.heads) * (b.dim + b.rot_dim), b.q_rank);
+    lay.begin_stack(b.q_rank);   // alone in its stack: a product takes whole groups of eight rows
+    lay.stacked(p + "uq", static_cast<int64_t>(b.heads) * (b.dim + b.rot_dim));
+    lay.end_stack(&b.w_uq);
     b.ld_uq = pad8(b.q_rank);
     lay.begin_stack(b.kv_rank);
     lay.stacked(p + "uk", static_cast<int64_t>(b.heads) * b.dim);
@@ -245,7 +247,9 @@ void place_rest(Branch& b, Layout& lay, const std::string& p, int width) {
   } else if (b.kind == BranchKind::kWkv) {
     const char* names[Branch::kMixes] = {"r", "k", "v", "g", "w"};
     for (int i = 0; i < Branch::kMixes; ++i) b.mu[i] = lay.vec(p + "mu." + names[i], width);
-    b.w_w2 = lay.matrix(p + "w2", static_cast<int64_t>(b.heads) * b.dim, b.rank_w);
+    lay.begin_stack(b.rank_w);
+    lay.stacked(p + "w2", static_cast<int64_t>(b.heads) * b.dim);
+    lay.end_stack(&b.w_w2);
     b.ld_w2 = pad8(b.rank_w);
     b.w0 = lay.vec(p + "w0", static_cast<int64_t>(b.heads) * b.dim);
     b.bonus = lay.table(p + "u", b.heads, b.dim);

@@ -417,7 +417,7 @@ int HybridDecoder<T>::mixer_latent(const Layer& L, const BranchBuffers& bb, int6
   a.out = mixed;
   a.ld_out = b.ld_o;
   DTRY(latent_prep(a, pos, n, s));
-  DTRY(gemm_rows(low_q, at<T>(b.w_uq), q_up, n, static_cast<int64_t>(b.heads) * (b.dim + b.rot_dim), b.q_rank, b.ld_uq, b.ld_uq, a.ld_up, s));
+  DTRY(gemm_rows(low_q, at<T>(b.w_uq), q_up, n, a.ld_up, b.q_rank, b.ld_uq, b.ld_uq, a.ld_up, s));
   DTRY(latent_rotate(a, pos, n, s));
   // keys and values of every position so far, out of the cached latents
   DTRY(kv_rows(a.cache, at<T>(b.w_ukv), pos + n, b.n_ukv, b.kv_rank, a.ld_cache, b.ld_ukv, s));
@@ -434,7 +434,7 @@ int HybridDecoder<T>::mixer_wkv(const Layer& L, const BranchBuffers& bb, int64_t
     DTRY(gemm_rows(mixes + i * n * m.ldw, at<T>(L.w_in) + static_cast<int64_t>(b.col_mix[i]) * m.ldw, proj + b.col_mix[i], n,
                    i < 4 ? pad8(cols) : pad8(b.rank_w), m.width, m.ldw, m.ldw, ldp, s));
   DTRY(tanh_rows(proj + b.col_mix[4], ldp, low_a, b.ld_w2, n, b.rank_w, s));
-  DTRY(gemm_rows(low_a, at<T>(b.w_w2), dz, n, cols, b.rank_w, b.ld_w2, b.ld_w2, ldz, s));
+  DTRY(gemm_rows(low_a, at<T>(b.w_w2), dz, n, ldz, b.rank_w, b.ld_w2, b.ld_w2, ldz, s));
   ScanArgs a;
   a.q = proj + b.col_mix[0];
   a.k = proj + b.col_mix[1];

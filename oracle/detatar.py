@@ -120,6 +120,20 @@ def route(z, correction, top, groups=None):
     return chosen, s[chosen] / (s[chosen].sum() + 1e-20)
 
 
+def route_margin(z, correction, top, groups=None):
+    """How close the choice is: the smallest gap between a taken and a refused choice score, groups included."""
+    s = np.exp(z - z.max())
+    choice = s / s.sum() + correction
+    gap = np.inf
+    if groups and groups["keep"] < groups["count"]:
+        best = -np.sort(-choice.reshape(groups["count"], -1).max(axis=1))
+        gap = best[groups["keep"] - 1] - best[groups["keep"]]
+        kept = np.argsort(-choice.reshape(groups["count"], -1).max(axis=1), kind="stable")[:groups["keep"]]
+        choice = choice.reshape(groups["count"], -1)[kept].ravel()
+    choice = -np.sort(-choice)
+    return min(gap, choice[top - 1] - choice[top]) if top < len(choice) else gap
+
+
 def moe(h, w, p, f):
     r = f["router"]
     out = np.zeros_like(h)
