@@ -378,6 +378,7 @@ int HybridDecoder<float>::latent_attention(const LatentArgs<float>& a, int64_t p
 }
 template <>
 int HybridDecoder<__nv_bfloat16>::latent_attention(const LatentArgs<__nv_bfloat16>& a, int64_t pos, int64_t n, cudaStream_t s) {
+  if (latent_tcgen05_ok(a.dim, a.rot_dim, a.vdim)) return latent_attention_tcgen05(a, pos, n, s);
   return latent_attention_fp32(a, pos, n, s);
 }
 
