@@ -83,7 +83,8 @@ def build(force: bool = False, verbose: bool = False) -> Path:
 # Sources that serving a layer-list model needs (no training-path kernels).
 LAYER_LIST_SOURCES = ["runtime.cu", "gemm.cu", "gemm_tcgen05.cu", "gemm_tcgen05_2cta.cu", "attention_tc.cu", "decode_api.cu",
                       "hybrid.cu", "hybrid_model.cpp", "hybrid_parallel.cu", "hybrid_prefill.cu", "hybrid_token.cu", "delta_chunk.cu",
-                      "latent_attention.cu", "latent_attention_tc.cu", "lightning_chunk.cu", "moe.cu", "parallel_rows.cu", "recurrent_scan.cu"]
+                      "latent_attention.cu", "latent_attention_tc.cu", "lightning_chunk.cu", "moe.cu", "parallel_rows.cu", "recurrent_scan.cu",
+                      "wkv_chunk.cu"]
 
 
 def build_trace_tool(family: str) -> Path:

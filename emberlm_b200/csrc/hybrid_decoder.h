@@ -82,6 +82,8 @@ struct HybridDecoder : DecoderBase {
 
   bool chunked_lightning(const Branch& b) const { return m.dtype == CTDK_DTYPE_BF16 && lightning_chunked_ok(b.dim, b.vdim); }
 
+  bool chunked_wkv(const Branch& b) const { return m.dtype == CTDK_DTYPE_BF16 && wkv_chunked_ok(b.dim); }
+
   int carve(Bump& b);
   int build_phases();
   int upload(cudaStream_t s);

@@ -19,7 +19,7 @@ int HybridDecoder<T>::carve_parallel(Bump& b) {
   const int64_t R = max_portion, W = m.width, n_layers = static_cast<int64_t>(m.layers.size());
   const bool exact = m.dtype == CTDK_DTYPE_F32;
   int64_t n_in = 8, n_side = 8, heads_out = 8, low = 8, q_up_n = 0, q_rot_n = 0, kv_n = 0, act_n = 8, dz_n = 0, o_n = 0, parts = 0, abs_n = 0;
-  int64_t low_w = 8, choices = 0, counts = 0, tiles = 0, slots = 0, gu_n = 0, ea_n = 0, tegu_n = 0;
+  int64_t low_w = 8, chunk_n = 0, decay_n = 0, choices = 0, counts = 0, tiles = 0, slots = 0, gu_n = 0, ea_n = 0, tegu_n = 0;
   bool mix = false, shared = false;
   bufs.assign(m.layers.size(), {});
   ropes.clear();
@@ -58,6 +58,11 @@ int HybridDecoder<T>::carve_parallel(Bump& b) {
       dz_n = std::max<int64_t>(dz_n, pad8(out_n));
       o_n = std::max<int64_t>(o_n, out_n);
       low_w = std::max<int64_t>(low_w, br.ld_w2);
+      if (chunked_wkv(br)) {
+        const int64_t tiles_n = (R + kWkvChunk - 1) / kWkvChunk * br.heads, d = wkv_tile(br.dim);
+        chunk_n = std::max(chunk_n, tiles_n * d * d);
+        decay_n = std::max(decay_n, tiles_n * d);
+      }
     }
     bufs[l].push_back(bb);
     if (L.ffn == FeedForward::kGeluGlu) act_n = std::max<int64_t>(act_n, L.ffp);
@@ -92,6 +97,8 @@ int HybridDecoder<T>::carve_parallel(Bump& b) {
   o32 = b.floats(R * o_n);
   dz = b.floats(R * dz_n);
   low_a = typed(R * low_w);
+  chunk_state = b.floats(chunk_n);
+  cdecay = b.floats(decay_n);
   low_q = typed(R * low);
   q_up = b.floats(R * q_up_n);
   q_rot = typed(R * q_rot_n);
@@ -436,6 +443,31 @@ int HybridDecoder<T>::mixer_wkv(const Layer& L, const BranchBuffers& bb, int64_t
                    i < 4 ? pad8(cols) : pad8(b.rank_w), m.width, m.ldw, m.ldw, ldp, s));
   DTRY(tanh_rows(proj + b.col_mix[4], ldp, low_a, b.ld_w2, n, b.rank_w, s));
   DTRY(gemm_rows(low_a, at<T>(b.w_w2), dz, n, ldz, b.rank_w, b.ld_w2, b.ld_w2, ldz, s));
+  if (chunked_wkv(b) && n >= kChunkedRows) {
+    WkvArgs c;
+    c.r = proj + b.col_mix[0];
+    c.k = proj + b.col_mix[1];
+    c.v = proj + b.col_mix[2];
+    c.gate = proj + b.col_mix[3];
+    c.ldp = ldp;
+    c.z = dz;
+    c.ldz = ldz;
+    c.w0 = vec(b.w0);
+    c.bonus = vec(b.bonus);
+    c.w_norm = vec(b.w_norm);
+    c.state = bb.state;
+    c.chunk_state = chunk_state;
+    c.decay = cdecay;
+    c.out = reinterpret_cast<__nv_bfloat16*>(mixed);   // chunked_wkv: the model's type
+    c.ld_out = b.ld_o;
+    c.H = b.heads;
+    c.dim = b.dim;
+    c.eps = m.eps;
+    c.rows = n;
+    c.resume = pos > 0;
+    DTRY(wkv_chunked(c, s));
+    return gemm_rows(mixed, at<T>(b.w_o), y1, n, m.width, cols, b.ld_o, b.ld_o, m.width, s);
+  }
   ScanArgs a;
   a.q = proj + b.col_mix[0];
   a.k = proj + b.col_mix[1];

@@ -95,6 +95,26 @@ int cast_rows(const float* src, int64_t lds, T* dst, int64_t ldd, int64_t rows, 
 // dst[t][c] = tanh(src[t][c]), zero up to ldd
 template <typename T>
 int tanh_rows(const float* src, int64_t lds, T* dst, int64_t ldd, int64_t rows, int n, cudaStream_t s);
+// Chunk-parallel form for bfloat16 models (wkv_chunk.cu), up to the gated norm: r, k, v, gate are columns of
+// the projection, decays e^(-e^(z + w0)). Scratch, with d = wkv_tile(dim): chunk_state [chunks][H][d][d],
+// decay [chunks][H][d].
+constexpr int kWkvChunk = 64;
+struct WkvArgs {
+  const float *r = nullptr, *k = nullptr, *v = nullptr, *gate = nullptr;
+  int64_t ldp = 0;
+  const float *z = nullptr, *w0 = nullptr, *bonus = nullptr, *w_norm = nullptr;
+  int64_t ldz = 0;
+  float *state = nullptr, *chunk_state = nullptr, *decay = nullptr;
+  __nv_bfloat16* out = nullptr;
+  int64_t ld_out = 0;
+  int H = 0, dim = 0;
+  float eps = 0.0f;
+  int64_t rows = 0;
+  int resume = 0;
+};
+inline int wkv_tile(int dim) { return dim <= 64 ? 64 : 128; }
+bool wkv_chunked_ok(int dim);
+int wkv_chunked(const WkvArgs& a, cudaStream_t s);
 // per head: rms over dim, * w[head * dim ..] * silu(gate)
 template <typename T>
 int silu_head_norm_rows(const float* o, const float* w, const float* gate, int64_t ldg, T* dst, int64_t ld, int64_t rows, int H, int dim,

@@ -69,7 +69,9 @@ FFS = [dc.dense(150), dc.dense(9), dc.dense(256), dc.moe(5, 2, 36), dc.moe(8, 8,
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("case", range(len(MIXERS)))
 def test_each_mixer_alone(case, dtype):
-    cfg = dc.model(50, 72, [dict(MIXERS[case], mlp=dc.dense(8))], groups=[1, 2, 9][case % 3])
+    # a norm over a single column is its sign: the large eps keeps it from magnifying rounding
+    eps = 1e-1 if MIXERS[case]["mixer"]["dim"] == 1 else 1e-5
+    cfg = dc.model(50, 72, [dict(MIXERS[case], mlp=dc.dense(8))], groups=[1, 2, 9][case % 3], eps=eps)
     w = close(dc.weights(cfg, 10 + case, rank=[9, 32, 64][case % 3]), "rg2")
     t = hc.tokens(cfg, 150, case)
     dec = decoder(cfg, w, dtype)
@@ -223,7 +225,7 @@ def test_far_memory_of_the_recurrence_is_carried(dtype):
 def test_time_mixing_with_strong_and_weak_decays(w0, bonus, dtype):
     """Decays that wipe a channel within a token (e^-148) or hardly move it: nothing overflows. The large eps
     keeps heads whose output is small from magnifying their own rounding."""
-    cfg = dc.model(40, 48, [dc.wkv(2, 64), dc.wkv(1, 20), dc.wkv(1, 128)], eps=1e-2)
+    cfg = dc.model(40, 48, [dc.wkv(2, 64), dc.wkv(1, 20), dc.wkv(1, 128)], eps=0.3)
     w = dc.weights(cfg, 81)
     for i in range(3):
         w[f"l{i}.mix.w0"] = hc.bf16(w[f"l{i}.mix.w0"] * 0.3 + w0)
