@@ -500,22 +500,24 @@ def run_decode(args) -> dict:
 
 
 def run_serving(args) -> dict:
-    """Prefill and greedy decode, batch 1, of the layer-list design Zutalix in bfloat16 beside the preset
-    decoder closest to it at equal width, depth, feed-forward width and vocabulary (random weights). A
-    "step" is one prompt of 4096 tokens plus 128 greedy tokens; value = prompt tokens/s of the larger
-    Zutalix; `models` holds every figure."""
+    """Prefill and greedy decode, batch 1, of a layer-list design (Zutalix, Detatar) in bfloat16 beside the
+    preset decoder closest to it (and Detatar beside Zutalix) at equal width, depth, active feed-forward width
+    and vocabulary (random weights). A "step" is one prompt of 4096 tokens plus 128 greedy tokens; value =
+    prompt tokens/s of the design's larger size; `models` holds every figure."""
+    design = args.workload.removesuffix("_serving")
+    models = ("zutalix", "preset") if design == "zutalix" else (design, "zutalix", "preset")
     from emberlm_b200 import serve_bench
     import torch
     torch.cuda.set_device(0)
     rows = []
     for size in sorted(serve_bench.SIZES):
-        rows += serve_bench.run(size, steps=args.steps, warmup=max(args.warmup, 3), sampler=lambda: ClockSampler(0))
-    main_row = next(r for r in reversed(rows) if r["model"].startswith("zutalix"))
+        rows += serve_bench.run(size, steps=args.steps, warmup=max(args.warmup, 3), models=models, sampler=lambda: ClockSampler(0))
+    main_row = next(r for r in reversed(rows) if r["model"].startswith(design))
     return {"metric": "prefill tokens/s (batch 1, 4096-token prompt)", "value": main_row["prefill_tokens_per_s"], "unit": "tokens/s",
             "n_gpus": 1, "steps": args.steps, "warmup": max(args.warmup, 3),
             "ms_per_step": main_row["prefill_ms"] + main_row["token_ms"] * main_row["new_tokens"], "higher_is_better": True,
             "scaling": "replicas only", "vs_baseline": None, "dtype": "bf16", "data": "synthetic", "impl": "ours",
-            "config": {"workload": "zutalix_serving", "model": main_row["model"], "prompt_len": main_row["prompt_len"],
+            "config": {"workload": args.workload, "model": main_row["model"], "prompt_len": main_row["prompt_len"],
                        "new_tokens": main_row["new_tokens"], "l2": "weights larger than L2"},
             "clocks": main_row["clocks"], "gpu_launches": main_row["gpu_launches"], "models": rows}
 
@@ -593,7 +595,7 @@ def main():
     ap.add_argument("--steps", type=int, default=10)
     ap.add_argument("--warmup", type=int, default=3)
     ap.add_argument("--impl", choices=["ours", "reference"], default="ours")
-    ap.add_argument("--workload", choices=sorted(WORKLOADS) + ["qwen3_0_6b_decode", "zutalix_serving"], default=DEFAULT_WORKLOAD)
+    ap.add_argument("--workload", choices=sorted(WORKLOADS) + ["qwen3_0_6b_decode", "zutalix_serving", "detatar_serving"], default=DEFAULT_WORKLOAD)
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--precision", choices=["tf32", "3xtf32"], default="tf32",
                     help="3xtf32: every contraction splits its operands into TF32 high and low parts (near-fp32 results)")
@@ -603,7 +605,7 @@ def main():
     args = ap.parse_args()
     if args.warmup < 3 and args.impl == "ours":
         print(f"note: --warmup {args.warmup} < 3; timing rules ask for at least 3", file=sys.stderr)
-    if args.workload == "zutalix_serving":
+    if args.workload.endswith("_serving"):
         out = run_serving(args) if args.impl == "ours" else {"impl": "reference", "unavailable": "the reference has no such model"}
     elif args.workload == "qwen3_0_6b_decode":
         out = run_decode(args) if args.impl == "ours" else run_decode_reference(args)

@@ -39,7 +39,7 @@ int HybridDecoder<T>::carve_parallel(Bump& b) {
       q_up_n = std::max<int64_t>(q_up_n, pad8(static_cast<int64_t>(br.heads) * (br.dim + br.rot_dim)));
       q_rot_n = std::max<int64_t>(q_rot_n, static_cast<int64_t>(br.heads) * latent_q_pitch(br.dim, br.rot_dim));
       kv_n = std::max<int64_t>(kv_n, br.n_ukv);
-      parts = std::max<int64_t>(parts, static_cast<int64_t>(br.heads) * kLatentSplits * (bb.n_latent_rot + kAttnStats));
+      parts = std::max<int64_t>(parts, static_cast<int64_t>(br.heads) * kLatentSplits * (bb.n_latent_rot + kAttnStats4));
       abs_n = std::max<int64_t>(abs_n, br.heads * bb.ld_latent);
       for (size_t i = 0; i < ropes.size() && bb.rope < 0; ++i)
         if (ropes[i].spec == br.rope) bb.rope = static_cast<int>(i);
@@ -148,7 +148,7 @@ int HybridDecoder<T>::build_parallel_phases() {
   phases.clear();
   stage_floats = 0;
   const int ldw = static_cast<int>(m.ldw), W = m.width;
-  const int wpg = m.norm_groups >= 8 ? 1 : 8 / m.norm_groups;
+  const int wpg = m.norm_groups >= kListWarps ? 1 : kListWarps / m.norm_groups;
   int cur = 0;
   auto need = [&](int64_t floats) { stage_floats = std::max<int>(stage_floats, static_cast<int>(floats)); };
   auto list = [&] {
@@ -160,7 +160,7 @@ int HybridDecoder<T>::build_parallel_phases() {
   auto add_op = [&](TokenPhase& p, int kind, int64_t at, int64_t n, int64_t ld, const float* src, const float* src2 = nullptr,
                     const float* w = nullptr) {
     p.op[p.n_ops++] = StageOp{kind, static_cast<int>(at), static_cast<int>(n), static_cast<int>(ld), src, src2, w};
-    need(at + (kind == kOpRoute ? n + route_scratch(static_cast<int>(n), p.route_groups) : std::max(n, ld)));
+    need(at + (kind == kOpRoute ? ld + n + route_scratch(static_cast<int>(n), p.route_groups) : std::max(n, ld)));
   };
   auto add_gemv = [&](TokenPhase& p, const T* w, float* y, int64_t rows, int64_t K, int64_t in) -> TokenGemv& {
     TokenGemv g{};
@@ -178,6 +178,7 @@ int HybridDecoder<T>::build_parallel_phases() {
     TokenShift& f = p.shift;
     f.groups = m.norm_groups;
     f.wpg = wpg;
+    f.vec = W % (4 * m.norm_groups) == 0 ? 1 : 0;
     f.ld = ldw;
     f.w = vec(w);
     if (l > 0) {
@@ -249,7 +250,8 @@ int HybridDecoder<T>::build_parallel_phases() {
       t.kv_norm = vec(br.kv_norm);
       t.q_up = tq;
       t.q_abs = tq_abs;
-      t.blocks = (br.heads + kLatentHeads - 1) / kLatentHeads;
+      const int hb = sizeof(T) == 2 ? kLatentHeads : kLatentHeadsF32;
+      t.blocks = (br.heads + hb - 1) / hb;
       t.splits = std::min(kLatentSplits, std::max(8, 2 * sm_count() / t.blocks));
     } else {
       t.kind = kTokWkv;
@@ -264,13 +266,12 @@ int HybridDecoder<T>::build_parallel_phases() {
       t.w0 = vec(br.w0);
       t.bonus = vec(br.bonus);
     }
-    // what the experts stage: the choice and h
+    // the choice, and h for the chosen experts
     auto expert_up = [&](TokenPhase& q, int64_t offset) {
       q.route_groups = e.groups;
       q.route_keep = e.keep;
       q.route_top = e.top;
-      add_op(q, kOpRoute, offset, e.outputs(), 0, zs + L.col_router, nullptr, vec(e.correction));
-      add_op(q, kOpCopy, offset, W, ldw, th);   // over the scratch of the choice
+      add_op(q, kOpRoute, offset, e.outputs(), ldw, zs + L.col_router, th, vec(e.correction));
       TokenGemv& g = add_gemv(q, at<T>(e.w_gu), tegu, static_cast<int64_t>(e.top) * 2 * e.effp, ldw, offset);
       g.mode = kGemvExpertUp;
       g.per = g.pitch = 2 * e.effp;
@@ -313,30 +314,34 @@ int HybridDecoder<T>::build_parallel_phases() {
       const int64_t esize = static_cast<int64_t>(sizeof(T));
       TokenPhase q = list();   // queries; the position's cache row
       items(q, kTokLatentKeys, 0);
+      add_gemv(q, at<T>(br.w_uq), tq, static_cast<int64_t>(br.heads) * (br.dim + br.rot_dim), br.ld_uq, 0);
+      if (moe) expert_up(q, br.ld_uq);   // one warp chooses while the others go on
       add_op(q, kOpRmsNorm, 0, br.q_rank, br.ld_uq, tproj + br.col_q, nullptr, vec(br.q_norm));
       add_op(q, kOpLatentStore, 0, 0, 0, nullptr);
-      add_gemv(q, at<T>(br.w_uq), tq, static_cast<int64_t>(br.heads) * (br.dim + br.rot_dim), br.ld_uq, 0);
-      if (moe) expert_up(q, br.ld_uq);
       phases.push_back(q);
 
       const int key_cols = 16 * (16 / static_cast<int>(sizeof(T)));
       TokenPhase k = list();   // queries against the cache rows
       items(k, kTokLatentKeys, br.heads * ((t.rot_col + key_cols - 1) / key_cols));
       down(k, 0);
-      need(16 * (key_cols + 1));
+      need(kListThreads / 16 * (key_cols + 1));
       k.extra = at<T>(br.w_ukv);
       k.extra_bytes = static_cast<int64_t>(br.row_uv) * br.ld_ukv * esize;
       phases.push_back(k);
 
       TokenPhase sc = list();
       items(sc, kTokLatentScan, t.blocks * t.splits);
-      const int64_t chunks = t.ld_cache / (16 / esize);
-      need(kLatentHeads * (t.ld_cache + kLatentKeys + 1) + 4 * kLatentKeys * (chunks | 1));
+      const int64_t slices = (t.ld_cache + 15) / 16 * 16 + 8;   // bfloat16 pitch
+      const int64_t tile = sizeof(T) == 2 ? kLatentKeys * slices / 2 : 4 * kLatentKeys * (t.ld_cache / 4 | 1);
+      const int64_t queries = sizeof(T) == 2 ? kLatentHeads * (slices + kLatentKeys + 8 + 8 * (kLatentKeys + 4) + 1)
+                                             : kLatentHeadsF32 * (t.ld_cache + kLatentKeys + 1);
+      sc.br[0].buffers = 4 * (queries + 2 * tile) <= 190 * 1024 ? 2 : 1;
+      need(queries + sc.br[0].buffers * tile);
       phases.push_back(sc);
 
       TokenPhase v = list();
       items(v, kTokLatentOut, br.heads * ((br.vdim + kLatentOutRows - 1) / kLatentOutRows));
-      need(t.rot_col + t.splits);
+      need(t.rot_col * (1 + kLatentOutParts) + kLatentSplits);
       v.extra = at<T>(br.w_ukv) + static_cast<int64_t>(br.row_uv) * br.ld_ukv;
       v.extra_bytes = static_cast<int64_t>(br.heads) * br.vdim * br.ld_ukv * esize;
       phases.push_back(v);
@@ -348,7 +353,7 @@ int HybridDecoder<T>::build_parallel_phases() {
     } else {
       TokenPhase q = list();
       items(q, kTokWkv, t.items);
-      need(br.ld_w2 + 4 * br.dim + 8 * 32);
+      need(br.ld_w2 + 4 * br.dim + kListThreads);
       if (moe) expert_up(q, 0);
       phases.push_back(q);
 

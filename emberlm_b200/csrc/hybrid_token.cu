@@ -6,10 +6,12 @@
 // the weights of a coming phase are on their way into L2. Vectors between phases are fp32; every CTA
 // stages (and norms) its own copy. All waits are bounded.
 #include <cfloat>
+#include <type_traits>
 
 #include "decode_core.h"
 #include "hybrid_kernels.h"
 #include "hybrid_token.h"
+#include "mma_bf16.cuh"
 #include "moe_route.cuh"
 #include "parallel_kernels.h"
 
@@ -18,6 +20,7 @@ namespace hybrid {
 namespace {
 
 constexpr int kThreads = 256, kWarps = 8;
+constexpr int token_threads(bool list) { return list ? kListThreads : kThreads; }
 
 __device__ __forceinline__ float ldg_f(const float* p) { return __ldcg(p); }
 
@@ -69,9 +72,9 @@ struct Chunk<__nv_bfloat16> {
   }
 };
 
-// dot(W[row, part of K], xs) over a warp that owns the chunks part, part + WPR, ...: all lanes get the sum.
+// dot(W[row, part of K], xs) over a warp that owns the chunks part, part + WPR, ...: the lane's share of the sum.
 template <typename T>
-__device__ __forceinline__ float row_dot(const T* __restrict__ row, const float* xs, int K, int part, int wpr) {
+__device__ __forceinline__ float row_part(const T* __restrict__ row, const float* xs, int K, int part, int wpr) {
   constexpr int N = Chunk<T>::kN;
   const int lane = threadIdx.x & 31;
   const int n = K / N, step = 32 * wpr;
@@ -89,7 +92,12 @@ __device__ __forceinline__ float row_dot(const T* __restrict__ row, const float*
     c.load(row + static_cast<int64_t>(i) * N);
     acc = c.dot(xs + i * N, acc);
   }
-  return warp_sum(acc);
+  return acc;
+}
+// All lanes get the sum.
+template <typename T>
+__device__ __forceinline__ float row_dot(const T* __restrict__ row, const float* xs, int K, int part, int wpr) {
+  return warp_sum(row_part<T>(row, xs, K, part, wpr));
 }
 
 template <int N>
@@ -407,11 +415,16 @@ __device__ __forceinline__ float conv_channel(const TokenPhase& ph, const TokenB
 // dot of a low-rank row with a staged fp32 vector (rank rounded up to 8, both zero-padded)
 template <typename T>
 __device__ __forceinline__ float short_dot(const T* row, const float* x, int n) {
+  constexpr int N = Chunk<T>::kN, U = 4;   // chunks in flight
   float acc = 0.0f;
-  for (int i = 0; i < n; i += Chunk<T>::kN) {
-    Chunk<T> c;
-    c.load(row + i);
-    acc = c.dot(x + i, acc);
+  for (int i = 0; i < n; i += U * N) {
+    Chunk<T> c[U];
+#pragma unroll
+    for (int u = 0; u < U; ++u)
+      if (i + u * N < n) c[u].load(row + i + u * N);
+#pragma unroll
+    for (int u = 0; u < U; ++u)
+      if (i + u * N < n) acc = c[u].dot(x + i + u * N, acc);
   }
   return acc;
 }
@@ -492,6 +505,7 @@ __device__ void delta_item(const TokenPhase& ph, const TokenBranch& br, int item
 }
 
 // ---- parallel arrangement ----
+// One CTA per SM with twice the threads: what a phase stages is staged once per SM.
 
 // Experts of the token, chosen by every CTA for itself.
 struct Routed {
@@ -499,136 +513,303 @@ struct Routed {
   float weight[32];
 };
 
-// The staged rows of ShiftNormArgs for one token. A thread keeps to its own columns.
-template <typename T>
-__device__ void stage_shift_norm(const TokenArgs& a, const TokenPhase& ph, int64_t tok, int pos, float* sm) {
+// Items 0 .. n - 1 dealt to the threads, U loads of a thread in flight: put(i, load(i)).
+template <int U, typename Load, typename Put>
+__device__ __forceinline__ void batched(int n, int first, int threads, Load load, Put put) {
+  for (int i0 = first; i0 < n; i0 += U * threads) {
+    decltype(load(0)) v[U];
+#pragma unroll
+    for (int u = 0; u < U; ++u)
+      if (i0 + u * threads < n) v[u] = load(i0 + u * threads);
+#pragma unroll
+    for (int u = 0; u < U; ++u)
+      if (i0 + u * threads < n) put(i0 + u * threads, v[u]);
+  }
+}
+struct Pair4 {
+  float4 a, b;
+};
+__device__ __forceinline__ float4 ldg4(const float* p) { return __ldcg(reinterpret_cast<const float4*>(p)); }
+__device__ __forceinline__ float sq4(const float4& a) { return a.x * a.x + a.y * a.y + a.z * a.z + a.w * a.w; }
+
+// V neighbouring columns.
+template <int V>
+struct Cols {
+  float v[V];
+  __device__ __forceinline__ void load(const float* p) {   // of memory that other CTAs write
+    if constexpr (V == 4) {
+      const float4 f = ldg4(p);
+      v[0] = f.x;
+      v[1] = f.y;
+      v[2] = f.z;
+      v[3] = f.w;
+    } else {
+      v[0] = ldg_f(p);
+    }
+  }
+  template <typename U>
+  __device__ __forceinline__ void get(const U* p) {   // weights, shared memory
+    if constexpr (V == 4) {
+      const float4 f = load4(p);
+      v[0] = f.x;
+      v[1] = f.y;
+      v[2] = f.z;
+      v[3] = f.w;
+    } else {
+      v[0] = to_f(*p);
+    }
+  }
+  __device__ __forceinline__ void put(float* p) const {
+    if constexpr (V == 4) store4(p, make_float4(v[0], v[1], v[2], v[3]));
+    else *p = v[0];
+  }
+};
+
+// The staged rows of ShiftNormArgs for one token. A thread keeps to its own columns, which lie in one group
+// per turn; everything that does not depend on the norm is requested before it.
+template <typename T, int V>
+__device__ __forceinline__ void stage_shift_norm(const TokenArgs& a, const TokenPhase& ph, int64_t tok, int pos) {
+  extern __shared__ __align__(16) float sm[];
+  constexpr int U = V == 4 ? 1 : 2;   // turns in flight
   const TokenShift& f = ph.shift;
   const int W = a.width, gs = W / f.groups, lane = threadIdx.x & 31, wid = threadIdx.x >> 5;
-  const int g0 = wid / f.wpg, gstep = kWarps / f.wpg, wj = wid % f.wpg;
-  const bool active = g0 < gstep, writer = blockIdx.x == 0;
+  const int g0 = wid / f.wpg, gstep = kListWarps / f.wpg, wj = wid % f.wpg, step = 32 * V * f.wpg;
+  const bool active = g0 < gstep, writer = blockIdx.x == 0, shifted = f.shift != nullptr;
   const T* e = ph.first_token ? static_cast<const T*>(a.embed) + tok * a.ld_embed : nullptr;
   float *xs = sm, *part = sm + f.red;
-  __syncthreads();   // the scratch may still be read as part of an earlier phase
+  const float* prev = shifted ? f.state + ((pos + 1) & 1) * 2 * W : nullptr;
+  float* next = shifted ? f.state + (pos & 1) * 2 * W : nullptr;
   for (int g = g0; active && g < f.groups; g += gstep) {
     float ss = 0.0f;
-    for (int c = g * gs + wj * 32 + lane; c < (g + 1) * gs; c += 32 * f.wpg) {
-      float x;
-      if (e != nullptr) {
-        x = to_f(e[c]) * a.embed_scale;
-      } else {
-        x = ldg_f(f.y1 + c) * sigmoid_f(ldg_f(f.z1 + c) + f.b1[c]);
-        if (f.y2 != nullptr) x += ldg_f(f.y2 + c) * sigmoid_f(ldg_f(f.z2 + c) + f.b2[c]);
-        x += ldg_f(f.x + c);
+    const int end = (g + 1) * gs;
+    for (int c0 = g * gs + (wj * 32 + lane) * V; c0 < end; c0 += U * step) {
+      Cols<V> x[U], y1[U], z1[U], b1[U], y2[U], z2[U], b2[U];
+#pragma unroll
+      for (int u = 0; u < U; ++u) {
+        const int c = c0 + u * step;
+        if (c >= end) break;
+        if (e != nullptr) {
+          x[u].get(e + c);
+          continue;
+        }
+        x[u].load(f.x + c);
+        y1[u].load(f.y1 + c);
+        z1[u].load(f.z1 + c);
+        b1[u].get(f.b1 + c);
+        if (f.y2 != nullptr) {
+          y2[u].load(f.y2 + c);
+          z2[u].load(f.z2 + c);
+          b2[u].get(f.b2 + c);
+        }
       }
-      if (writer && f.x_out != nullptr) f.x_out[c] = x;
-      xs[c] = x;
-      ss += x * x;
+#pragma unroll
+      for (int u = 0; u < U; ++u) {
+        const int c = c0 + u * step;
+        if (c >= end) break;
+#pragma unroll
+        for (int k = 0; k < V; ++k) {
+          if (e != nullptr) {
+            x[u].v[k] *= a.embed_scale;
+          } else {
+            float r = y1[u].v[k] * sigmoid_f(z1[u].v[k] + b1[u].v[k]);
+            if (f.y2 != nullptr) r += y2[u].v[k] * sigmoid_f(z2[u].v[k] + b2[u].v[k]);
+            x[u].v[k] += r;
+          }
+          ss += x[u].v[k] * x[u].v[k];
+        }
+        x[u].put(xs + c);
+        if (writer && f.x_out != nullptr) x[u].put(f.x_out + c);
+      }
     }
     ss = warp_sum(ss);
     if (lane == 0) part[g * f.wpg + wj] = ss;
   }
+  // the first turns' weights and previous row are on their way over the barrier
+  Cols<V> w0[U], s0[U], p0[U];
+  auto request = [&](int c0, int end) {
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const int c = c0 + u * step;
+      if (c >= end) break;
+      w0[u].get(f.w + c);
+      if (!shifted) continue;
+      s0[u].get(f.shift + c);
+      if (pos > 0) p0[u].load(prev + c);
+    }
+  };
+  if (active && g0 < f.groups) request(g0 * gs + (wj * 32 + lane) * V, (g0 + 1) * gs);
   __syncthreads();
-  const float* prev = f.state != nullptr ? f.state + ((pos + 1) & 1) * 2 * W : nullptr;
-  float* next = f.state != nullptr ? f.state + (pos & 1) * 2 * W : nullptr;
   for (int g = g0; active && g < f.groups; g += gstep) {
     float ss = 0.0f;
     for (int k = 0; k < f.wpg; ++k) ss += part[g * f.wpg + k];
     const float sc = rsqrtf(ss / static_cast<float>(gs) + a.eps);
-    for (int c = g * gs + wj * 32 + lane; c < (g + 1) * gs; c += 32 * f.wpg) {
-      const float h = xs[c] * sc * f.w[c];
-      xs[c] = h;
-      if (f.shift == nullptr) continue;
-      const float m = fmaf((pos > 0 ? ldg_f(prev + c) : 0.0f) - h, f.shift[c], h);
-      sm[f.ld + c] = m;
-      if (writer) {
-        f.h_out[c] = h;
-        next[c] = h;
-        if (f.n_mix > 0) next[W + c] = m;
-      }
-      if (f.n_mix == 0) continue;
-      const float d = (pos > 0 ? ldg_f(prev + W + c) : 0.0f) - m;
+    const int begin = g * gs + (wj * 32 + lane) * V, end = (g + 1) * gs;
+    for (int c0 = begin; c0 < end; c0 += U * step) {
+      if (g != g0 || c0 != begin) request(c0, end);
 #pragma unroll
-      for (int i = 0; i < kTokenMixes; ++i) sm[(2 + i) * f.ld + c] = fmaf(d, f.mu[i][c], m);
+      for (int u = 0; u < U; ++u) {
+        const int c = c0 + u * step;
+        if (c >= end) break;
+        Cols<V> h, m, mu[kTokenMixes], pm;
+        if (f.n_mix > 0) {
+          if (pos > 0) pm.load(prev + W + c);
+#pragma unroll
+          for (int i = 0; i < kTokenMixes; ++i) mu[i].get(f.mu[i] + c);
+        }
+        h.get(xs + c);
+#pragma unroll
+        for (int k = 0; k < V; ++k) h.v[k] *= sc * w0[u].v[k];
+        h.put(xs + c);
+        if (!shifted) continue;
+#pragma unroll
+        for (int k = 0; k < V; ++k) m.v[k] = fmaf((pos > 0 ? p0[u].v[k] : 0.0f) - h.v[k], s0[u].v[k], h.v[k]);
+        m.put(sm + f.ld + c);
+        if (writer) {
+          h.put(f.h_out + c);
+          h.put(next + c);
+          if (f.n_mix > 0) m.put(next + W + c);
+        }
+        if (f.n_mix == 0) continue;
+#pragma unroll
+        for (int i = 0; i < kTokenMixes; ++i) {
+          Cols<V> o;
+#pragma unroll
+          for (int k = 0; k < V; ++k) o.v[k] = fmaf((pos > 0 ? pm.v[k] : 0.0f) - m.v[k], mu[i].v[k], m.v[k]);
+          o.put(sm + (2 + i) * f.ld + c);
+        }
+      }
     }
   }
-  const int rows = f.shift == nullptr ? 1 : 2 + f.n_mix, pad = f.ld - W;
-  for (int i = threadIdx.x; i < rows * pad; i += kThreads) sm[i / pad * f.ld + W + i % pad] = 0.0f;
+  const int rows = shifted ? 2 + f.n_mix : 1, pad = f.ld - W;
+  for (int i = threadIdx.x; i < rows * pad; i += kListThreads) sm[i / pad * f.ld + W + i % pad] = 0.0f;
   __syncthreads();
 }
 
 template <typename T>
-__device__ void stage_list(const TokenArgs& a, const TokenPhase& ph, int64_t tok, int pos, float* sm, float* red, Routed& routed) {
+__device__ __noinline__ void stage_list(const TokenArgs& a, const TokenPhase& ph, int64_t tok, int pos, float* red, Routed& routed) {
+  extern __shared__ __align__(16) float sm[];
   const int lane = threadIdx.x & 31, wid = threadIdx.x >> 5;
   for (int i = 0; i < ph.n_ops; ++i) {
     const StageOp& op = ph.op[i];
     float* xs = sm + op.at;
     if (op.kind == kOpShiftNorm) {
-      stage_shift_norm<T>(a, ph, tok, pos, sm);
+      if (ph.shift.vec) stage_shift_norm<T, 4>(a, ph, tok, pos);
+      else stage_shift_norm<T, 1>(a, ph, tok, pos);
     } else if (op.kind == kOpRmsNorm) {
-      float ss[1] = {0.0f};
-      for (int c = threadIdx.x; c < op.n; c += kThreads) {
-        const float v = ldg_f(op.src + c);
-        xs[c] = v;
-        ss[0] += v * v;
-      }
-      block_sum<1>(ss, red);
-      const float sc = rsqrtf(ss[0] / static_cast<float>(op.n) + a.eps);
-      for (int c = threadIdx.x; c < op.ld; c += kThreads) xs[c] = c < op.n ? xs[c] * sc * op.w[c] : 0.0f;
-    } else if (op.kind == kOpCopy) {
-      for (int c = threadIdx.x; c < op.ld; c += kThreads) xs[c] = c < op.n ? ldg_f(op.src + c) : 0.0f;
-    } else if (op.kind == kOpRoute) {
-      if (wid == 0) {   // logits, then the scratch of the choice, at `at`
-        for (int c = lane; c < op.n; c += 32) xs[c] = ldg_f(op.src + c);
-        __syncwarp();
-        route_token(xs, op.w, op.n, ph.route_groups, ph.route_keep, ph.route_top, xs + op.n, routed.index, routed.weight);
-      }
-      __syncthreads();
-    } else if (op.kind == kOpGelu) {
-      for (int c = threadIdx.x; c < op.n; c += kThreads) xs[c] = gelu_tanh_f(ldg_f(op.src + c)) * ldg_f(op.src + op.ld + c);
-    } else if (op.kind == kOpShared) {
-      const float g = sigmoid_f(ldg_f(op.src2));
-      for (int c = threadIdx.x; c < op.n; c += kThreads) xs[c] = g * silu_f(ldg_f(op.src + c)) * ldg_f(op.src + op.ld + c);
-    } else if (op.kind == kOpExperts) {
-      const int n = op.n;
-      for (int c = threadIdx.x; c < ph.route_top * n; c += kThreads) {
-        const int k = c / n;
-        const float* g = op.src + 2 * k * n + c % n;
-        xs[c] = routed.index[k] < op.ld ? routed.weight[k] * silu_f(ldg_f(g)) * ldg_f(g + n) : 0.0f;   // ld: number of experts
-      }
-    } else if (op.kind == kOpHeadNorm) {
-      const TokenBranch& br = ph.br[0];
-      for (int h = wid; h < br.H; h += kWarps) {
-        const float* o = op.src + h * br.dim;
+      // every warp that takes part forms the sum by itself and stores its share: no barrier
+      const int n4 = op.n >> 2, w0 = ph.route_top > 0 ? 1 : 0, parts = kListWarps - w0;
+      if (wid >= w0) {
+        constexpr int U = 8;   // 1024 columns at once
         float ss = 0.0f;
-        for (int d = lane; d < br.dim; d += 32) {
-          const float v = ldg_f(o + d);
+        for (int c = (op.n & ~3) + lane; c < op.n; c += 32) {
+          const float v = ldg_f(op.src + c);
           ss += v * v;
         }
-        const float sc = rsqrtf(warp_sum(ss) / static_cast<float>(br.dim) + a.eps);
-        for (int d = lane; d < br.dim; d += 32) {
-          const int c = h * br.dim + d;
-          xs[c] = ldg_f(o + d) * sc * op.w[c] * silu_f(ldg_f(op.src2 + c));
+        for (int c0 = lane; c0 < n4; c0 += 32 * U) {
+          float4 v[U];
+#pragma unroll
+          for (int u = 0; u < U; ++u) v[u] = c0 + 32 * u < n4 ? ldg4(op.src + 4 * (c0 + 32 * u)) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+          for (int u = 0; u < U; ++u) ss += sq4(v[u]);
         }
+        const float sc = rsqrtf(warp_sum(ss) / static_cast<float>(op.n) + a.eps);
+        for (int c = (wid - w0) * 32 + lane; c < n4; c += 32 * parts) {
+          const float4 v = ldg4(op.src + 4 * c), w = load4(op.w + 4 * c);
+          store4(xs + 4 * c, make_float4(v.x * sc * w.x, v.y * sc * w.y, v.z * sc * w.z, v.w * sc * w.w));
+        }
+        if (wid == w0)
+          for (int c = (op.n & ~3) + lane; c < op.ld; c += 32) xs[c] = c < op.n ? ldg_f(op.src + c) * sc * op.w[c] : 0.0f;
       }
-      for (int c = op.n + threadIdx.x; c < op.ld; c += kThreads) xs[c] = 0.0f;
-    } else if (blockIdx.x == gridDim.x - 1) {   // kOpLatentStore
+    } else if (op.kind == kOpCopy) {
+      batched<1>(op.n >> 2, threadIdx.x, kListThreads, [&](int c) { return ldg4(op.src + 4 * c); }, [&](int c, const float4& v) { store4(xs + 4 * c, v); });
+      for (int c = (op.n & ~3) + threadIdx.x; c < op.ld; c += kListThreads) xs[c] = c < op.n ? ldg_f(op.src + c) : 0.0f;
+    } else if (op.kind == kOpRoute) {
+      // one warp chooses (logits and scratch behind the copy), the others copy src2 to `at`
+      float* z = xs + op.ld;
+      if (wid == 0) {
+        for (int c = lane; c < op.n; c += 32) z[c] = ldg_f(op.src + c);
+        __syncwarp();
+        route_token(z, op.w, op.n, ph.route_groups, ph.route_keep, ph.route_top, z + op.n, routed.index, routed.weight);
+      } else {
+        const int W = a.width, t = threadIdx.x - 32, threads = kListThreads - 32;
+        batched<2>(W >> 2, t, threads, [&](int c) { return ldg4(op.src2 + 4 * c); }, [&](int c, const float4& v) { store4(xs + 4 * c, v); });
+        for (int c = (W & ~3) + t; c < op.ld; c += threads) xs[c] = c < W ? ldg_f(op.src2 + c) : 0.0f;
+      }
+    } else if (op.kind == kOpGelu) {
+      batched<1>(op.n >> 2, threadIdx.x, kListThreads, [&](int c) { return Pair4{ldg4(op.src + 4 * c), ldg4(op.src + op.ld + 4 * c)}; },
+                 [&](int c, const Pair4& v) {
+                   store4(xs + 4 * c, make_float4(gelu_tanh_f(v.a.x) * v.b.x, gelu_tanh_f(v.a.y) * v.b.y, gelu_tanh_f(v.a.z) * v.b.z,
+                                                  gelu_tanh_f(v.a.w) * v.b.w));
+                 });
+    } else if (op.kind == kOpShared) {
+      const float g = sigmoid_f(ldg_f(op.src2));
+      batched<1>(op.n >> 2, threadIdx.x, kListThreads, [&](int c) { return Pair4{ldg4(op.src + 4 * c), ldg4(op.src + op.ld + 4 * c)}; },
+                 [&](int c, const Pair4& v) {
+                   store4(xs + 4 * c, make_float4(g * silu_f(v.a.x) * v.b.x, g * silu_f(v.a.y) * v.b.y, g * silu_f(v.a.z) * v.b.z,
+                                                  g * silu_f(v.a.w) * v.b.w));
+                 });
+    } else if (op.kind == kOpExperts) {
+      const int n4 = op.n >> 2;   // ld: number of experts; an identity output's columns are not read
+      batched<2>(ph.route_top * n4, threadIdx.x, kListThreads,
+                 [&](int c) {
+                   const float* g = op.src + 8 * (c / n4) * n4 + 4 * (c % n4);
+                   return Pair4{ldg4(g), ldg4(g + 4 * n4)};
+                 },
+                 [&](int c, const Pair4& v) {
+                   const float w = routed.index[c / n4] < op.ld ? routed.weight[c / n4] : 0.0f;
+                   store4(xs + 4 * c, make_float4(w * silu_f(v.a.x) * v.b.x, w * silu_f(v.a.y) * v.b.y, w * silu_f(v.a.z) * v.b.z,
+                                                  w * silu_f(v.a.w) * v.b.w));
+                 });
+    } else if (op.kind == kOpHeadNorm) {
+      const TokenBranch& br = ph.br[0];
+      auto heads = [&](auto per_lane, auto at_once) {   // dim <= 32 per_lane; at_once heads in flight
+        constexpr int E = decltype(per_lane)::value, B = decltype(at_once)::value;
+        for (int h0 = wid; h0 < br.H; h0 += B * kListWarps) {
+          float o[B][E], x[B][E], w[B][E];
+#pragma unroll
+          for (int j = 0; j < B; ++j)
+#pragma unroll
+            for (int u = 0; u < E; ++u) {
+              const int h = h0 + j * kListWarps, d = lane + 32 * u, c = h * br.dim + d;
+              const bool in = h < br.H && d < br.dim;
+              o[j][u] = in ? ldg_f(op.src + c) : 0.0f;
+              x[j][u] = in ? ldg_f(op.src2 + c) : 0.0f;
+              w[j][u] = in ? op.w[c] : 0.0f;
+            }
+#pragma unroll
+          for (int j = 0; j < B; ++j) {
+            float ss = 0.0f;
+#pragma unroll
+            for (int u = 0; u < E; ++u) ss += o[j][u] * o[j][u];
+            const float sc = rsqrtf(warp_sum(ss) / static_cast<float>(br.dim) + a.eps);
+            const int h = h0 + j * kListWarps;
+#pragma unroll
+            for (int u = 0; u < E; ++u)
+              if (h < br.H && lane + 32 * u < br.dim) xs[h * br.dim + lane + 32 * u] = o[j][u] * sc * w[j][u] * silu_f(x[j][u]);
+          }
+        }
+      };
+      if (br.dim <= 64) heads(std::integral_constant<int, 2>(), std::integral_constant<int, 2>());
+      else heads(std::integral_constant<int, 8>(), std::integral_constant<int, 1>());   // dim <= 256
+      for (int c = op.n + threadIdx.x; c < op.ld; c += kListThreads) xs[c] = 0.0f;
+    } else if (blockIdx.x == gridDim.x - 1 && wid == kListWarps - 1) {   // kOpLatentStore
       const TokenBranch& br = ph.br[0];
       const float* x = ph.proj + br.col_k;
       T* row = static_cast<T*>(br.cache) + static_cast<int64_t>(pos) * br.ld_cache;
-      float ss[1] = {0.0f};
-      for (int c = threadIdx.x; c < br.kv_rank; c += kThreads) {
+      float ss = 0.0f;
+#pragma unroll 8
+      for (int c = lane; c < br.kv_rank; c += 32) {
         const float v = ldg_f(x + c);
-        ss[0] += v * v;
+        ss += v * v;
       }
-      block_sum<1>(ss, red);
-      const float sc = rsqrtf(ss[0] / static_cast<float>(br.kv_rank) + a.eps);
-      for (int c = threadIdx.x; c < br.kv_rank; c += kThreads) row[c] = from_f<T>(ldg_f(x + c) * sc * br.kv_norm[c]);
+      const float sc = rsqrtf(warp_sum(ss) / static_cast<float>(br.kv_rank) + a.eps);
+      batched<8>(br.kv_rank, lane, 32, [&](int c) { return ldg_f(x + c) * br.kv_norm[c]; }, [&](int c, float v) { row[c] = from_f<T>(v * sc); });
       const int half = br.rot_dim / 2;
-      for (int p = threadIdx.x; p < half; p += kThreads) {
-        const float u = ldg_f(x + br.kv_rank + p), v = ldg_f(x + br.kv_rank + half + p);
+      for (int p = lane; p < half; p += 32) {
+        const float c0 = ldg_f(x + br.kv_rank + p), c1 = ldg_f(x + br.kv_rank + half + p);
         const float2 cs = br.table[static_cast<int64_t>(pos) * half + p];
-        row[br.rot_col + p] = from_f<T>(u * cs.x - v * cs.y);
-        row[br.rot_col + half + p] = from_f<T>(v * cs.x + u * cs.y);
+        row[br.rot_col + p] = from_f<T>(c0 * cs.x - c1 * cs.y);
+        row[br.rot_col + half + p] = from_f<T>(c1 * cs.x + c0 * cs.y);
       }
     }
   }
@@ -648,53 +829,76 @@ __device__ __forceinline__ float gemv_row(const TokenGemv& g, int r, const float
   float v = 0.0f;
   for (int k = 0; k < g.top; ++k) {
     const int e = routed.index[k];
-    if (e < g.experts) v += row_dot<T>(W + (static_cast<int64_t>(e) * g.pitch + r) * g.K, sm + g.in + k * g.K, g.K, part, wpr);
-    else if (part == 0) v = fmaf(routed.weight[k], ldg_f(g.h + r), v);
+    if (e < g.experts) v += row_part<T>(W + (static_cast<int64_t>(e) * g.pitch + r) * g.K, sm + g.in + k * g.K, g.K, part, wpr);
   }
-  if (g.W2 != nullptr) v += row_dot<T>(static_cast<const T*>(g.W2) + static_cast<int64_t>(r) * g.K2, sm + g.in2, g.K2, part, wpr);
+  if (g.W2 != nullptr) v += row_part<T>(static_cast<const T*>(g.W2) + static_cast<int64_t>(r) * g.K2, sm + g.in2, g.K2, part, wpr);
+  v = warp_sum(v);
+  if (part == 0)
+    for (int k = 0; k < g.top; ++k)
+      if (routed.index[k] >= g.experts) v = fmaf(routed.weight[k], ldg_f(g.h + r), v);
   return v;
 }
 
 // 32 value columns of one wkv head (as delta_item: a lane per column, key rows dealt to the warps).
 template <typename T>
-__device__ void wkv_item(const TokenPhase& ph, const TokenBranch& br, int item, int pos, float* sm) {
+__device__ __forceinline__ void wkv_item(const TokenPhase& ph, const TokenBranch& br, int item, int pos) {
+  extern __shared__ __align__(16) float sm[];
   const int nb = (br.dim + 31) / 32, h = item / nb, lane = threadIdx.x & 31, wid = threadIdx.x >> 5;
   const int dim = br.dim, c = (item % nb) * 32 + lane, rw = (br.rank_w + 7) & ~7;
   float *low = sm, *q = low + rw, *k = q + dim, *g = k + dim, *b = g + dim, *red = b + dim;
+  const bool live = c < dim;
+  float* S = br.state + static_cast<int64_t>(h) * dim * dim + c;
+  float s[16];   // dim <= 256: rows wid, wid + 16, ...
+#pragma unroll
+  for (int i = 0; i < 16; ++i) {
+    const int r = wid + kListWarps * i;
+    if (kListWarps * i >= dim) break;
+    s[i] = (r < dim && live && pos > 0) ? ldg_f(S + static_cast<int64_t>(r) * dim) : 0.0f;
+  }
+  const float v = live ? ldg_f(ph.proj + br.col_v + h * dim + c) : 0.0f;
   __syncthreads();
-  for (int i = threadIdx.x; i < rw; i += kThreads) low[i] = i < br.rank_w ? tanhf(ldg_f(ph.proj + br.col_w1 + i)) : 0.0f;
-  __syncthreads();
-  for (int d = threadIdx.x; d < dim; d += kThreads) {
+  for (int i = threadIdx.x; i < rw; i += kListThreads) low[i] = i < br.rank_w ? tanhf(ldg_f(ph.proj + br.col_w1 + i)) : 0.0f;
+  for (int d = threadIdx.x; d < dim; d += kListThreads) {
     const int ch = h * dim + d;
     q[d] = ldg_f(ph.proj + br.col_r + ch);
     k[d] = ldg_f(ph.proj + br.col_k + ch);
     b[d] = br.bonus[ch];
+  }
+  __syncthreads();
+  for (int d = threadIdx.x; d < dim; d += kListThreads) {
+    const int ch = h * dim + d;
     g[d] = expf(-expf(short_dot(static_cast<const T*>(br.w_w2) + static_cast<int64_t>(ch) * rw, low, rw) + br.w0[ch]));
   }
-  const bool live = c < dim;
-  const float v = live ? ldg_f(ph.proj + br.col_v + h * dim + c) : 0.0f;
-  float* S = br.state + static_cast<int64_t>(h) * dim * dim + c;
   __syncthreads();
   float o = 0.0f;
-  if (live) {
-#pragma unroll 8
-    for (int r = wid; r < dim; r += kWarps) {
-      const float s0 = pos > 0 ? ldg_f(S + static_cast<int64_t>(r) * dim) : 0.0f, kv = k[r] * v;
-      o = fmaf(fmaf(b[r], kv, s0), q[r], o);
-      S[static_cast<int64_t>(r) * dim] = fmaf(g[r], s0, kv);
-    }
+#pragma unroll
+  for (int i = 0; i < 16; ++i) {
+    const int r = wid + kListWarps * i;
+    if (kListWarps * i >= dim) break;
+    if (r >= dim) continue;
+    const float kv = k[r] * v;
+    o = fmaf(fmaf(b[r], kv, s[i]), q[r], o);
+    if (live) S[static_cast<int64_t>(r) * dim] = fmaf(g[r], s[i], kv);
   }
-  o = column_sum(o, red);
-  if (wid == 0 && live) br.out[h * dim + c] = o;
+  __syncthreads();
+  red[wid * 32 + lane] = o;
+  __syncthreads();
+  if (wid != 0 || !live) return;
+  o = 0.0f;
+#pragma unroll
+  for (int i = 0; i < kListWarps; ++i) o += red[i * 32 + lane];
+  br.out[h * dim + c] = o;
 }
 
+constexpr int kKeyGroups = kListThreads / 16;
 template <typename T>
 constexpr int kKeyCols = 16 * Chunk<T>::kN;   // latent columns of a key item
 
 // Queries against the cache rows: W_uk^T q for one block of latent columns of a head; the first block also
-// turns the rotated part. Threads: 16 column groups of one 16-byte chunk, 16 groups of key dimensions.
+// turns the rotated part. Threads: 16 column groups of one 16-byte chunk, kKeyGroups groups of key dimensions.
 template <typename T>
-__device__ void latent_keys_item(const TokenPhase& ph, const TokenBranch& br, int item, int pos, float* sm) {
+__device__ __forceinline__ void latent_keys_item(const TokenBranch& br, int item, int pos) {
+  extern __shared__ __align__(16) float sm[];
   constexpr int N = Chunk<T>::kN, COLS = kKeyCols<T>;
   const int nb = (br.rot_col + COLS - 1) / COLS, h = item / nb, r0 = item % nb * COLS;
   const int cg = threadIdx.x & 15, dg = threadIdx.x >> 4, col = r0 + cg * N;
@@ -704,8 +908,8 @@ __device__ void latent_keys_item(const TokenPhase& ph, const TokenBranch& br, in
   for (int e = 0; e < N; ++e) acc[e] = 0.0f;
   if (col < br.ld_ukv) {
     const T* w = static_cast<const T*>(br.w_ukv) + static_cast<int64_t>(h) * br.dim * br.ld_ukv + col;
-#pragma unroll 8
-    for (int d = dg; d < br.dim; d += 16) {
+#pragma unroll 4
+    for (int d = dg; d < br.dim; d += kKeyGroups) {
       Chunk<T> c;
       c.load(w + static_cast<int64_t>(d) * br.ld_ukv);
       const float x = ldg_f(q + d);
@@ -719,37 +923,48 @@ __device__ void latent_keys_item(const TokenPhase& ph, const TokenBranch& br, in
 #pragma unroll
   for (int e = 0; e < N; ++e) sm[dg * (COLS + 1) + cg * N + e] = acc[e];
   __syncthreads();
-  float* out = br.q_abs + static_cast<int64_t>(h) * br.ld_cache;
-  for (int c = threadIdx.x; c < COLS; c += kThreads) {
+  // fp32, or for bfloat16 caches high and low parts, one plane [H][ld_cache] after the other
+  auto put = [&](int c, float v) {
+    const int64_t i = static_cast<int64_t>(h) * br.ld_cache + c;
+    if constexpr (sizeof(T) == 4) {
+      static_cast<float*>(br.q_abs)[i] = v;
+    } else {
+      const T hi = from_f<T>(v);
+      T* q2 = static_cast<T*>(br.q_abs);
+      q2[i] = hi;
+      q2[static_cast<int64_t>(br.H) * br.ld_cache + i] = from_f<T>(v - to_f(hi));
+    }
+  };
+  for (int c = threadIdx.x; c < COLS; c += kListThreads) {
     float v = 0.0f;
 #pragma unroll
-    for (int g = 0; g < 16; ++g) v += sm[g * (COLS + 1) + c];
-    if (r0 + c < br.kv_rank) out[r0 + c] = v * br.scale;
+    for (int g = 0; g < kKeyGroups; ++g) v += sm[g * (COLS + 1) + c];
+    if (r0 + c < br.kv_rank) put(r0 + c, v * br.scale);
   }
   if (r0 == 0) {
     const int half = br.rot_dim / 2;
-    for (int p = threadIdx.x; p < half; p += kThreads) {
+    for (int p = threadIdx.x; p < half; p += kListThreads) {
       const float u = ldg_f(q + br.dim + p), v = ldg_f(q + br.dim + half + p);
       const float2 cs = br.table[static_cast<int64_t>(pos) * half + p];
-      out[br.rot_col + p] = (u * cs.x - v * cs.y) * br.scale;
-      out[br.rot_col + half + p] = (v * cs.x + u * cs.y) * br.scale;
+      put(br.rot_col + p, (u * cs.x - v * cs.y) * br.scale);
+      put(br.rot_col + half + p, (v * cs.x + u * cs.y) * br.scale);
     }
   }
 }
 
-// Position ranges in use for L cached positions, and their length.
+// Position ranges in use for L cached positions, and their length (whole tiles).
 __device__ __forceinline__ int latent_ranges(int L, int splits, int& per) {
-  int n = (L + kLatentKeys - 1) / kLatentKeys;
-  if (n > splits) n = splits;
-  per = (L + n - 1) / n;
-  return (L + per - 1) / per;
+  const int tiles = (L + kLatentKeys - 1) / kLatentKeys, each = (tiles + splits - 1) / splits;
+  per = each * kLatentKeys;
+  return (tiles + each - 1) / each;
 }
 
-// kLatentHeads query heads over one range of cached positions: running maximum, sum and the weighted sum of
-// the latents per head. Scores: a warp per head, a lane per position. Sums: a thread per pair of columns.
-template <typename T, int PAIRS>
-__device__ void latent_scan_item(const TokenBranch& br, int item, int pos, float* sm) {
-  constexpr int N = Chunk<T>::kN, HB = kLatentHeads, KT = kLatentKeys;
+// kLatentHeadsF32 query heads over one range of cached positions: running maximum, sum and the weighted sum
+// of the latents per head. Scores: a warp per head, a lane per position. Sums: a thread per pair of columns.
+__device__ __forceinline__ void latent_scan_f32_item(const TokenBranch& br, int item, int pos) {
+  extern __shared__ __align__(16) float sm[];
+  using T = float;
+  constexpr int N = Chunk<T>::kN, HB = kLatentHeadsF32, KT = kLatentKeys;
   const int blk = item / br.splits, sp = item % br.splits;
   int per;
   const int n_act = latent_ranges(pos + 1, br.splits, per);
@@ -760,28 +975,36 @@ __device__ void latent_scan_item(const TokenBranch& br, int item, int pos, float
   float* qs = sm;                                       // [HB][ldc]
   float* ps = qs + HB * ldc;                            // [HB][KT] scores, then weights
   float* st = ps + HB * KT;                             // [HB] correction of the sums
-  uint4* tile = reinterpret_cast<uint4*>(st + HB);      // [KT][pitch]
-  for (int i = threadIdx.x; i < HB * ldc; i += kThreads) {
-    const int h = blk * HB + i / ldc;
-    qs[i] = h < br.H ? ldg_f(br.q_abs + static_cast<int64_t>(h) * ldc + i % ldc) : 0.0f;
-  }
-  float m = -FLT_MAX, l = 0.0f;   // of head wid
-  float2 acc[PAIRS][HB];
-#pragma unroll
-  for (int p = 0; p < PAIRS; ++p)
-#pragma unroll
-    for (int h = 0; h < HB; ++h) acc[p][h] = make_float2(0.0f, 0.0f);
+  uint4* tiles = reinterpret_cast<uint4*>(st + HB);     // [br.buffers][KT][pitch]
   const uint4* cache = reinterpret_cast<const uint4*>(static_cast<const T*>(br.cache));
+  auto request = [&](int jb) {   // rows past the range stay what they were: their weights are zero
+    uint4* tile = tiles + ((jb - j0) / KT & (br.buffers - 1)) * KT * pitch;
+    const int n = min(KT, j1 - jb) * chunks;
+#pragma unroll 2
+    for (int i = threadIdx.x; i < n; i += kListThreads) cp_async16(tile + i / chunks * pitch + i % chunks, cache + static_cast<int64_t>(jb) * chunks + i);
+    cp_async_commit();
+  };
+  request(j0);
+  {
+    const int c4 = ldc >> 2, valid = (min(br.H, (blk + 1) * HB) - blk * HB) * c4;
+    const float* src = static_cast<const float*>(br.q_abs) + static_cast<int64_t>(blk) * HB * ldc;
+    batched<2>(HB * c4, threadIdx.x, kListThreads, [&](int i) { return i < valid ? ldg4(src + 4 * i) : make_float4(0.f, 0.f, 0.f, 0.f); },
+               [&](int i, const float4& x) { store4(qs + 4 * i, x); });
+  }
+  float m = -FLT_MAX, l = 0.0f;   // of head wid (the first HB warps)
+  float2 acc[HB];   // kv_rank <= 2 kListThreads
+#pragma unroll
+  for (int h = 0; h < HB; ++h) acc[h] = make_float2(0.0f, 0.0f);
+  const int col = 2 * threadIdx.x;
   for (int jb = j0; jb < j1; jb += KT) {
     const int nk = min(KT, j1 - jb);
+    const uint4* tile = tiles + ((jb - j0) / KT & (br.buffers - 1)) * KT * pitch;
+    const bool ahead = br.buffers > 1 && jb + KT < j1;
+    if (ahead) request(jb + KT);
+    if (ahead) cp_async_wait<1>();
+    else cp_async_wait<0>();
     __syncthreads();
-#pragma unroll 4
-    for (int i = threadIdx.x; i < KT * chunks; i += kThreads) {
-      const int r = i / chunks, c = i % chunks;
-      tile[r * pitch + c] = r < nk ? __ldcg(cache + static_cast<int64_t>(jb + r) * chunks + c) : make_uint4(0u, 0u, 0u, 0u);
-    }
-    __syncthreads();
-    {
+    if (wid < HB) {
       const float* q = qs + wid * ldc;
       float s0 = 0.0f, s1 = 0.0f;
 #pragma unroll 2
@@ -800,42 +1023,188 @@ __device__ void latent_scan_item(const TokenBranch& br, int item, int pos, float
       if (lane == 0) st[wid] = c;
     }
     __syncthreads();
-#pragma unroll
-    for (int p = 0; p < PAIRS; ++p) {
-      const int col = 2 * (threadIdx.x + p * kThreads);
-      if (col >= br.kv_rank) break;
+    if (col < br.kv_rank) {
 #pragma unroll
       for (int h = 0; h < HB; ++h) {
-        acc[p][h].x *= st[h];
-        acc[p][h].y *= st[h];
+        acc[h].x *= st[h];
+        acc[h].y *= st[h];
       }
       const T* row = reinterpret_cast<const T*>(tile) + col;
 #pragma unroll 1
-      for (int j = 0; j < KT; j += 4) {
+      for (int j = 0; j < nk; j += 4) {
         float x[4], y[4];
 #pragma unroll
         for (int u = 0; u < 4; ++u) {
-          x[u] = to_f(row[(j + u) * pitch * N]);
-          y[u] = to_f(row[(j + u) * pitch * N + 1]);
+          const bool in = j + u < nk;   // what lies behind the range need not be a number
+          x[u] = in ? to_f(row[(j + u) * pitch * N]) : 0.0f;
+          y[u] = in ? to_f(row[(j + u) * pitch * N + 1]) : 0.0f;
         }
 #pragma unroll
         for (int h = 0; h < HB; ++h) {
           const float4 w = *reinterpret_cast<const float4*>(ps + h * KT + j);
-          acc[p][h].x = fmaf(w.x, x[0], fmaf(w.y, x[1], fmaf(w.z, x[2], fmaf(w.w, x[3], acc[p][h].x))));
-          acc[p][h].y = fmaf(w.x, y[0], fmaf(w.y, y[1], fmaf(w.z, y[2], fmaf(w.w, y[3], acc[p][h].y))));
+          acc[h].x = fmaf(w.x, x[0], fmaf(w.y, x[1], fmaf(w.z, x[2], fmaf(w.w, x[3], acc[h].x))));
+          acc[h].y = fmaf(w.x, y[0], fmaf(w.y, y[1], fmaf(w.z, y[2], fmaf(w.w, y[3], acc[h].y))));
         }
       }
     }
+    __syncthreads();   // before this tile's place or the weights are written again
+    if (br.buffers == 1 && jb + KT < j1) request(jb + KT);
   }
-  const int PS = br.rot_col + kAttnStats;
+  const int PS = br.rot_col + kAttnStats4;
   auto part = [&](int h) { return br.part + (static_cast<int64_t>(blk * HB + h) * br.splits + sp) * PS; };
-#pragma unroll
-  for (int p = 0; p < PAIRS; ++p) {
-    const int col = 2 * (threadIdx.x + p * kThreads);
-    if (col >= br.kv_rank) break;
+  if (col < br.kv_rank) {
 #pragma unroll
     for (int h = 0; h < HB; ++h)   // rows end on an even column: rot_col is a multiple of eight
-      if (blk * HB + h < br.H) *reinterpret_cast<float2*>(part(h) + kAttnStats + col) = acc[p][h];
+      if (blk * HB + h < br.H) *reinterpret_cast<float2*>(part(h) + kAttnStats4 + col) = acc[h];
+  }
+  if (lane == 0 && wid < HB && blk * HB + wid < br.H) {
+    part(wid)[0] = m;
+    part(wid)[1] = l;
+  }
+}
+
+// The same for bfloat16 caches on the tensor cores: kLatentHeads heads are the rows of the products. Queries
+// and weights are split into a bfloat16 sum of two terms (16 mantissa bits, fp32 sums). Scores: a warp per 16
+// positions and eighth of the columns; sums: a warp per 32 NB columns.
+template <int NB>
+__device__ __forceinline__ void latent_scan_bf16_item(const TokenBranch& br, int item, int pos) {
+  extern __shared__ __align__(16) float sm[];
+  using bf16 = __nv_bfloat16;
+  constexpr int HB = kLatentHeads, KT = kLatentKeys, LP = KT + 8;
+  static_assert(HB == kListWarps, "a warp per head");
+  const int blk = item / br.splits, sp = item % br.splits;
+  int per;
+  const int n_act = latent_ranges(pos + 1, br.splits, per);
+  if (sp >= n_act) return;
+  const int lane = threadIdx.x & 31, wid = threadIdx.x >> 5, ldc = br.ld_cache, cols = (ldc + 15) & ~15, pitch = cols + 8;
+  const int j0 = sp * per, j1 = min(pos + 1, j0 + per), chunks = ldc / 8;
+  bf16* qh = reinterpret_cast<bf16*>(sm);               // [HB][pitch] queries, high and low
+  bf16* ql = qh + HB * pitch;
+  bf16* ph = ql + HB * pitch;                           // [HB][LP] weights, high and low
+  bf16* pl = ph + HB * LP;
+  float* sc = reinterpret_cast<float*>(pl + HB * LP);   // [8][HB][KT + 4] scores per eighth of the columns
+  float* st = sc + 8 * HB * (KT + 4);                   // [HB] correction of the sums
+  bf16* tiles = reinterpret_cast<bf16*>(st + HB);       // [br.buffers][KT][pitch]
+  const bf16* cache = static_cast<const bf16*>(br.cache);
+  auto tile_at = [&](int jb) { return tiles + ((jb - j0) / KT & (br.buffers - 1)) * KT * pitch; };
+  auto request = [&](int jb) {   // a warp per row; rows past the end are zero
+    bf16* tile = tile_at(jb);
+    for (int r = wid; r < KT; r += kListWarps) {
+      const bf16* src = cache + static_cast<int64_t>(jb + r) * ldc;
+      for (int c = lane; c < chunks; c += 32) {
+        if (jb + r < j1) cp_async16(tile + r * pitch + c * 8, src + c * 8);
+        else *reinterpret_cast<uint4*>(tile + r * pitch + c * 8) = make_uint4(0u, 0u, 0u, 0u);
+      }
+    }
+    cp_async_commit();
+  };
+  for (int r = wid; r < 2 * HB; r += kListWarps) {   // queries: a warp per row and plane
+    const int h = blk * HB + r % HB;
+    const bf16* src = static_cast<const bf16*>(br.q_abs) + (static_cast<int64_t>(r / HB) * br.H + h) * ldc;
+    for (int c = lane; c < chunks; c += 32) {
+      if (h < br.H) cp_async16(qh + r * pitch + c * 8, src + c * 8);
+      else *reinterpret_cast<uint4*>(qh + r * pitch + c * 8) = make_uint4(0u, 0u, 0u, 0u);
+    }
+  }
+  request(j0);
+  if (cols > ldc)   // columns up to the product's slice of 16
+    for (int i = threadIdx.x; i < 2 * HB + br.buffers * KT; i += kListThreads)
+      *reinterpret_cast<uint4*>((i < 2 * HB ? qh + i * pitch : tiles + (i - 2 * HB) * pitch) + ldc) = make_uint4(0u, 0u, 0u, 0u);
+  const int slice = wid >> 1, n0 = (wid & 1) * 16, steps = cols / 16, s0 = steps * slice / 8, s1 = steps * (slice + 1) / 8;
+  const int c0 = wid * NB * 32;   // the warp's columns of the sums
+  float m = -FLT_MAX, l = 0.0f;   // of head wid
+  float acc[NB * 4][4];
+#pragma unroll
+  for (int t = 0; t < NB * 4; ++t)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) acc[t][e] = 0.0f;
+  for (int jb = j0; jb < j1; jb += KT) {
+    const int nk = min(KT, j1 - jb);
+    const bf16* tile = tile_at(jb);
+    const bool ahead = br.buffers > 1 && jb + KT < j1;
+    if (ahead) request(jb + KT);
+    if (ahead) cp_async_wait<1>();
+    else cp_async_wait<0>();
+    __syncthreads();
+    {
+      float s[2][4] = {};
+#pragma unroll 2
+      for (int k = s0; k < s1; ++k) {
+        uint32_t Ah[4], Al[4], B[4];
+        ldsm_a(Ah, qh, pitch, 0, k * 16, lane);
+        ldsm_a(Al, ql, pitch, 0, k * 16, lane);
+        ldsm_b(B, tile, pitch, k * 16, n0, lane);
+#pragma unroll
+        for (int t = 0; t < 2; ++t) {
+          mma_bf16(s[t], Ah, B[2 * t], B[2 * t + 1]);
+          mma_bf16(s[t], Al, B[2 * t], B[2 * t + 1]);
+        }
+      }
+      float* dst = sc + (slice * HB + (lane >> 2)) * (KT + 4) + n0 + (lane & 3) * 2;
+#pragma unroll
+      for (int t = 0; t < 2; ++t)
+#pragma unroll
+        for (int f = 0; f < 2; ++f)
+          *reinterpret_cast<float2*>(dst + f * 8 * (KT + 4) + t * 8) = make_float2(s[t][2 * f], s[t][2 * f + 1]);
+    }
+    __syncthreads();
+    {
+      const float* src = sc + wid * (KT + 4) + lane;
+      float s = 0.0f;
+#pragma unroll
+      for (int k = 0; k < 8; ++k) s += src[k * HB * (KT + 4)];
+      if (lane >= nk) s = -FLT_MAX;
+      const float mn = fmaxf(m, warp_max(s));
+      const float p = lane < nk ? expf(s - mn) : 0.0f, c = expf(m - mn);
+      l = l * c + warp_sum(p);
+      m = mn;
+      const bf16 hi = __float2bfloat16(p);
+      ph[wid * LP + lane] = hi;
+      pl[wid * LP + lane] = __float2bfloat16(p - __bfloat162float(hi));
+      if (lane == 0) st[wid] = c;
+    }
+    __syncthreads();
+    if (c0 < br.kv_rank) {
+      const float f0 = st[lane >> 2], f1 = st[(lane >> 2) + 8];
+#pragma unroll
+      for (int t = 0; t < NB * 4; ++t) {
+        acc[t][0] *= f0;
+        acc[t][1] *= f0;
+        acc[t][2] *= f1;
+        acc[t][3] *= f1;
+      }
+#pragma unroll
+      for (int k = 0; k < KT; k += 16) {
+        uint32_t Ah[4], Al[4];
+        ldsm_a(Ah, ph, LP, 0, k, lane);
+        ldsm_a(Al, pl, LP, 0, k, lane);
+#pragma unroll
+        for (int t = 0; t < NB * 4; t += 2) {
+          if (c0 + t * 8 >= br.kv_rank) break;
+          uint32_t B[4];
+          ldsm_b_trans(B, tile, pitch, k, c0 + t * 8, lane);
+#pragma unroll
+          for (int e = 0; e < 2; ++e) {
+            mma_bf16(acc[t + e], Ah, B[2 * e], B[2 * e + 1]);
+            mma_bf16(acc[t + e], Al, B[2 * e], B[2 * e + 1]);
+          }
+        }
+      }
+    }
+    __syncthreads();   // before this tile's place or the weights are written again
+    if (br.buffers == 1 && jb + KT < j1) request(jb + KT);
+  }
+  const int PS = br.rot_col + kAttnStats4;
+  auto part = [&](int h) { return br.part + (static_cast<int64_t>(blk * HB + h) * br.splits + sp) * PS; };
+#pragma unroll
+  for (int t = 0; t < NB * 4; ++t) {
+    const int col = c0 + t * 8 + (lane & 3) * 2;
+    if (col >= br.kv_rank) break;
+#pragma unroll
+    for (int f = 0; f < 2; ++f) {
+      const int h = (lane >> 2) + 8 * f;
+      if (blk * HB + h < br.H) *reinterpret_cast<float2*>(part(h) + kAttnStats4 + col) = make_float2(acc[t][2 * f], acc[t][2 * f + 1]);
+    }
   }
   if (lane == 0 && blk * HB + wid < br.H) {
     part(wid)[0] = m;
@@ -843,14 +1212,30 @@ __device__ void latent_scan_item(const TokenBranch& br, int item, int pos, float
   }
 }
 
+constexpr int kOutParts = kLatentOutParts;
+
 // kLatentOutRows value rows of a head: merges the head's ranges, then W_uv times the mean latent, gated.
 template <typename T>
-__device__ void latent_out_item(const TokenPhase& ph, const TokenBranch& br, int item, int pos, float* sm) {
+__device__ __forceinline__ void latent_out_item(const TokenPhase& ph, const TokenBranch& br, int item, int pos) {
+  extern __shared__ __align__(16) float sm[];
   const int nb = (br.vdim + kLatentOutRows - 1) / kLatentOutRows, h = item / nb, r0 = item % nb * kLatentOutRows;
-  const int lane = threadIdx.x & 31, wid = threadIdx.x >> 5, PS = br.rot_col + kAttnStats;
+  const int lane = threadIdx.x & 31, wid = threadIdx.x >> 5, PS = br.rot_col + kAttnStats4;
   int per;
   const int n_act = latent_ranges(pos + 1, br.splits, per);
-  float *o = sm, *w = o + br.rot_col;   // [rot_col] mean latent, [splits] weights of the ranges
+  // [rot_col] mean latent, [splits] weights of the ranges, [kOutParts][rot_col] partial sums
+  float *o = sm, *sums = o + br.rot_col, *w = sums + kOutParts * br.rot_col;
+  // the weight rows are requested before the ranges are merged: ROWS rows per warp, HELD chunks per lane of each
+  constexpr int N = Chunk<T>::kN, ROWS = kLatentOutRows / kListWarps, HELD = 2;
+  const int ld = br.ld_ukv;
+  const T* rows = static_cast<const T*>(br.w_ukv) + (static_cast<int64_t>(br.row_uv) + h * br.vdim) * ld;
+  Chunk<T> held[ROWS][HELD];
+#pragma unroll
+  for (int u = 0; u < ROWS; ++u)
+#pragma unroll
+    for (int k = 0; k < HELD; ++k)
+      if (r0 + wid + u * kListWarps < br.vdim && (k * 32 + lane) * N < ld)
+        held[u][k].load(rows + static_cast<int64_t>(r0 + wid + u * kListWarps) * ld + (k * 32 + lane) * N);
+  const float gate = sigmoid_f(ldg_f(ph.proj + br.col_g + h));
   const float* part = br.part + static_cast<int64_t>(h) * br.splits * PS;
   __syncthreads();
   if (wid == 0) {
@@ -868,30 +1253,52 @@ __device__ void latent_out_item(const TokenPhase& ph, const TokenBranch& br, int
     for (int s = lane; s < n_act; s += 32) w[s] *= l;
   }
   __syncthreads();
-  for (int c = threadIdx.x; c < br.rot_col; c += kThreads) {
-    float v = 0.0f;
-    if (c < br.kv_rank)
+  {   // four columns per thread; the ranges are dealt to kOutParts groups of threads
+    const int quads = br.rot_col / 4, n = quads * kOutParts;
+    for (int i = threadIdx.x; i < n; i += kListThreads) {
+      const int c = i % quads * 4, first = i / quads;
+      float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll 8
-      for (int s = 0; s < n_act; ++s) v = fmaf(w[s], ldg_f(part + static_cast<int64_t>(s) * PS + kAttnStats + c), v);
-    o[c] = v;
+      for (int s = first; s < n_act; s += kOutParts) {
+        const float4 x = ldg4(part + static_cast<int64_t>(s) * PS + kAttnStats4 + c);
+        v = make_float4(fmaf(w[s], x.x, v.x), fmaf(w[s], x.y, v.y), fmaf(w[s], x.z, v.z), fmaf(w[s], x.w, v.w));
+      }
+      store4(sums + first * br.rot_col + c, v);
+    }
   }
   __syncthreads();
-  const float gate = sigmoid_f(ldg_f(ph.proj + br.col_g + h));
-  for (int r = r0 + wid; r < min(br.vdim, r0 + kLatentOutRows); r += kWarps) {
-    const T* row = static_cast<const T*>(br.w_ukv) + (static_cast<int64_t>(br.row_uv) + h * br.vdim + r) * br.ld_ukv;
-    const float v = row_dot<T>(row, o, br.ld_ukv, 0, 1);
-    if (lane == 0) br.out[h * br.vdim + r] = v * gate;
+  for (int c = threadIdx.x; c < br.rot_col; c += kListThreads) {
+    float v = 0.0f;
+#pragma unroll
+    for (int g = 0; g < kOutParts; ++g) v += sums[g * br.rot_col + c];
+    o[c] = c < br.kv_rank ? v : 0.0f;
+  }
+  __syncthreads();
+#pragma unroll
+  for (int u = 0; u < ROWS; ++u) {
+    float v = 0.0f;
+#pragma unroll
+    for (int k = 0; k < HELD; ++k)
+      if ((k * 32 + lane) * N < ld) v = held[u][k].dot(o + (k * 32 + lane) * N, v);
+    const int r = r0 + wid + u * kListWarps;
+    for (int c = HELD * 32 + lane; c * N < ld && r < br.vdim; c += 32) {
+      Chunk<T> w1;
+      w1.load(rows + static_cast<int64_t>(r) * ld + c * N);
+      v = w1.dot(o + c * N, v);
+    }
+    v = warp_sum(v);
+    if (lane == 0 && r < br.vdim) br.out[h * br.vdim + r] = v * gate;
   }
 }
 
 template <typename T>
-__device__ void list_item(const TokenPhase& ph, int item, int pos, float* sm) {
+__device__ __forceinline__ void list_item(const TokenPhase& ph, int item, int pos) {
   const TokenBranch& br = ph.br[0];
-  if (br.kind == kTokWkv) wkv_item<T>(ph, br, item, pos, sm);
-  else if (br.kind == kTokLatentKeys) latent_keys_item<T>(ph, br, item, pos, sm);
-  else if (br.kind == kTokLatentOut) latent_out_item<T>(ph, br, item, pos, sm);
-  else if (br.kv_rank <= 2 * kThreads) latent_scan_item<T, 1>(br, item, pos, sm);
-  else latent_scan_item<T, 2>(br, item, pos, sm);
+  if (br.kind == kTokWkv) wkv_item<T>(ph, br, item, pos);
+  else if (br.kind == kTokLatentKeys) latent_keys_item<T>(br, item, pos);
+  else if (br.kind == kTokLatentOut) latent_out_item<T>(ph, br, item, pos);
+  else if constexpr (sizeof(T) == 2) br.kv_rank <= 512 ? latent_scan_bf16_item<1>(br, item, pos) : latent_scan_bf16_item<2>(br, item, pos);
+  else latent_scan_f32_item(br, item, pos);
 }
 
 // Staging, products, items. The items lie at the front of the grid, so rows start behind them.
@@ -899,14 +1306,14 @@ template <typename T>
 __device__ unsigned long long list_phase(const TokenArgs& a, const TokenPhase& ph, int64_t tok, int pos, float* sm, float* red, float* part_red,
                                          Routed& routed) {
   const int lane = threadIdx.x & 31, wid = threadIdx.x >> 5;
-  if (ph.n_ops > 0) stage_list<T>(a, ph, tok, pos, sm, red, routed);
+  if (ph.n_ops > 0) stage_list<T>(a, ph, tok, pos, red, routed);
   unsigned long long best = 0ull;
   int total = 0;
   for (int i = 0; i < ph.n_gemv; ++i) total += ph.gemv[i].rows;
   const int items = ph.n_branch > 0 ? ph.br[0].items : 0;
   int cta = static_cast<int>(blockIdx.x) - items % static_cast<int>(gridDim.x);
   if (cta < 0) cta += gridDim.x;
-  const int wpr = ph.wpr, groups = kWarps / (wpr > 0 ? wpr : 1), part = wpr > 0 ? wid % wpr : 0;
+  const int wpr = ph.wpr, groups = kListWarps / (wpr > 0 ? wpr : 1), part = wpr > 0 ? wid % wpr : 0;
   auto find = [&](int n, int& r) {
     int i = 0;
     while (n >= ph.gemv[i].rows) n -= ph.gemv[i++].rows;
@@ -921,7 +1328,7 @@ __device__ unsigned long long list_phase(const TokenArgs& a, const TokenPhase& p
     }
   };
   if (wpr == 1) {
-    for (int n = cta * kWarps + wid; n < total; n += gridDim.x * kWarps) {
+    for (int n = cta * kListWarps + wid; n < total; n += gridDim.x * kListWarps) {
       int r;
       const TokenGemv& g = ph.gemv[find(n, r)];
       const float v = gemv_row<T>(g, r, sm, 0, 1, routed);
@@ -946,12 +1353,12 @@ __device__ unsigned long long list_phase(const TokenArgs& a, const TokenPhase& p
   }
   for (int it = blockIdx.x; it < items; it += gridDim.x) {
     __syncthreads();
-    list_item<T>(ph, it, pos, sm);
+    list_item<T>(ph, it, pos);
   }
   return best;
 }
 
-template <typename T>
+template <typename T, int kThreads>
 __device__ void prefetch_phase(const TokenPhase& ph) {
   if (ph.extra != nullptr) {
     const char* base = static_cast<const char*>(ph.extra);
@@ -970,7 +1377,8 @@ __device__ void prefetch_phase(const TokenPhase& ph) {
 
 // LIST: every phase is a kStageList phase (parallel arrangement); otherwise none is.
 template <typename T, bool LIST>
-__global__ void __launch_bounds__(kThreads, 2) hybrid_token_kernel(const __grid_constant__ TokenArgs a) {
+__global__ void __launch_bounds__(LIST ? kListThreads : kThreads, LIST ? 1 : 2) hybrid_token_kernel(const __grid_constant__ TokenArgs a) {
+  constexpr int kThreads = token_threads(LIST), kWarps = kThreads / 32;
   extern __shared__ __align__(16) float sm[];
   __shared__ TokenPhase ph_s[2];
   __shared__ float red[2 * kWarps];
@@ -1066,7 +1474,7 @@ __global__ void __launch_bounds__(kThreads, 2) hybrid_token_kernel(const __grid_
           atomicMax(&words[t & 1], best);
         }
       }
-      if (ph.prefetch >= 0) prefetch_phase<T>(a.phases[ph.prefetch]);
+      if (ph.prefetch >= 0) prefetch_phase<T, kThreads>(a.phases[ph.prefetch]);
       if (i + 1 < a.n_phases) fetch(i + 1);
       if (i + 1 == a.n_phases && a.out_tokens == nullptr) break;   // logits are complete at the end of the kernel
       if (!(alive = grid_barrier(a.sync, a.status, 91, epoch))) break;
@@ -1118,10 +1526,11 @@ int token_grid(size_t smem, bool list, int* grid) {
   if (e == cudaSuccess) e = cudaDeviceGetAttribute(&coop, cudaDevAttrCooperativeLaunch, dev);
   if (e == cudaSuccess)
     e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
-  if (e == cudaSuccess) e = cudaOccupancyMaxActiveBlocksPerMultiprocessor(&per_sm, kernel, kThreads, smem);
+  if (e == cudaSuccess) e = cudaOccupancyMaxActiveBlocksPerMultiprocessor(&per_sm, kernel, token_threads(list), smem);
   if (e != cudaSuccess) return fail(CTDK_ELAUNCH, "hybrid token kernel: %s", cudaGetErrorString(e));
   CTDK_REQUIRE(coop != 0 && per_sm >= 1, "hybrid token kernel: no cooperative launch with %zu bytes of shared memory", smem);
-  *grid = sm_count() * (per_sm > 2 ? 2 : per_sm);
+  const int most = list ? 1 : 2;   // CTAs per SM the kernel is made for
+  *grid = sm_count() * (per_sm > most ? most : per_sm);
   return CTDK_OK;
 }
 
@@ -1131,7 +1540,7 @@ int launch_token_kernel(const TokenArgs& a, bool list, int grid, size_t smem, cu
     return fail(CTDK_ELAUNCH, "hybrid token kernel: clearing the barrier words failed");
   TokenArgs args = a;
   void* params[] = {&args};
-  const cudaError_t e = cudaLaunchCooperativeKernel(list ? reinterpret_cast<const void*>(hybrid_token_kernel<T, true>) : reinterpret_cast<const void*>(hybrid_token_kernel<T, false>), dim3(grid), dim3(kThreads),
+  const cudaError_t e = cudaLaunchCooperativeKernel(list ? reinterpret_cast<const void*>(hybrid_token_kernel<T, true>) : reinterpret_cast<const void*>(hybrid_token_kernel<T, false>), dim3(grid), dim3(token_threads(list)),
                                                     params, smem, s);
   if (e != cudaSuccess) return fail(CTDK_ELAUNCH, "hybrid token kernel: %s", cudaGetErrorString(e));
   return check_launch("hybrid token kernel");

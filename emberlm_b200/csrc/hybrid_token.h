@@ -11,11 +11,15 @@ namespace hybrid {
 
 constexpr int kAttnSplits = 16;   // most key ranges per key/value head
 constexpr int kAttnStats = 2;     // running maximum and sum in front of a partial output
+constexpr int kAttnStats4 = 4;    // the same, with room that keeps the output 16-byte aligned
 
-constexpr int kLatentHeads = 8;    // query heads that share one pass over the latent cache
-constexpr int kLatentSplits = 64;  // most position ranges per block of heads
+constexpr int kListThreads = 512, kListWarps = kListThreads / 32;   // of a CTA that runs kStageList phases, one per SM
+constexpr int kLatentHeads = 16;   // query heads that share one pass over the latent cache (bfloat16)
+constexpr int kLatentHeadsF32 = 8; // the same for fp32 models
+constexpr int kLatentSplits = 96;  // most position ranges per block of heads
 constexpr int kLatentKeys = 32;    // cache rows staged at once
 constexpr int kLatentOutRows = 32; // value rows of an output item
+constexpr int kLatentOutParts = 4; // thread groups that share the merging of the ranges
 
 enum StageKind { kStageNorm = 0, kStageGlu = 1, kStageMixed = 2, kStageList = 3 };
 enum TokenBranchKind { kTokAttention = 0, kTokLightning = 1, kTokDelta = 2, kTokWkv = 3, kTokLatentKeys = 4, kTokLatentScan = 5, kTokLatentOut = 6 };
@@ -39,7 +43,7 @@ enum StageOpKind {
   kOpShiftNorm,     // TokenShift below: h at 0, the shifted row at ldw, the mixes behind it
   kOpRmsNorm,       // n values of src, normed, * w
   kOpCopy,          // n values of src
-  kOpRoute,         // chooses the experts from the n router logits src, correction w (kept until the next choice)
+  kOpRoute,         // src2 (width values) padded to ld; chooses the experts from the n router logits src, correction w (kept until the next choice)
   kOpGelu,          // gelu(src[c]) src[ld + c], c < n
   kOpShared,        // sigmoid(src2[0]) silu(src[c]) src[ld + c], c < n
   kOpExperts,       // per chosen expert: weight silu(gate) up, n columns from its 2 n values of src
@@ -56,6 +60,7 @@ constexpr int kMaxGemv = 6, kMaxOps = 4, kTokenMixes = 5;
 // position reads the slot of the one before and writes its own (slot = position mod 2).
 struct TokenShift {
   int groups, wpg, n_mix, ld, red;   // red: first float of the reduction scratch
+  int vec;                           // columns can be taken four at a time
   const float *x, *y1, *y2, *z1, *z2, *b1, *b2, *w, *shift, *mu[kTokenMixes];
   float *x_out, *h_out, *state;
 };
@@ -90,10 +95,10 @@ struct TokenBranch {
   const void* w_w2;
   const float *w0, *bonus;
   // latent attention
-  int rot_dim, kv_rank, rot_col, ld_cache, ld_ukv, row_uv, splits, blocks;
+  int rot_dim, kv_rank, rot_col, ld_cache, ld_ukv, row_uv, splits, blocks, buffers;   // buffers: cache tiles in flight (1 or 2)
   const void* w_ukv;
   const float *kv_norm, *q_up;   // queries [H][dim + rot_dim]
-  float* q_abs;          // [H][ld_cache] queries against the cache rows, scaled
+  void* q_abs;           // [H][ld_cache] queries against the cache rows, scaled: fp32, or two bfloat16 planes
 };
 
 struct TokenPhase {

@@ -45,6 +45,83 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(const LatentArgs<T> a,
   }
 }
 
+// The same for widths that are multiples of four: a row's side stays in registers, B float4 per lane.
+template <typename T, int B>
+__global__ void __launch_bounds__(256) latent_prep4_kernel(const LatentArgs<T> a, int64_t first, int64_t rows) {
+  pdl_launch();
+  pdl_wait();
+  const int lane = threadIdx.x & 31;
+  const int64_t nw = static_cast<int64_t>(gridDim.x) * 8;
+  for (int64_t i = (static_cast<int64_t>(blockIdx.x) * 256 + threadIdx.x) >> 5; i < 2 * rows; i += nw) {
+    const int64_t r = i >> 1;
+    const bool is_q = (i & 1) == 0;
+    const int n = is_q ? a.q_rank : a.kv_rank;
+    const float* x = a.proj + r * a.ldp + (is_q ? a.col_q : a.col_k);
+    const float* w = is_q ? a.q_norm : a.kv_norm;
+    T* dst = is_q ? a.low_q + r * a.ld_low : a.cache + (first + r) * a.ld_cache;
+    float4 v[B];
+    float ss = 0.0f;
+#pragma unroll
+    for (int u = 0; u < B; ++u) {
+      const int c = (u * 32 + lane) * 4;
+      v[u] = c < n ? load4(x + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+#pragma unroll
+    for (int u = 0; u < B; ++u) ss += v[u].x * v[u].x + v[u].y * v[u].y + v[u].z * v[u].z + v[u].w * v[u].w;
+    const float sc = rsqrtf(warp_sum(ss) / static_cast<float>(n) + a.eps);
+#pragma unroll
+    for (int u = 0; u < B; ++u) {
+      const int c = (u * 32 + lane) * 4;
+      if (c < n) {
+        const float4 g = load4(w + c);
+        store4(dst + c, make_float4(v[u].x * sc * g.x, v[u].y * sc * g.y, v[u].z * sc * g.z, v[u].w * sc * g.w));
+      }
+    }
+    if (is_q) continue;
+    const int half = a.rot_dim / 2;
+    for (int p = lane; p < half; p += 32) {
+      const float u = x[n + p], y = x[n + half + p];
+      const float2 cs = a.table[(first + r) * half + p];
+      dst[a.rot_col + p] = from_f<T>(u * cs.x - y * cs.y);
+      dst[a.rot_col + half + p] = from_f<T>(y * cs.x + u * cs.y);
+    }
+  }
+}
+
+// Head sizes that are multiples of eight and a rotated part of sixteen: a CTA per row, units of eight columns
+// (unrotated) or of two times eight (the two halves of the rotated part).
+template <typename T>
+__global__ void __launch_bounds__(256) latent_rotate8_kernel(const LatentArgs<T> a, int64_t first, int64_t rows) {
+  pdl_launch();
+  pdl_wait();
+  const int D = a.dim + a.rot_dim, half = a.rot_dim / 2, flat = a.dim / 8, per = flat + half / 8, n = a.H * per;
+  for (int64_t r = blockIdx.x; r < rows; r += gridDim.x) {
+    const float* row = a.q_up + r * a.ld_up;
+    const float2* table = a.table + (first + r) * half;
+    T* out = a.q + r * a.H * D;
+#pragma unroll 2
+    for (int i = threadIdx.x; i < n; i += 256) {
+      const int h = i / per, u = i % per;
+      const int c = u < flat ? 8 * u : a.dim + 8 * (u - flat);
+      const float* x = row + h * D + c;
+      T* dst = out + h * D + c;
+      const float4 p = load4(x), q = load4(x + 4);
+      if (u < flat) {
+        store4(dst, p);
+        store4(dst + 4, q);
+        continue;
+      }
+      const float4 s = load4(x + half), t = load4(x + half + 4);
+      const float4* cs = reinterpret_cast<const float4*>(table + 8 * (u - flat));   // two pairs (cos, sin)
+      const float4 c0 = cs[0], c1 = cs[1], c2 = cs[2], c3 = cs[3];
+      store4(dst, make_float4(p.x * c0.x - s.x * c0.y, p.y * c0.z - s.y * c0.w, p.z * c1.x - s.z * c1.y, p.w * c1.z - s.w * c1.w));
+      store4(dst + 4, make_float4(q.x * c2.x - t.x * c2.y, q.y * c2.z - t.y * c2.w, q.z * c3.x - t.z * c3.y, q.w * c3.z - t.w * c3.w));
+      store4(dst + half, make_float4(s.x * c0.x + p.x * c0.y, s.y * c0.z + p.y * c0.w, s.z * c1.x + p.z * c1.y, s.w * c1.z + p.w * c1.w));
+      store4(dst + half + 4, make_float4(t.x * c2.x + q.x * c2.y, t.y * c2.z + q.y * c2.w, t.z * c3.x + q.z * c3.y, t.w * c3.z + q.w * c3.w));
+    }
+  }
+}
+
 // One thread per (row, head, column of the padded head).
 template <typename T>
 __global__ void __launch_bounds__(256) latent_rotate_kernel(const LatentArgs<T> a, int64_t first, int64_t rows) {
@@ -139,10 +216,18 @@ __global__ void __launch_bounds__(256) latent_attention_fp32_kernel(const Latent
 
 template <typename T>
 int latent_prep(const LatentArgs<T>& a, int64_t first, int64_t rows, cudaStream_t s) {
+  const int wide = a.q_rank > a.kv_rank ? a.q_rank : a.kv_rank;
+  if (a.q_rank % 4 == 0 && a.kv_rank % 4 == 0 && wide <= 1024) {
+    const int grid = row_grid(2 * rows, 8);
+    if (wide <= 256) LAUNCH("latent prep", (latent_prep4_kernel<T, 2>), grid, 0, a, first, rows);
+    if (wide <= 512) LAUNCH("latent prep", (latent_prep4_kernel<T, 4>), grid, 0, a, first, rows);
+    LAUNCH("latent prep", (latent_prep4_kernel<T, 8>), grid, 0, a, first, rows);
+  }
   LAUNCH("latent prep", latent_prep_kernel<T>, row_grid(2 * rows, 8), 0, a, first, rows);
 }
 template <typename T>
 int latent_rotate(const LatentArgs<T>& a, int64_t first, int64_t rows, cudaStream_t s) {
+  if (a.dim % 8 == 0 && a.rot_dim % 16 == 0) LAUNCH("latent rotate", latent_rotate8_kernel<T>, row_grid(rows), 0, a, first, rows);
   LAUNCH("latent rotate", latent_rotate_kernel<T>, row_grid(rows * a.H * latent_q_pitch(a.dim, a.rot_dim), 256), 0, a, first, rows);
 }
 template <typename T>

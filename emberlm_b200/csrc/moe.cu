@@ -90,7 +90,16 @@ __global__ void __launch_bounds__(256) moe_gather_kernel(const MoeArgs a, const 
     const T* src = h + i / a.top * ld_h;
     T* dst = xe + static_cast<int64_t>(slot) * ld_h;
     const int vecs = static_cast<int>(ld_h * sizeof(T) / 16);   // the pitch is a multiple of 8 elements
-    for (int c = lane; c < vecs; c += 32) reinterpret_cast<uint4*>(dst)[c] = reinterpret_cast<const uint4*>(src)[c];
+    constexpr int U = 8;   // in flight
+    for (int c0 = lane; c0 < vecs; c0 += 32 * U) {
+      uint4 v[U];
+#pragma unroll
+      for (int u = 0; u < U; ++u)
+        if (c0 + 32 * u < vecs) v[u] = reinterpret_cast<const uint4*>(src)[c0 + 32 * u];
+#pragma unroll
+      for (int u = 0; u < U; ++u)
+        if (c0 + 32 * u < vecs) reinterpret_cast<uint4*>(dst)[c0 + 32 * u] = v[u];
+    }
   }
 }
 

@@ -5,9 +5,11 @@
 //   o_i = (r_i e^(b_(i-1)))^T S + sum_(j < i) (r_i . k_j e^(b_(i-1) - b_j)) v_j + (r_i . u k_i) v_i
 //   S'  = diag(e^(b_last)) S + sum_j (k_j e^(b_last - b_j)) v_j^T
 // Three kernels: every chunk's own contribution to the state, a scan over the chunks in fp32, and the
-// outputs with the norm over each head and the output gate. Exponents are never positive: between 16-row
-// blocks both factors are taken relative to the running sum in front of the later block, inside a block the
-// difference is formed per pair. r, k, v are bfloat16 (projections); whatever carries a decay is split into
+// outputs with the norm over each head and the output gate. The pair factors e^(b_(i-1) - b_j) are split at
+// the running sum of the chunk's middle row while the chunk's decays stay above 2^-kReach in every channel
+// (then both factors stay within fp32 and bfloat16 range). Otherwise no exponent is ever positive: between
+// 16-row blocks both factors are taken relative to the running sum in front of the later block, inside a
+// block the difference is formed per pair. r, k, v are bfloat16 (projections); whatever carries a decay is split into
 // a bfloat16 sum of two terms before it meets a tensor core (16 mantissa bits, fp32 sums), the state itself
 // is carried in fp32. mma.sync m16n8k16.
 #include <cuda_bf16.h>
@@ -24,6 +26,7 @@ constexpr int C = kWkvChunk;
 constexpr int kPad = 8;        // bfloat16 columns behind every shared-memory row: conflict-free ldmatrix
 constexpr float kLog2e = 1.4426950408889634f;
 constexpr float kFloor = -150.0f;   // a log2 decay below this wipes the channel either way
+constexpr float kReach = 100.0f;
 
 __device__ __forceinline__ float ex2(float x) {
   float y;
@@ -41,7 +44,7 @@ __device__ __forceinline__ float4 fetch4(const float* p, int left, bool vec) {
   if (left > 3) x.w = p[3];
   return x;
 }
-__device__ __forceinline__ float log2_decay(float z) { return fmaxf(-expf(z) * kLog2e, kFloor); }
+__device__ __forceinline__ float log2_decay(float z) { return fmaxf(-ex2(z * kLog2e) * kLog2e, kFloor); }
 __device__ __forceinline__ void put_split(__nv_bfloat16* hi, __nv_bfloat16* lo, const float4& v) {
   uint32_t h0, l0, h1, l1;
   split_bf16x2(v.x, v.y, h0, l0);
@@ -215,8 +218,9 @@ __global__ void __launch_bounds__(128) wkv_state_kernel(const WkvArgs a, int chu
 template <int D>
 struct OutCfg {
   static constexpr int LB = D + 4, L = D + kPad, LA = C + kPad;
-  // b, r, k, v, (16-row block factors | r e^b) x 2, scores x 2, state x 2
-  static constexpr int kBytes = C * LB * 4 + 3 * C * L * 2 + 2 * C * L * 2 + 2 * C * LA * 2 + 2 * D * L * 2 + 256 * 4 + D * 4;
+  // b, r, k, v, (query factors | r e^b) x 2, (key factors | scores) x 2, state x 2
+  static_assert(L >= LA, "the scores lie where the key factors were");
+  static constexpr int kBytes = C * LB * 4 + 3 * C * L * 2 + 2 * C * L * 2 + 2 * C * L * 2 + 2 * D * L * 2 + 256 * 4 + D * 4;
 };
 
 // grid (chunks, heads), 256 threads.
@@ -234,8 +238,8 @@ __global__ void __launch_bounds__(256) wkv_out_kernel(const WkvArgs a) {
   __nv_bfloat16* fh = vs + C * L;                                       // [C][L] factors, high and low
   __nv_bfloat16* fl = fh + C * L;
   __nv_bfloat16* ah = fl + C * L;                                       // [C][LA] scores, high and low
-  __nv_bfloat16* al = ah + C * LA;
-  __nv_bfloat16* sh = al + C * LA;                                      // [D][L] state, high and low
+  __nv_bfloat16* al = ah + C * L;
+  __nv_bfloat16* sh = al + C * L;                                       // [D][L] state, high and low
   __nv_bfloat16* sl = sh + D * L;
   pdl_launch();
   pdl_wait();
@@ -267,86 +271,152 @@ __global__ void __launch_bounds__(256) wkv_out_kernel(const WkvArgs a) {
     store4(b_s + r * LB + d, g);
   }
   for (int d = tid; d < D; d += 256) u_s[d] = d < a.dim ? a.bonus[h * a.dim + d] : 0.0f;
-  for (int i = tid; i < C * LA / 4; i += 256) reinterpret_cast<uint2*>(ah)[i] = reinterpret_cast<uint2*>(al)[i] = make_uint2(0u, 0u);
   __syncthreads();
   running_sums<D, LB>(b_s, scratch);
 
-  // pairs inside a 16-row block: a thread has row i and the columns jq, jq + 4, ... up to i
-  {
-    const int blk = tid >> 6 << 4, il = (tid >> 2) & 15, jq = tid & 3, i = blk + il;
-    float s[4] = {0.f, 0.f, 0.f, 0.f};
-    const float* bi = b_s + (i - 1) * LB;
-#pragma unroll 2
-    for (int d = 0; d < D; d += 4) {
-      const float4 r = load4(rs + i * L + d), u = load4(u_s + d);
-      const float4 b = i > 0 ? load4(bi + d) : make_float4(0.f, 0.f, 0.f, 0.f);
+  float reach = 0.0f;
+  for (int d = tid; d < D; d += 256) reach = fminf(reach, b_s[(C - 1) * LB + d]);
+  if (__syncthreads_or(reach < -kReach) == 0) {
+    __nv_bfloat16 *xh = ah, *xl = al;   // [C][L] key factors, where the scores will be
+    const float* ref = b_s + (C / 2 - 1) * LB;
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int jl = jq + 4 * e, j = blk + jl;
-        if (jl > il) break;
-        const float4 k = load4(ks + j * L + d);
-        float4 f = u;
-        if (jl < il) {
-          const float4 bj = load4(b_s + j * LB + d);
-          f = make_float4(ex2(b.x - bj.x), ex2(b.y - bj.y), ex2(b.z - bj.z), ex2(b.w - bj.w));
-        }
-        s[e] = fmaf(r.x * k.x, f.x, fmaf(r.y * k.y, f.y, fmaf(r.z * k.z, f.z, fmaf(r.w * k.w, f.w, s[e]))));
-      }
+    for (int u = 0; u < T; ++u) {
+      const int i = (tid + u * 256) * 4, r = i / D, d = i % D;
+      const float4 z = load4(ref + d), b = load4(b_s + r * LB + d), k = load4(ks + r * L + d), q = load4(rs + r * L + d);
+      const float4 p = r > 0 ? load4(b_s + (r - 1) * LB + d) : make_float4(0.f, 0.f, 0.f, 0.f);
+      put_split(xh + r * L + d, xl + r * L + d, make_float4(k.x * ex2(z.x - b.x), k.y * ex2(z.y - b.y), k.z * ex2(z.z - b.z), k.w * ex2(z.w - b.w)));
+      put_split(fh + r * L + d, fl + r * L + d, make_float4(q.x * ex2(p.x - z.x), q.y * ex2(p.y - z.y), q.z * ex2(p.z - z.z), q.w * ex2(p.w - z.w)));
     }
-#pragma unroll
-    for (int e = 0; e < 4; ++e) {
-      const int jl = jq + 4 * e;
-      if (jl > il) break;
-      const __nv_bfloat16 hi = __float2bfloat16(s[e]);
-      ah[i * LA + blk + jl] = hi;
-      al[i * LA + blk + jl] = __float2bfloat16(s[e] - __bfloat162float(hi));
-    }
-  }
-  // pairs in different blocks: rows of block I against all rows before it
-  for (int I = 1; I < C / 16; ++I) {
-    const float* ref = b_s + (16 * I - 1) * LB;
-    for (int x = tid * 4; x < 16 * (I + 1) * D; x += 1024) {
-      const int r = x / D, d = x % D;
-      const float4 z = load4(ref + d);
-      float4 f;
-      if (r < 16 * I) {
-        const float4 b = load4(b_s + r * LB + d), k = load4(ks + r * L + d);
-        f = make_float4(k.x * ex2(z.x - b.x), k.y * ex2(z.y - b.y), k.z * ex2(z.z - b.z), k.w * ex2(z.w - b.w));
-      } else {
-        const float4 b = load4(b_s + (r - 1) * LB + d), q = load4(rs + r * L + d);
-        f = make_float4(q.x * ex2(b.x - z.x), q.y * ex2(b.y - z.y), q.z * ex2(b.z - z.z), q.w * ex2(b.w - z.w));
+    {   // the bonus terms, four threads per row
+      const int i = tid >> 2;
+      float s = 0.0f;
+#pragma unroll 4
+      for (int d = (tid & 3) * 4; d < D; d += 16) {
+        const float4 r = load4(rs + i * L + d), k = load4(ks + i * L + d), u = load4(u_s + d);
+        s = fmaf(r.x * k.x, u.x, fmaf(r.y * k.y, u.y, fmaf(r.z * k.z, u.z, fmaf(r.w * k.w, u.w, s))));
       }
-      put_split(fh + r * L + d, fl + r * L + d, f);
+      s += __shfl_xor_sync(0xffffffffu, s, 1);
+      s += __shfl_xor_sync(0xffffffffu, s, 2);
+      if ((tid & 3) == 0) scratch[i] = s;
     }
     __syncthreads();
-    if (wid < I) {   // a warp per 16 x 16 block of scores
-      float acc[2][4] = {};
+    // a warp has 16 rows and 32 columns of the scores
+    const int i0 = (wid & 3) * 16, j0 = (wid >> 2) * 32;
+    float acc[4][4] = {};
+    if (j0 < i0 + 16) {
 #pragma unroll 2
       for (int k0 = 0; k0 < D; k0 += 16) {
-        uint32_t Ah[4], Al[4], Bh[4], Bl[4];
-        ldsm_a(Ah, fh, L, 16 * I, k0, lane);
-        ldsm_a(Al, fl, L, 16 * I, k0, lane);
-        ldsm_b(Bh, fh, L, k0, 16 * wid, lane);
-        ldsm_b(Bl, fl, L, k0, 16 * wid, lane);
+        uint32_t Ah[4], Al[4];
+        ldsm_a(Ah, fh, L, i0, k0, lane);
+        ldsm_a(Al, fl, L, i0, k0, lane);
 #pragma unroll
-        for (int t = 0; t < 2; ++t) {
-          mma_bf16(acc[t], Ah, Bh[2 * t], Bh[2 * t + 1]);
-          mma_bf16(acc[t], Ah, Bl[2 * t], Bl[2 * t + 1]);
-          mma_bf16(acc[t], Al, Bh[2 * t], Bh[2 * t + 1]);
+        for (int t = 0; t < 4; t += 2) {
+          if (j0 + t * 8 >= i0 + 16) break;
+          uint32_t Bh[4], Bl[4];
+          ldsm_b(Bh, xh, L, k0, j0 + t * 8, lane);
+          ldsm_b(Bl, xl, L, k0, j0 + t * 8, lane);
+#pragma unroll
+          for (int e = 0; e < 2; ++e) {
+            mma_bf16(acc[t + e], Ah, Bh[2 * e], Bh[2 * e + 1]);
+            mma_bf16(acc[t + e], Ah, Bl[2 * e], Bl[2 * e + 1]);
+            mma_bf16(acc[t + e], Al, Bh[2 * e], Bh[2 * e + 1]);
+          }
+        }
+      }
+    }
+    __syncthreads();
+#pragma unroll
+    for (int t = 0; t < 4; ++t)
+#pragma unroll
+      for (int f = 0; f < 2; ++f) {
+        const int i = i0 + (lane >> 2) + 8 * f, j = j0 + 8 * t + (lane & 3) * 2;
+        const float x = j < i ? acc[t][2 * f] : (j == i ? scratch[i] : 0.0f);
+        const float y = j + 1 < i ? acc[t][2 * f + 1] : (j + 1 == i ? scratch[i] : 0.0f);
+        uint32_t hi, lo;
+        split_bf16x2(x, y, hi, lo);
+        *reinterpret_cast<uint32_t*>(ah + i * LA + j) = hi;
+        *reinterpret_cast<uint32_t*>(al + i * LA + j) = lo;
+      }
+  } else {
+    for (int i = tid; i < C * LA / 4; i += 256) reinterpret_cast<uint2*>(ah)[i] = reinterpret_cast<uint2*>(al)[i] = make_uint2(0u, 0u);
+    __syncthreads();
+    // pairs inside a 16-row block: a thread has row i and the columns jq, jq + 4, ... up to i
+    {
+      const int blk = tid >> 6 << 4, il = (tid >> 2) & 15, jq = tid & 3, i = blk + il;
+      float s[4] = {0.f, 0.f, 0.f, 0.f};
+      const float* bi = b_s + (i - 1) * LB;
+#pragma unroll 2
+      for (int d = 0; d < D; d += 4) {
+        const float4 r = load4(rs + i * L + d), u = load4(u_s + d);
+        const float4 b = i > 0 ? load4(bi + d) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int jl = jq + 4 * e, j = blk + jl;
+          if (jl > il) break;
+          const float4 k = load4(ks + j * L + d);
+          float4 f = u;
+          if (jl < il) {
+            const float4 bj = load4(b_s + j * LB + d);
+            f = make_float4(ex2(b.x - bj.x), ex2(b.y - bj.y), ex2(b.z - bj.z), ex2(b.w - bj.w));
+          }
+          s[e] = fmaf(r.x * k.x, f.x, fmaf(r.y * k.y, f.y, fmaf(r.z * k.z, f.z, fmaf(r.w * k.w, f.w, s[e]))));
         }
       }
 #pragma unroll
-      for (int t = 0; t < 2; ++t)
-#pragma unroll
-        for (int f = 0; f < 2; ++f) {
-          const int i = 16 * I + (lane >> 2) + 8 * f, j = 16 * wid + 8 * t + (lane & 3) * 2;
-          uint32_t hi, lo;
-          split_bf16x2(acc[t][2 * f], acc[t][2 * f + 1], hi, lo);
-          *reinterpret_cast<uint32_t*>(ah + i * LA + j) = hi;
-          *reinterpret_cast<uint32_t*>(al + i * LA + j) = lo;
-        }
+      for (int e = 0; e < 4; ++e) {
+        const int jl = jq + 4 * e;
+        if (jl > il) break;
+        const __nv_bfloat16 hi = __float2bfloat16(s[e]);
+        ah[i * LA + blk + jl] = hi;
+        al[i * LA + blk + jl] = __float2bfloat16(s[e] - __bfloat162float(hi));
+      }
     }
-    __syncthreads();
+    // pairs in different blocks: rows of block I against all rows before it
+    for (int I = 1; I < C / 16; ++I) {
+      const float* ref = b_s + (16 * I - 1) * LB;
+      for (int x = tid * 4; x < 16 * (I + 1) * D; x += 1024) {
+        const int r = x / D, d = x % D;
+        const float4 z = load4(ref + d);
+        float4 f;
+        if (r < 16 * I) {
+          const float4 b = load4(b_s + r * LB + d), k = load4(ks + r * L + d);
+          f = make_float4(k.x * ex2(z.x - b.x), k.y * ex2(z.y - b.y), k.z * ex2(z.z - b.z), k.w * ex2(z.w - b.w));
+        } else {
+          const float4 b = load4(b_s + (r - 1) * LB + d), q = load4(rs + r * L + d);
+          f = make_float4(q.x * ex2(b.x - z.x), q.y * ex2(b.y - z.y), q.z * ex2(b.z - z.z), q.w * ex2(b.w - z.w));
+        }
+        put_split(fh + r * L + d, fl + r * L + d, f);
+      }
+      __syncthreads();
+      if (wid < I) {   // a warp per 16 x 16 block of scores
+        float acc[2][4] = {};
+#pragma unroll 2
+        for (int k0 = 0; k0 < D; k0 += 16) {
+          uint32_t Ah[4], Al[4], Bh[4], Bl[4];
+          ldsm_a(Ah, fh, L, 16 * I, k0, lane);
+          ldsm_a(Al, fl, L, 16 * I, k0, lane);
+          ldsm_b(Bh, fh, L, k0, 16 * wid, lane);
+          ldsm_b(Bl, fl, L, k0, 16 * wid, lane);
+#pragma unroll
+          for (int t = 0; t < 2; ++t) {
+            mma_bf16(acc[t], Ah, Bh[2 * t], Bh[2 * t + 1]);
+            mma_bf16(acc[t], Ah, Bl[2 * t], Bl[2 * t + 1]);
+            mma_bf16(acc[t], Al, Bh[2 * t], Bh[2 * t + 1]);
+          }
+        }
+#pragma unroll
+        for (int t = 0; t < 2; ++t)
+#pragma unroll
+          for (int f = 0; f < 2; ++f) {
+            const int i = 16 * I + (lane >> 2) + 8 * f, j = 16 * wid + 8 * t + (lane & 3) * 2;
+            uint32_t hi, lo;
+            split_bf16x2(acc[t][2 * f], acc[t][2 * f + 1], hi, lo);
+            *reinterpret_cast<uint32_t*>(ah + i * LA + j) = hi;
+            *reinterpret_cast<uint32_t*>(al + i * LA + j) = lo;
+          }
+      }
+      __syncthreads();
+    }
   }
   // r e^(b_(i-1)) takes the factors' place
 #pragma unroll

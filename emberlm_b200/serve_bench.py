@@ -1,5 +1,5 @@
-"""Serving throughput (prefill and greedy decode, batch 1) of the layer-list family beside the preset
-decoder closest to it, at equal width, depth, feed-forward width and vocabulary. Random weights.
+"""Serving throughput (prefill and greedy decode, batch 1) of the layer-list designs beside the preset
+decoder closest to them, at equal width, depth, (active) feed-forward width and vocabulary. Random weights.
 
   python -m emberlm_b200.serve_bench --size 0.6b            # one JSON line per model
   python -m emberlm_b200.serve_bench --size 1.7b --layers 4 # a short stack (per-kernel profiles)
@@ -58,6 +58,79 @@ def zutalix_shapes(cfg: dict, rank: int) -> dict:
             ff = lay["mlp"]["ff"]
             s |= {p + "norm2": [W], p + "norm2b": [W], p + "mlp.gate": [ff, W], p + "mlp.up": [ff, W], p + "mlp.down": [W, ff]}
     return s
+
+
+# (heads, dim, rot_dim, vdim, kv_rank, q_rank), (wkv heads, dim, rank); the active experts and the shared one
+# add up to the preset's feed-forward width
+DETATAR_SIZES = {"0.6b": ((16, 64, 32, 64, 256, 512), (16, 64, 64)), "1.7b": ((16, 128, 64, 128, 512, 1024), (32, 64, 64))}
+EXPERTS, IDENTITY, TOP, GROUPS = 32, 4, 4, (4, 3)
+
+
+def detatar_config(preset: dict, size: str, layers: int) -> dict:
+    """A Detatar of the preset's width, vocabulary and `layers` layers: one time-mixing layer in four, the rest
+    latent attention; a dense feed-forward in the first layer, mixtures of experts in the others."""
+    (H, D, DR, DV, R, Q), (RH, RD, _) = DETATAR_SIZES[size]
+    ff = preset["intermediate_size"]
+    lat = {"heads": H, "dim": D, "rot_dim": DR, "vdim": DV, "kv_rank": R, "q_rank": Q, "scale": (D + DR) ** -0.5, "rot": {"base": 1e6, "dims": DR}}
+    moe = {"kind": "moe", "expert": {"ff": ff // 6}, "shared": {"ff": ff - TOP * (ff // 6)},
+           "router": {"experts": EXPERTS, "identity": IDENTITY, "top": TOP, "groups": {"count": GROUPS[0], "keep": GROUPS[1]}}}
+    kinds = [("wkv", {"heads": RH, "dim": RD}) if i % 4 == 3 else ("latent_attention", lat) for i in range(layers)]
+    return {"architecture": "Detatar", "vocab": preset["vocab_size"], "width": preset["hidden_size"], "embedding": {"scale": 1.0},
+            "norm": {"eps": 1e-5, "groups": 2},
+            "layers": [{"type": t, "mixer": m, "mlp": moe if i else {"kind": "dense", "ff": ff}} for i, (t, m) in enumerate(kinds)]}
+
+
+def detatar_shapes(cfg: dict, rank: int) -> dict:
+    W = cfg["width"]
+    s = {"embed": [cfg["vocab"], W], "final.norm": [W], "head": [cfg["vocab"], W]}
+
+    def glu(p, ff):
+        return {p + "gate": [ff, W], p + "up": [ff, W], p + "down": [W, ff]}
+
+    for i, lay in enumerate(cfg["layers"]):
+        p, m, f = f"l{i}.", lay["mixer"], lay["mlp"]
+        q, H = p + "mix.", m["heads"]
+        s |= {p + "norm1": [W], p + "shift": [W], p + "rg1": [W, W], p + "rg1.b": [W], p + "rg2": [W, W], p + "rg2.b": [W]}
+        if lay["type"] == "latent_attention":
+            s |= {q + "dq": [m["q_rank"], W], q + "dq.norm": [m["q_rank"]], q + "uq": [H * (m["dim"] + m["rot_dim"]), m["q_rank"]],
+                  q + "dkv": [m["kv_rank"] + m["rot_dim"], W], q + "dkv.norm": [m["kv_rank"]], q + "uk": [H * m["dim"], m["kv_rank"]],
+                  q + "uv": [H * m["vdim"], m["kv_rank"]], q + "g": [H, W], q + "o": [W, H * m["vdim"]]}
+        else:
+            n = H * m["dim"]
+            s |= {q + "mu." + x: [W] for x in "rkvgw"} | {q + x: [n, W] for x in "rkvg"}
+            s |= {q + "w1": [rank, W], q + "w2": [n, rank], q + "w0": [n], q + "u": [H, m["dim"]], q + "norm": [n], q + "o": [W, n]}
+        if f["kind"] == "dense":
+            s |= glu(p + "mlp.", f["ff"])
+        else:
+            n = f["router"]["experts"] + f["router"]["identity"]
+            for e in range(f["router"]["experts"]):
+                s |= glu(f"{p}mlp.e{e}.", f["expert"]["ff"])
+            s |= {p + "mlp.router": [n, W], p + "mlp.correction": [n], p + "mlp.shared.sg": [1, W]} | glu(p + "mlp.shared.", f["shared"]["ff"])
+    return s
+
+
+def build_detatar(size: str, layers: int | None, max_seq: int, max_portion: int, dtype: str = "bf16"):
+    preset = E.PRESETS[SIZES[size][0]]
+    cfg = detatar_config(preset, size, layers or preset["num_hidden_layers"])
+    model = E.HybridModel(cfg, detatar_shapes(cfg, DETATAR_SIZES[size][1][2]), dtype)
+    dec = E.HybridDecoder(model, max_seq, max_portion)
+    gen = torch.Generator(device="cuda").manual_seed(1234)
+    views = dec.named_parameters()
+    streamed = 0.0   # parameters a token reads: experts by the share of them that are chosen, no embedding
+    for t in model.tensors:
+        name = t.name.decode()
+        v = views[name]
+        if t.is_matrix:
+            v.normal_(0.0, 0.02, generator=gen)
+        elif name.endswith(("correction", ".b", "w0", ".u")):
+            v.normal_(-1.0 if name.endswith("w0") else 0.0, 0.02 if name.endswith("correction") else 0.5, generator=gen)
+        elif name.endswith("shift") or ".mu." in name:
+            v.uniform_(0.0, 1.0, generator=gen)
+        else:
+            v.fill_(1.0)
+        share = TOP / (EXPERTS + IDENTITY) if ".mlp.e" in name else (0.0 if name == "embed" else 1.0)
+        streamed += share * t.rows * t.cols
+    return dec, sum(t.rows * t.cols for t in model.tensors), int(streamed)
 
 
 def build_zutalix(size: str, layers: int | None, max_seq: int, max_portion: int, dtype: str = "bf16"):
@@ -126,12 +199,16 @@ def run(size: str, layers: int | None = None, prompt_len: int = 4096, new_tokens
     rows = []
     for which in models:
         max_seq = prompt_len + new_tokens + 64
-        dec, params = (build_zutalix(size, layers, max_seq, prompt_len) if which == "zutalix" else build_preset(size, layers, max_seq))
+        preset = which == "preset"
+        if which == "detatar":
+            dec, params, streamed = build_detatar(size, layers, max_seq, prompt_len)
+        else:
+            dec, params = build_preset(size, layers, max_seq) if preset else build_zutalix(size, layers, max_seq, prompt_len)
+            streamed = params
         r = measure(dec, dec.vocab, prompt_len, new_tokens, steps, warmup, sampler)
-        bytes_per = 2 if which == "zutalix" else 4
-        rows.append({"model": f"zutalix-{size}" if which == "zutalix" else SIZES[size][0],
-                     "dtype": "bf16" if which == "zutalix" else "tf32 prefill, fp32 decode", "params": params, "prompt_len": prompt_len,
-                     "new_tokens": new_tokens, **r, "decode_weight_gbs": params * bytes_per / r["token_ms"] / 1e6})
+        rows.append({"model": SIZES[size][0] if preset else f"{which}-{size}", "dtype": "tf32 prefill, fp32 decode" if preset else "bf16",
+                     "params": params, "streamed_params": streamed, "prompt_len": prompt_len, "new_tokens": new_tokens, **r,
+                     "decode_weight_gbs": streamed * (4 if preset else 2) / r["token_ms"] / 1e6})
         del dec
         torch.cuda.empty_cache()
     return rows
@@ -145,7 +222,7 @@ def main():
     ap.add_argument("--new", type=int, default=128)
     ap.add_argument("--steps", type=int, default=5)
     ap.add_argument("--warmup", type=int, default=3)
-    ap.add_argument("--models", default="zutalix,preset")
+    ap.add_argument("--models", default="detatar,zutalix,preset")
     a = ap.parse_args()
     for r in run(a.size, a.layers, a.prompt, a.new, a.steps, a.warmup, tuple(a.models.split(","))):
         print(json.dumps(r), flush=True)

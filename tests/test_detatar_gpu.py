@@ -63,7 +63,7 @@ MIXERS = [dc.latent(4, 36, 16, 24, 40, 28), dc.latent(6, 64, 64, 64, 128, 96), d
           dc.latent(2, 16, 32, 256, 64, 48), dc.latent(1, 64, 128, 40, 1000, 8),
           dc.wkv(3, 40), dc.wkv(6, 64), dc.wkv(2, 128), dc.wkv(1, 17), dc.wkv(1, 200), dc.wkv(9, 1), dc.wkv(2, 32), dc.wkv(2, 100)]
 FFS = [dc.dense(150), dc.dense(9), dc.dense(256), dc.moe(5, 2, 36), dc.moe(8, 8, 16, shared=24), dc.moe(6, 3, 64, identity=3, groups=(3, 2), shared=9),
-       dc.moe(30, 6, 128, identity=2, groups=(8, 3)), dc.moe(1, 1, 20, identity=1), dc.moe(40, 1, 8, groups=(40, 1)), dc.moe(2, 2, 300, identity=2)]
+       dc.moe(30, 6, 128, identity=2, groups=(8, 3)), dc.moe(1, 1, 20, identity=1), dc.moe(40, 1, 8, groups=(40, 1)), dc.moe(270, 3, 8, identity=2, groups=(16, 4)), dc.moe(100, 5, 16, shared=8), dc.moe(2, 2, 300, identity=2)]
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
