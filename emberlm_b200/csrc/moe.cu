@@ -24,7 +24,8 @@ __global__ void __launch_bounds__(256) moe_clear_kernel(int32_t* count, int n) {
   for (int i = threadIdx.x; i < n; i += 256) count[i] = 0;
 }
 
-// One warp per row.
+// One warp per row. A row's place among its expert's rows is counted in shared memory first, so that the
+// counters in global memory see one addition per CTA and expert.
 __global__ void __launch_bounds__(256) moe_choose_kernel(const MoeArgs a, int64_t rows) {
   extern __shared__ float sm[];
   pdl_launch();
@@ -32,6 +33,9 @@ __global__ void __launch_bounds__(256) moe_choose_kernel(const MoeArgs a, int64_
   const int lane = threadIdx.x & 31, wid = threadIdx.x >> 5;
   const int per = a.outputs + route_scratch(a.outputs, a.groups);
   float* z = sm + wid * per;
+  int32_t* seen = reinterpret_cast<int32_t*>(sm + 8 * per);   // [experts] of this CTA, then where they start
+  for (int e = threadIdx.x; e < a.experts; e += 256) seen[e] = 0;
+  __syncthreads();
   const int64_t nw = static_cast<int64_t>(gridDim.x) * 8;
   for (int64_t r = static_cast<int64_t>(blockIdx.x) * 8 + wid; r < rows; r += nw) {
     __syncwarp();
@@ -40,9 +44,18 @@ __global__ void __launch_bounds__(256) moe_choose_kernel(const MoeArgs a, int64_
     route_token(z, a.correction, a.outputs, a.groups, a.keep, a.top, z + a.outputs, a.index + r * a.top, a.weight + r * a.top);
     if (lane < a.top) {
       const int e = a.index[r * a.top + lane];
-      if (e < a.experts) atomicAdd(&a.count[e], 1);
+      a.slot[r * a.top + lane] = e < a.experts ? atomicAdd(&seen[e], 1) : 0;
     }
   }
+  __syncthreads();
+  for (int e = threadIdx.x; e < a.experts; e += 256)
+    if (seen[e] > 0) seen[e] = atomicAdd(&a.count[e], seen[e]);
+  __syncthreads();
+  for (int64_t r = static_cast<int64_t>(blockIdx.x) * 8 + wid; r < rows; r += nw)
+    if (lane < a.top) {
+      const int e = a.index[r * a.top + lane];
+      if (e < a.experts) a.slot[r * a.top + lane] += seen[e];
+    }
 }
 
 // One CTA: first tile of every expert, the expert of every tile.
@@ -72,7 +85,7 @@ __global__ void __launch_bounds__(1024) moe_tiles_kernel(const MoeArgs a) {
   }
 }
 
-// One warp per chosen output: takes a slot and copies the row there.
+// One warp per chosen output: the row goes to its slot.
 template <typename T>
 __global__ void __launch_bounds__(256) moe_gather_kernel(const MoeArgs a, const T* __restrict__ h, int64_t ld_h, T* __restrict__ xe, int width,
                                                          int64_t n) {
@@ -82,9 +95,8 @@ __global__ void __launch_bounds__(256) moe_gather_kernel(const MoeArgs a, const 
   const int64_t nw = static_cast<int64_t>(gridDim.x) * 8;
   for (int64_t i = (static_cast<int64_t>(blockIdx.x) * 256 + threadIdx.x) >> 5; i < n; i += nw) {
     const int e = a.index[i];
-    int slot = -1;
-    if (e < a.experts && lane == 0) slot = atomicAdd(&a.count[a.experts + e], 1);
-    slot = __shfl_sync(0xffffffffu, slot, 0);
+    const int slot = e < a.experts ? a.count[a.experts + e] + a.slot[i] : -1;
+    __syncwarp();   // every lane has read the place before it becomes the slot
     if (lane == 0) a.slot[i] = slot;
     if (slot < 0) continue;
     const T* src = h + i / a.top * ld_h;
@@ -205,12 +217,13 @@ __global__ void __launch_bounds__(256)
 int moe_route(const MoeArgs& a, int64_t rows, cudaStream_t s) {
   CTDK_REQUIRE(a.outputs <= 1024 && a.top <= 32 && a.outputs % a.groups == 0, "moe: more than 1024 outputs or 32 choices");
   TRY_LAUNCH("moe clear", moe_clear_kernel, (1), 256, 0, a.count, 2 * a.experts);
-  const size_t smem = static_cast<size_t>(8) * (a.outputs + route_scratch(a.outputs, a.groups)) * 4;
+  const size_t smem = (static_cast<size_t>(8) * (a.outputs + route_scratch(a.outputs, a.groups)) + a.experts) * 4;
   if (smem > 48 * 1024) {
     const cudaError_t e = cudaFuncSetAttribute(moe_choose_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
     if (e != cudaSuccess) return fail(CTDK_ELAUNCH, "moe: %s", cudaGetErrorString(e));
   }
-  TRY_LAUNCH("moe choose", moe_choose_kernel, (row_grid(rows, 8)), 256, smem, a, rows);
+  const int64_t ctas = (rows + 7) / 8;
+  TRY_LAUNCH("moe choose", moe_choose_kernel, (static_cast<unsigned>(ctas < sm_count() ? ctas : sm_count())), 256, smem, a, rows);
   TRY_LAUNCH("moe tiles", moe_tiles_kernel, (1), 1024, 0, a);
   return CTDK_OK;
 }

@@ -132,7 +132,7 @@ struct MoeArgs {
   int experts = 0, outputs = 0, top = 0, groups = 1, keep = 1;
   int32_t *index = nullptr, *slot = nullptr;    // [rows][top]
   float* weight = nullptr;                      // [rows][top]
-  int32_t* count = nullptr;                     // [2][experts]: rows per expert, then slots handed out
+  int32_t* count = nullptr;                     // [2][experts]: rows per expert, first slot of each
   int32_t* tiles = nullptr;                     // [max_tiles + 2]: expert per tile, number of tiles, number of slots
   int max_tiles = 0;
 };

@@ -39,7 +39,7 @@ __device__ __forceinline__ void vstore(U* p, const Vec<V>& r) {
 // rows in front of its run are formed again (h needs one row back, a mix of shifted rows two). Columns are
 // dealt so that a warp's columns lie in one group: wpg warps per group.
 template <typename T, int V>
-__global__ void __launch_bounds__(256) shift_norm_kernel(const ShiftNormArgs<T> a, int64_t rows, int run, int wpg) {
+__global__ void __launch_bounds__(256, 4) shift_norm_kernel(const ShiftNormArgs<T> a, int64_t rows, int run, int wpg) {
   extern __shared__ __align__(16) float sm[];
   const int W = a.width, gs = W / a.groups, lane = threadIdx.x & 31, wid = threadIdx.x >> 5;
   const int Wp = (W + 3) & ~3;
@@ -227,8 +227,9 @@ int launch_shift_norm(const ShiftNormArgs<T>& a, int64_t rows, cudaStream_t s) {
   const int wpg = a.groups >= 8 ? 1 : 8 / a.groups;
   const int arrays = a.n_mix > 0 ? 3 : (a.shift != nullptr ? 2 : 1);
   const size_t smem = (static_cast<size_t>((a.width + 3) / 4 * 4) * arrays + 2 * static_cast<size_t>(a.groups) * wpg) * 4;
-  const int64_t run64 = rows / (static_cast<int64_t>(sm_count()) * 3);
-  const int run = a.gather != nullptr || run64 < 1 ? 1 : (run64 > 16 ? 16 : static_cast<int>(run64));
+  const int64_t slots = static_cast<int64_t>(sm_count()) * 4;   // CTAs that run at once
+  const int64_t run64 = rows >= slots / 2 ? (rows + slots - 1) / slots : 1;
+  const int run = a.gather != nullptr ? 1 : (run64 > 16 ? 16 : static_cast<int>(run64));
   if (smem > 48 * 1024) {
     const cudaError_t e = cudaFuncSetAttribute(shift_norm_kernel<T, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
     if (e != cudaSuccess) return fail(CTDK_ELAUNCH, "shift norm: %s", cudaGetErrorString(e));

@@ -5,11 +5,12 @@
 //   o_i = (r_i e^(b_(i-1)))^T S + sum_(j < i) (r_i . k_j e^(b_(i-1) - b_j)) v_j + (r_i . u k_i) v_i
 //   S'  = diag(e^(b_last)) S + sum_j (k_j e^(b_last - b_j)) v_j^T
 // Three kernels: every chunk's own contribution to the state, a scan over the chunks in fp32, and the
-// outputs with the norm over each head and the output gate. The pair factors e^(b_(i-1) - b_j) are split at
-// the running sum of the chunk's middle row while the chunk's decays stay above 2^-kReach in every channel
-// (then both factors stay within fp32 and bfloat16 range). Otherwise no exponent is ever positive: between
-// 16-row blocks both factors are taken relative to the running sum in front of the later block, inside a
-// block the difference is formed per pair. r, k, v are bfloat16 (projections); whatever carries a decay is split into
+// outputs with the norm over each head and the output gate. The pair factors e^(b_(i-1) - b_j) are split:
+// between the chunk's halves at the running sum of the boundary, inside a half at that of its middle row,
+// provided that no 16 rows decay by more than 2^-kReach in any channel (then both factors stay within fp32
+// and bfloat16 range). Otherwise no exponent is ever positive: between 16-row blocks both factors are taken
+// relative to the running sum in front of the later block, inside a block the difference is formed per pair.
+// r, k, v are bfloat16 (projections); whatever carries a decay is split into
 // a bfloat16 sum of two terms before it meets a tensor core (16 mantissa bits, fp32 sums), the state itself
 // is carried in fp32. mma.sync m16n8k16.
 #include <cuda_bf16.h>
@@ -275,35 +276,24 @@ __global__ void __launch_bounds__(256) wkv_out_kernel(const WkvArgs a) {
   running_sums<D, LB>(b_s, scratch);
 
   float reach = 0.0f;
-  for (int d = tid; d < D; d += 256) reach = fminf(reach, b_s[(C - 1) * LB + d]);
+  for (int x = tid; x < 4 * D; x += 256) {
+    const int d = x % D, q = x / D;
+    reach = fminf(reach, b_s[(16 * q + 15) * LB + d] - (q > 0 ? b_s[(16 * q - 1) * LB + d] : 0.0f));
+  }
   if (__syncthreads_or(reach < -kReach) == 0) {
     __nv_bfloat16 *xh = ah, *xl = al;   // [C][L] key factors, where the scores will be
-    const float* ref = b_s + (C / 2 - 1) * LB;
-#pragma unroll
-    for (int u = 0; u < T; ++u) {
-      const int i = (tid + u * 256) * 4, r = i / D, d = i % D;
-      const float4 z = load4(ref + d), b = load4(b_s + r * LB + d), k = load4(ks + r * L + d), q = load4(rs + r * L + d);
-      const float4 p = r > 0 ? load4(b_s + (r - 1) * LB + d) : make_float4(0.f, 0.f, 0.f, 0.f);
-      put_split(xh + r * L + d, xl + r * L + d, make_float4(k.x * ex2(z.x - b.x), k.y * ex2(z.y - b.y), k.z * ex2(z.z - b.z), k.w * ex2(z.w - b.w)));
+    auto query_factor = [&](int r, int d, const float4& z) {
+      const float4 q = load4(rs + r * L + d), p = r > 0 ? load4(b_s + (r - 1) * LB + d) : make_float4(0.f, 0.f, 0.f, 0.f);
       put_split(fh + r * L + d, fl + r * L + d, make_float4(q.x * ex2(p.x - z.x), q.y * ex2(p.y - z.y), q.z * ex2(p.z - z.z), q.w * ex2(p.w - z.w)));
-    }
-    {   // the bonus terms, four threads per row
-      const int i = tid >> 2;
-      float s = 0.0f;
-#pragma unroll 4
-      for (int d = (tid & 3) * 4; d < D; d += 16) {
-        const float4 r = load4(rs + i * L + d), k = load4(ks + i * L + d), u = load4(u_s + d);
-        s = fmaf(r.x * k.x, u.x, fmaf(r.y * k.y, u.y, fmaf(r.z * k.z, u.z, fmaf(r.w * k.w, u.w, s))));
-      }
-      s += __shfl_xor_sync(0xffffffffu, s, 1);
-      s += __shfl_xor_sync(0xffffffffu, s, 2);
-      if ((tid & 3) == 0) scratch[i] = s;
-    }
-    __syncthreads();
-    // a warp has 16 rows and 32 columns of the scores
+    };
+    auto key_factor = [&](int r, int d, const float4& z) {
+      const float4 k = load4(ks + r * L + d), b = load4(b_s + r * LB + d);
+      put_split(xh + r * L + d, xl + r * L + d, make_float4(k.x * ex2(z.x - b.x), k.y * ex2(z.y - b.y), k.z * ex2(z.z - b.z), k.w * ex2(z.w - b.w)));
+    };
+    // a warp has 16 rows and 32 columns of the scores; tiles above the diagonal are left out
     const int i0 = (wid & 3) * 16, j0 = (wid >> 2) * 32;
     float acc[4][4] = {};
-    if (j0 < i0 + 16) {
+    auto scores = [&] {
 #pragma unroll 2
       for (int k0 = 0; k0 < D; k0 += 16) {
         uint32_t Ah[4], Al[4];
@@ -323,7 +313,38 @@ __global__ void __launch_bounds__(256) wkv_out_kernel(const WkvArgs a) {
           }
         }
       }
+    };
+#pragma unroll
+    for (int u = 0; u < T; ++u) {   // inside the halves
+      const int i = (tid + u * 256) * 4, r = i / D, d = i % D;
+      const float4 z = load4(b_s + ((r & 32) + 15) * LB + d);
+      query_factor(r, d, z);
+      key_factor(r, d, z);
     }
+    {   // the bonus terms, four threads per row
+      const int i = tid >> 2;
+      float s = 0.0f;
+#pragma unroll 4
+      for (int d = (tid & 3) * 4; d < D; d += 16) {
+        const float4 r = load4(rs + i * L + d), k = load4(ks + i * L + d), u = load4(u_s + d);
+        s = fmaf(r.x * k.x, u.x, fmaf(r.y * k.y, u.y, fmaf(r.z * k.z, u.z, fmaf(r.w * k.w, u.w, s))));
+      }
+      s += __shfl_xor_sync(0xffffffffu, s, 1);
+      s += __shfl_xor_sync(0xffffffffu, s, 2);
+      if ((tid & 3) == 0) scratch[i] = s;
+    }
+    __syncthreads();
+    if ((i0 & 32) == j0) scores();
+    __syncthreads();
+#pragma unroll
+    for (int u = 0; u < T / 2; ++u) {   // queries of the second half, keys of the first
+      const int i = (tid + u * 256) * 4, r = i / D, d = i % D;
+      const float4 z = load4(b_s + 31 * LB + d);
+      query_factor(r + 32, d, z);
+      key_factor(r, d, z);
+    }
+    __syncthreads();
+    if (i0 >= 32 && j0 == 0) scores();
     __syncthreads();
 #pragma unroll
     for (int t = 0; t < 4; ++t)

@@ -97,7 +97,7 @@ def test_each_feed_forward_alone(case, dtype):
         r = f["router"]
         gap = np.array([od.route_margin(w["l0.mlp.router"].astype(float) @ x, w["l0.mlp.correction"].astype(float), r["top"], r.get("groups"))
                         for x in h])
-        keep = gap > (1e-2 if dtype == "bf16" else 1e-5)
+        keep = gap > ((1e-2 if r["experts"] < 64 else 2e-3) if dtype == "bf16" else 1e-5)   # scores shrink with their number
         assert keep.sum() > 100
     dec = decoder(cfg, w, dtype)
     got, want = share(cfg, w, dec, t)
