@@ -5,6 +5,14 @@
 // launch; every phase deals its rows (or its heads) to the CTAs, and while a CTA waits at a barrier
 // the weights of a coming phase are on their way into L2. Vectors between phases are fp32; every CTA
 // stages (and norms) its own copy. All waits are bounded.
+//
+// Phases of the parallel arrangement (kStageList; a kernel of its own with one CTA of 16 warps per SM) are
+// more uniform: operations that fill the staged vector, up to six products reading parts of it, and the
+// items of a mixer (recurrent heads, ranges of the latent cache). The feed-forward's products ride along in
+// the mixer's phases: per latent-attention layer
+//   [norm, shift + every projection] | [queries, choice of the experts + their gate / up rows]
+//   | [queries against the cache rows + down rows] | [ranges of the cache] | [merge, values] | [output]
+// and for time mixing [norm, shift, mixes + projections] | [state + experts' rows] | [output + down rows].
 #include <cfloat>
 #include <type_traits>
 

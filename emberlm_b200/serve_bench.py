@@ -63,7 +63,7 @@ def zutalix_shapes(cfg: dict, rank: int) -> dict:
 # (heads, dim, rot_dim, vdim, kv_rank, q_rank), (wkv heads, dim, rank); the active experts and the shared one
 # add up to the preset's feed-forward width
 DETATAR_SIZES = {"0.6b": ((16, 64, 32, 64, 256, 512), (16, 64, 64)), "1.7b": ((16, 128, 64, 128, 512, 1024), (32, 64, 64))}
-EXPERTS, IDENTITY, TOP, GROUPS = 32, 4, 4, (4, 3)
+EXPERTS, IDENTITY, TOP, GROUPS = 40, 8, 4, (8, 5)
 
 
 def detatar_config(preset: dict, size: str, layers: int) -> dict:

@@ -554,7 +554,9 @@ int ctdk_decode_reset(void* decoder, void* stream);
  * Layer-list decoders ("hybrid" family). The model is described by its config.json: a list of layers,
  * each with one or two mixer branches (chunked attention with tied keys and values, lightning linear
  * attention, the delta rule with per-channel decay) and an optional clamped GLU, RMS norms before and
- * after every sublayer, an untied head. A handle from ctdk_hybrid_open owns the parsed description
+ * after every sublayer, an untied head ("Zutalix"); or each with one mixer (latent attention, time mixing
+ * with a bonus) behind a token shift, beside a GLU or a mixture of experts, both reading one grouped norm
+ * and each behind a sigmoid gate, layers that use another's weights ("Detatar"). A handle from ctdk_hybrid_open owns the parsed description
  * (host memory only); it names every tensor and where it lies in the parameter arena, and makes
  * decoders that all ctdk_decode_* calls above accept.
  *   config_json   text of config.json;
