@@ -17,6 +17,7 @@
 // checking; the epilogue predicates stores. Every mbarrier wait is bounded.
 #include <cuda.h>
 #include <cudaTypedefs.h>
+#include <cuda_bf16.h>
 
 #include <cstdlib>
 #include <mutex>
@@ -56,7 +57,19 @@ struct GemmArgs {
   // tiles[i], and only the first tiles[max_tiles] m-blocks exist. Null: one group.
   const int32_t* tiles = nullptr;
   int max_tiles = 0, n_pitch = 0;
+  // bfloat16 outputs (kOutBf16, kOutGlu)
+  __nv_bfloat16* out16 = nullptr;
+  int up_row = 0;   // kOutGlu: rows of B between a gate row and its up row; N counts pairs
 };
+
+// What the epilogue writes: fp32 sums, the same as bfloat16, or bfloat16 silu(gate) up of the two halves of
+// a tile's columns (the first half holds gate rows of B, the second their up rows).
+enum GemmOut { kOutF32 = 0, kOutBf16 = 1, kOutGlu = 2 };
+
+__device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
+  const __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
+  return *reinterpret_cast<const uint32_t*>(&v);
+}
 
 // Instruction descriptor: D=F32 (bit 4), A,B format at bits 7 and 10 (kind::tf32: 2 = TF32;
 // kind::f16: 1 = BF16), major-ness bits 15/16 (0 = K-major, 1 = MN-major), N>>3 at bit 17, M>>4 at bit 24.
@@ -79,11 +92,13 @@ __device__ __forceinline__ void tile_coords(int tile, int m_blocks, int n_blocks
 
 // BF16: bfloat16 operands, both K-major. A stage row is 128 bytes either way and an MMA takes 32 of
 // them (8 TF32 or 16 bfloat16 values), so tiles, swizzle and descriptors are the same bytes.
-template <int BN, bool A_MN, bool B_MN, bool BF16>
+template <int BN, bool A_MN, bool B_MN, bool BF16, int OUT>
 __global__ void __launch_bounds__(kThreads, 1)
     gemm_tf32_kernel(const __grid_constant__ CUtensorMap tmA,
                      const __grid_constant__ CUtensorMap tmB, const GemmArgs args) {
   static_assert(!BF16 || (!A_MN && !B_MN), "bfloat16 operands are K-major");
+  static_assert(OUT == kOutF32 || BF16, "bfloat16 outputs go with bfloat16 operands");
+  constexpr int TN = OUT == kOutGlu ? BN / 2 : BN;   // output columns of a tile
   using C = Cfg<BN>;
   constexpr int kElems = BF16 ? BKH : BK;   // values of a stage row
   extern __shared__ unsigned char smem_raw[];
@@ -100,7 +115,7 @@ __global__ void __launch_bounds__(kThreads, 1)
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const bool grouped = BF16 && args.tiles != nullptr;
   const int m_blocks = grouped ? args.tiles[args.max_tiles] : (args.M + BM - 1) / BM;
-  const int n_blocks = (args.N + BN - 1) / BN;
+  const int n_blocks = (args.N + TN - 1) / TN;
   const int num_tiles = m_blocks * n_blocks;
   const int k_blocks = (args.K + kElems - 1) / kElems;
   const int num_units = num_tiles * args.splits;  // unit u: tile u % num_tiles, k-range u / num_tiles
@@ -137,7 +152,7 @@ __global__ void __launch_bounds__(kThreads, 1)
       for (int unit = blockIdx.x; unit < num_units && ok; unit += gridDim.x) {
         int mb, nb;
         tile_coords(unit % num_tiles, m_blocks, n_blocks, mb, nb);
-        const int m0 = mb * BM, n0 = nb * BN;
+        const int m0 = mb * BM, n0 = nb * TN;
         const int b_row = grouped ? n0 + args.tiles[mb] * args.n_pitch : n0;
         const int split = unit / num_tiles;
         const int kb0 = static_cast<int>(static_cast<int64_t>(split) * k_blocks / args.splits);
@@ -164,6 +179,7 @@ __global__ void __launch_bounds__(kThreads, 1)
               tma_load_2d(b_dst + c * kChunkBytes, &tmB, &full[s], n0 + 32 * c, k0);
           } else {
             tma_load_2d(b_dst, &tmB, &full[s], k0, b_row);
+            if (OUT == kOutGlu) tma_load_2d(b_dst + C::kBTileBytes / 2, &tmB, &full[s], k0, b_row + args.up_row);
           }
           if (++s == C::kStages) {
             s = 0;
@@ -254,8 +270,37 @@ __global__ void __launch_bounds__(kThreads, 1)
       const float* xrow = args.aux != nullptr ? args.aux + grow * args.ldc : nullptr;
       const uint32_t t_row = tmem_base + static_cast<uint32_t>(acc * BN) +
                              (static_cast<uint32_t>(q * 32) << 16);
+      if constexpr (OUT != kOutF32) {
+        __nv_bfloat16* orow = args.out16 + grow * args.ldc;
 #pragma unroll 1
-      for (int ch = 0; ch < BN / 32; ++ch) {
+        for (int ch = 0; ch < TN / 32; ++ch) {
+          const int col0 = nb * TN + ch * 32;
+          if (col0 >= args.N) break;  // warp-uniform
+          float v[32];
+          tmem_ld_32x32(t_row + static_cast<uint32_t>(ch * 32), v);
+          if constexpr (OUT == kOutGlu) {
+            float u[32];
+            tmem_ld_32x32(t_row + static_cast<uint32_t>(TN + ch * 32), u);
+#pragma unroll
+            for (int j = 0; j < 32; ++j) v[j] = v[j] * __fdividef(1.0f, 1.0f + expf(-v[j])) * u[j];
+          }
+          if (row_ok) {
+            if (args.vec_ok && col0 + 32 <= args.N) {
+#pragma unroll
+              for (int j = 0; j < 32; j += 8)
+                *reinterpret_cast<uint4*>(orow + col0 + j) = make_uint4(pack_bf16(v[j], v[j + 1]), pack_bf16(v[j + 2], v[j + 3]),
+                                                                        pack_bf16(v[j + 4], v[j + 5]), pack_bf16(v[j + 6], v[j + 7]));
+            } else {
+#pragma unroll
+              for (int j = 0; j < 32; ++j)
+                if (col0 + j < args.N) orow[col0 + j] = __float2bfloat16(v[j]);
+            }
+          }
+          __syncwarp();  // tcgen05.ld is warp-collective: reconverge before the next chunk
+        }
+      }
+#pragma unroll 1
+      for (int ch = 0; OUT == kOutF32 && ch < BN / 32; ++ch) {
         const int col0 = nb * BN + ch * 32;
         if (col0 >= args.N) break;  // warp-uniform
         float v[32];
@@ -412,14 +457,15 @@ int encode_tensor_map(CUtensorMap* map, const float* base, int rank, const uint6
 
 namespace {
 
-template <int BN, bool A_MN, bool B_MN, bool BF16 = false>
+template <int BN, bool A_MN, bool B_MN, bool BF16 = false, int OUT = kOutF32>
 int launch(const CUtensorMap& ta, const CUtensorMap& tb, const GemmArgs& args,
            cudaStream_t stream) {
   using C = Cfg<BN>;
   static bool attr_set[64] = {false};
   int dev = 0;
   cudaGetDevice(&dev);
-  auto* kern = gemm_tf32_kernel<BN, A_MN, B_MN, BF16>;
+  auto* kern = gemm_tf32_kernel<BN, A_MN, B_MN, BF16, OUT>;
+  constexpr int TN = OUT == kOutGlu ? BN / 2 : BN;
   if (dev >= 0 && dev < 64 && !attr_set[dev]) {
     cudaError_t e =
         cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, C::kSmemBytes);
@@ -428,7 +474,7 @@ int launch(const CUtensorMap& ta, const CUtensorMap& tb, const GemmArgs& args,
                   C::kSmemBytes, cudaGetErrorString(e));
     attr_set[dev] = true;
   }
-  const int m_blocks = args.tiles != nullptr ? args.max_tiles : (args.M + BM - 1) / BM, n_blocks = (args.N + BN - 1) / BN;
+  const int m_blocks = args.tiles != nullptr ? args.max_tiles : (args.M + BM - 1) / BM, n_blocks = (args.N + TN - 1) / TN;
   const int tiles = m_blocks * n_blocks * args.splits;
   const int sms = sm_count();
   const int grid = tiles < sms ? tiles : sms;
@@ -778,34 +824,49 @@ int gemm_bf16_tcgen05(const void* A, const void* B, float* Cp, int64_t M, int64_
   }
 }
 
-// Grouped form: C[m-block i of 128 rows] = A[m-block i] B[tiles[i]]^T for the first tiles[max_tiles] m-blocks;
-// group g's N rows of B start at row g * n_pitch. tiles lies in device memory.
-int gemm_bf16_grouped(const void* A, int64_t lda, const void* B, int64_t ldb, int64_t n_pitch, float* Cp, int64_t ldc, int N, int K, int groups,
-                      const int32_t* tiles, int max_tiles, cudaStream_t stream) {
+namespace {
+
+template <int OUT>
+int launch_out16(int bn, const CUtensorMap& ta, const CUtensorMap& tb, const GemmArgs& args, cudaStream_t stream) {
+  switch (bn) {
+    case 64: return launch<64, false, false, true, OUT>(ta, tb, args, stream);
+    case 128: return launch<128, false, false, true, OUT>(ta, tb, args, stream);
+    default: return launch<256, false, false, true, OUT>(ta, tb, args, stream);
+  }
+}
+
+}  // namespace
+
+// C (bfloat16) = A B^T with bfloat16 operands, all pitches multiples of 8. up_row > 0: C = silu(gate) up with
+// N gate rows of B and their up rows up_row rows further. tiles != null (device memory): the grouped form,
+// C[m-block i of 128 rows] = A[m-block i] B[tiles[i]]^T for the first tiles[max_tiles] m-blocks, with group
+// g's rows of B from g * n_pitch on; M is then max_tiles * 128.
+int gemm_bf16_out16(const void* A, int64_t lda, const void* B, int64_t ldb, __nv_bfloat16* Cp, int64_t ldc, int64_t M, int N, int K, int up_row,
+                    const int32_t* tiles, int max_tiles, int64_t n_pitch, int groups, cudaStream_t stream) {
   auto a16 = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15u) == 0; };
-  CTDK_REQUIRE(a16(A) && a16(B) && (lda & 7) == 0 && (ldb & 7) == 0, "gemm_bf16_grouped: operands must be 16-byte aligned");
-  CTDK_REQUIRE(N >= 8 && K >= 1 && groups >= 1 && max_tiles >= 1 && n_pitch * groups <= INT32_MAX && n_pitch >= N, "gemm_bf16_grouped: bad shape");
-  const int bn = N >= 256 ? 256 : (N > 64 ? 128 : 64);
-  const int64_t M = static_cast<int64_t>(max_tiles) * BM;
-  CTDK_REQUIRE(M <= INT32_MAX, "gemm_bf16_grouped: too many rows");
+  CTDK_REQUIRE(a16(A) && a16(B) && a16(Cp) && (lda & 7) == 0 && (ldb & 7) == 0 && (ldc & 7) == 0, "gemm_bf16_out16: operands must be 16-byte aligned");
+  const int64_t b_rows = tiles != nullptr ? n_pitch * groups : up_row + N;
+  CTDK_REQUIRE(M >= 1 && N >= 1 && K >= 1 && M <= INT32_MAX && b_rows <= INT32_MAX && (tiles == nullptr || n_pitch >= up_row + N),
+               "gemm_bf16_out16: bad shape");
+  const int cols = up_row > 0 ? 2 * N : N;   // accumulator columns of all tiles
+  const int bn = cols >= 256 ? 256 : (cols > 64 ? 128 : 64);
   const uint64_t da[2] = {static_cast<uint64_t>(K), static_cast<uint64_t>(M)}, sa[1] = {static_cast<uint64_t>(lda) * 2};
-  const uint64_t db[2] = {static_cast<uint64_t>(K), static_cast<uint64_t>(n_pitch * groups)}, sb[1] = {static_cast<uint64_t>(ldb) * 2};
-  const uint32_t box_a[2] = {static_cast<uint32_t>(BKH), static_cast<uint32_t>(BM)}, box_b[2] = {static_cast<uint32_t>(BKH), static_cast<uint32_t>(bn)};
+  const uint64_t db[2] = {static_cast<uint64_t>(K), static_cast<uint64_t>(b_rows)}, sb[1] = {static_cast<uint64_t>(ldb) * 2};
+  const uint32_t box_a[2] = {static_cast<uint32_t>(BKH), static_cast<uint32_t>(BM)};
+  const uint32_t box_b[2] = {static_cast<uint32_t>(BKH), static_cast<uint32_t>(up_row > 0 ? bn / 2 : bn)};
   CUtensorMap ta, tb;
   int rc = encode_tensor_map_bf16(&ta, A, 2, da, sa, box_a);
   if (rc == CTDK_OK) rc = encode_tensor_map_bf16(&tb, B, 2, db, sb, box_b);
   if (rc != CTDK_OK) return rc;
   int* st = device_status_word();
   if (st == nullptr) return fail(CTDK_ELAUNCH, "gemm: no status word");
-  GemmArgs args{Cp, nullptr, ldc, static_cast<int>(M), N, K, CTDK_EPI_STORE, (a16(Cp) && (ldc & 3) == 0) ? 1 : 0, 1, st};
+  GemmArgs args{nullptr, nullptr, ldc, static_cast<int>(M), N, K, CTDK_EPI_STORE, 1, 1, st};
   args.tiles = tiles;
   args.max_tiles = max_tiles;
   args.n_pitch = static_cast<int>(n_pitch);
-  switch (bn) {
-    case 64: return launch<64, false, false, true>(ta, tb, args, stream);
-    case 128: return launch<128, false, false, true>(ta, tb, args, stream);
-    default: return launch<256, false, false, true>(ta, tb, args, stream);
-  }
+  args.out16 = Cp;
+  args.up_row = up_row;
+  return up_row > 0 ? launch_out16<kOutGlu>(bn, ta, tb, args, stream) : launch_out16<kOutBf16>(bn, ta, tb, args, stream);
 }
 
 // Near-fp32 GEMM (3xTF32 split). Returns 1 (not eligible) until the split kernel is built,

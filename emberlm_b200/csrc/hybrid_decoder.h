@@ -105,9 +105,9 @@ struct HybridDecoder : DecoderBase {
   // parallel arrangement (hybrid_parallel.cu)
   float *x2, *side, *shift_state, *shift_next;
   T *shifted, *mixes, *low_q, *q_rot, *kv_heads;
-  float *q_up, *kv_up, *moe_weight, *expert_gu, *expert_out, *shared_out;
+  float *q_up, *moe_weight, *expert_gu, *shared_out;
   int32_t *moe_index, *moe_slot, *moe_count, *moe_tiles;
-  T *expert_in, *expert_act;
+  T *expert_in, *expert_act, *expert_out;
   float *th, *tside, *tq, *tq_abs, *tegu;
   int64_t tside_pitch = 0;   // two side projections, alternating from layer to layer
   int carve_parallel(Bump& b);

@@ -12,6 +12,10 @@
 #include "moe_route.cuh"
 
 namespace ctdk {
+
+int gemm_bf16_out16(const void* A, int64_t lda, const void* B, int64_t ldb, __nv_bfloat16* C, int64_t ldc, int64_t M, int N, int K, int up_row,
+                    const int32_t* tiles, int max_tiles, int64_t n_pitch, int groups, cudaStream_t stream);
+
 namespace hybrid {
 
 template <typename T>
@@ -102,7 +106,6 @@ int HybridDecoder<T>::carve_parallel(Bump& b) {
   low_q = typed(R * low);
   q_up = b.floats(R * q_up_n);
   q_rot = typed(R * q_rot_n);
-  kv_up = b.floats(exact ? 0 : max_seq * kv_n);
   kv_heads = typed(max_seq * kv_n);
   act = typed(R * act_n);
   moe_index = ints(R * choices);
@@ -111,9 +114,9 @@ int HybridDecoder<T>::carve_parallel(Bump& b) {
   moe_count = ints(counts);
   moe_tiles = ints(tiles);
   expert_in = typed(slots * m.ldw);
-  expert_gu = b.floats(gu_n);
+  expert_gu = b.floats(exact ? gu_n : 0);
   expert_act = typed(ea_n);
-  expert_out = b.floats(slots * W);
+  expert_out = typed(slots * m.ldw);
   shared_out = b.floats(shared ? R * W : 0);
   want_dev = ints(R);
 
@@ -381,8 +384,7 @@ int HybridDecoder<float>::kv_rows(const float* cache, const float* w, int64_t ro
 template <>
 int HybridDecoder<__nv_bfloat16>::kv_rows(const __nv_bfloat16* cache, const __nv_bfloat16* w, int64_t rows, int64_t n, int64_t K, int64_t lda,
                                           int64_t ldw, cudaStream_t s) {
-  DTRY(gemm_rows(cache, w, kv_up, rows, n, K, lda, ldw, n, s));
-  return cast_rows(kv_up, n, kv_heads, n, rows, static_cast<int>(n), s);
+  return gemm_bf16_out16(cache, lda, w, ldw, kv_heads, n, rows, static_cast<int>(n), static_cast<int>(K), 0, nullptr, 0, 0, 1, s);
 }
 template <>
 int HybridDecoder<float>::latent_attention(const LatentArgs<float>& a, int64_t pos, int64_t n, cudaStream_t s) {
@@ -525,13 +527,9 @@ int HybridDecoder<T>::feed_forward_rows(const Layer& L, int64_t n, cudaStream_t 
   a.max_tiles = static_cast<int>(moe_max_tiles(n, e.experts, e.top));
   DTRY(moe_route(a, n, s));
   DTRY(moe_gather(a, h, m.ldw, expert_in, m.width, n, s));
-  const int64_t slots = static_cast<int64_t>(a.max_tiles) * kMoeTile;
-  DTRY(grouped_gemm(expert_in, m.ldw, at<T>(e.w_gu), m.ldw, 2 * e.effp, expert_gu, 2 * e.effp, 2 * e.effp, m.width, e.experts, a.tiles,
-                    a.max_tiles, s));
-  DTRY(glu_rows(expert_gu, 2 * e.effp, expert_act, e.effp, slots, e.effp, Glu::kSilu, a.tiles + a.max_tiles + 1, s));
-  DTRY(grouped_gemm(expert_act, e.effp, at<T>(e.w_down), e.ld_down, pad8(m.width), expert_out, m.width, m.width, e.eff, e.experts, a.tiles,
-                    a.max_tiles, s));
-  return moe_combine(a, expert_out, h, m.ldw, side + L.col_sg, L.n_side, shared, y2, m.width, n, s);
+  DTRY(experts_up(a, expert_in, m.ldw, at<T>(e.w_gu), m.ldw, m.width, e.effp, expert_act, expert_gu, s));
+  DTRY(experts_down(a, expert_act, e.effp, at<T>(e.w_down), e.ld_down, pad8(m.width), m.width, e.eff, expert_out, m.ldw, s));
+  return moe_combine(a, expert_out, m.ldw, h, m.ldw, side + L.col_sg, L.n_side, shared, y2, m.width, n, s);
 }
 
 // n <= max_portion rows at positions pos ..; `done` rows of the caller's portion came before.

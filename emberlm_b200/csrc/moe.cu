@@ -1,14 +1,15 @@
 // Mixture of experts over a prompt's portion: routing, the slots of every expert (padded to whole tiles of
 // the grouped product), gathering of the rows, and the weighted sum. An expert's rows may stand in any
 // order: every row is computed by itself.
+#include "decode_core.h"
 #include "hybrid_kernels.h"
 #include "moe_route.cuh"
 #include "parallel_kernels.h"
 
 namespace ctdk {
 
-int gemm_bf16_grouped(const void* A, int64_t lda, const void* B, int64_t ldb, int64_t n_pitch, float* C, int64_t ldc, int N, int K, int groups,
-                      const int32_t* tiles, int max_tiles, cudaStream_t stream);
+int gemm_bf16_out16(const void* A, int64_t lda, const void* B, int64_t ldb, __nv_bfloat16* C, int64_t ldc, int64_t M, int N, int K, int up_row,
+                    const int32_t* tiles, int max_tiles, int64_t n_pitch, int groups, cudaStream_t stream);
 
 namespace hybrid {
 namespace {
@@ -117,7 +118,7 @@ __global__ void __launch_bounds__(256) moe_gather_kernel(const MoeArgs a, const 
 
 template <typename T>
 __global__ void __launch_bounds__(256)
-    moe_combine_kernel(const MoeArgs a, const float* __restrict__ eo, const T* __restrict__ h, int64_t ld_h, const float* __restrict__ sg,
+    moe_combine_kernel(const MoeArgs a, const T* __restrict__ eo, int64_t ld_eo, const T* __restrict__ h, int64_t ld_h, const float* __restrict__ sg,
                        int64_t ld_sg, const float* __restrict__ shared, float* __restrict__ y, int width, int64_t rows) {
   pdl_launch();
   pdl_wait();
@@ -127,7 +128,7 @@ __global__ void __launch_bounds__(256)
       float v = shared != nullptr ? gate * shared[r * width + c] : 0.0f;
       for (int k = 0; k < a.top; ++k) {
         const int slot = a.slot[r * a.top + k];
-        const float u = slot < 0 ? to_f(h[r * ld_h + c]) : eo[static_cast<int64_t>(slot) * width + c];
+        const float u = to_f(slot < 0 ? h[r * ld_h + c] : eo[static_cast<int64_t>(slot) * ld_eo + c]);
         v = fmaf(a.weight[r * a.top + k], u, v);
       }
       y[r * width + c] = v;
@@ -136,7 +137,7 @@ __global__ void __launch_bounds__(256)
 }
 template <typename T>
 __global__ void __launch_bounds__(256)
-    moe_combine4_kernel(const MoeArgs a, const float* __restrict__ eo, const T* __restrict__ h, int64_t ld_h, const float* __restrict__ sg,
+    moe_combine4_kernel(const MoeArgs a, const T* __restrict__ eo, int64_t ld_eo, const T* __restrict__ h, int64_t ld_h, const float* __restrict__ sg,
                         int64_t ld_sg, const float* __restrict__ shared, float* __restrict__ y, int width, int64_t rows) {
   pdl_launch();
   pdl_wait();
@@ -152,7 +153,7 @@ __global__ void __launch_bounds__(256)
       for (int k = 0; k < a.top; ++k) {
         const int slot = a.slot[r * a.top + k];
         const float w = a.weight[r * a.top + k];
-        const float4 u = slot < 0 ? load4(h + r * ld_h + c) : load4(eo + static_cast<int64_t>(slot) * width + c);
+        const float4 u = load4(slot < 0 ? h + r * ld_h + c : eo + static_cast<int64_t>(slot) * ld_eo + c);
         v = make_float4(fmaf(w, u.x, v.x), fmaf(w, u.y, v.y), fmaf(w, u.z, v.z), fmaf(w, u.w, v.w));
       }
       store4(y + r * width + c, v);
@@ -212,6 +213,13 @@ __global__ void __launch_bounds__(256)
     if (rc_ != CTDK_OK) return rc_;                                                                              \
   } while (0)
 
+int grouped_simt(const MoeArgs& a, const float* A, int64_t lda, const float* W, int64_t ldw, int64_t n_pitch, float* C, int64_t ldc, int N,
+                 int K, cudaStream_t s) {
+  TRY_LAUNCH("grouped product (fp32)", grouped_simt_kernel, (static_cast<unsigned>((N + 63) / 64), static_cast<unsigned>(2 * a.max_tiles)), 256,
+             0, A, lda, W, ldw, n_pitch, C, ldc, N, K, a.tiles, a.max_tiles);
+  return CTDK_OK;
+}
+
 }  // namespace
 
 int moe_route(const MoeArgs& a, int64_t rows, cudaStream_t s) {
@@ -233,26 +241,35 @@ int moe_gather(const MoeArgs& a, const T* h, int64_t ld_h, T* xe, int width, int
   return CTDK_OK;
 }
 template <typename T>
-int moe_combine(const MoeArgs& a, const float* expert_out, const T* h, int64_t ld_h, const float* sg, int64_t ld_sg, const float* shared,
+int moe_combine(const MoeArgs& a, const T* expert_out, int64_t ld_eo, const T* h, int64_t ld_h, const float* sg, int64_t ld_sg, const float* shared,
                 float* y, int width, int64_t rows, cudaStream_t s) {
   auto* kernel = width % 4 == 0 ? moe_combine4_kernel<T> : moe_combine_kernel<T>;
-  TRY_LAUNCH("moe combine", kernel, (row_grid(rows)), 256, 0, a, expert_out, h, ld_h, sg, ld_sg, shared, y, width, rows);
+  TRY_LAUNCH("moe combine", kernel, (row_grid(rows)), 256, 0, a, expert_out, ld_eo, h, ld_h, sg, ld_sg, shared, y, width, rows);
   return CTDK_OK;
 }
-int grouped_gemm(const float* A, int64_t lda, const float* W, int64_t ldw, int64_t n_pitch, float* C, int64_t ldc, int N, int K, int,
-                 const int32_t* tiles, int max_tiles, cudaStream_t s) {
-  TRY_LAUNCH("grouped product (fp32)", grouped_simt_kernel, (static_cast<unsigned>((N + 63) / 64), static_cast<unsigned>(2 * max_tiles)), 256, 0,
-             A, lda, W, ldw, n_pitch, C, ldc, N, K, tiles, max_tiles);
-  return CTDK_OK;
+int experts_up(const MoeArgs& a, const float* xe, int64_t ld_x, const float* w, int64_t ldw, int K, int effp, float* act, float* scratch,
+               cudaStream_t s) {
+  DTRY(grouped_simt(a, xe, ld_x, w, ldw, 2 * effp, scratch, 2 * effp, 2 * effp, K, s));
+  return glu_rows(scratch, 2 * effp, act, effp, static_cast<int64_t>(a.max_tiles) * kMoeTile, effp, Glu::kSilu, a.tiles + a.max_tiles + 1, s);
 }
-int grouped_gemm(const __nv_bfloat16* A, int64_t lda, const __nv_bfloat16* W, int64_t ldw, int64_t n_pitch, float* C, int64_t ldc, int N, int K,
-                 int experts, const int32_t* tiles, int max_tiles, cudaStream_t s) {
-  return gemm_bf16_grouped(A, lda, W, ldw, n_pitch, C, ldc, N, K, experts, tiles, max_tiles, s);
+int experts_up(const MoeArgs& a, const __nv_bfloat16* xe, int64_t ld_x, const __nv_bfloat16* w, int64_t ldw, int K, int effp,
+               __nv_bfloat16* act, float*, cudaStream_t s) {
+  return gemm_bf16_out16(xe, ld_x, w, ldw, act, effp, static_cast<int64_t>(a.max_tiles) * kMoeTile, effp, K, effp, a.tiles, a.max_tiles,
+                         2 * effp, a.experts, s);
+}
+int experts_down(const MoeArgs& a, const float* act, int64_t ld_a, const float* w, int64_t ldw, int64_t n_pitch, int N, int K, float* out,
+                 int64_t ld_out, cudaStream_t s) {
+  return grouped_simt(a, act, ld_a, w, ldw, n_pitch, out, ld_out, N, K, s);
+}
+int experts_down(const MoeArgs& a, const __nv_bfloat16* act, int64_t ld_a, const __nv_bfloat16* w, int64_t ldw, int64_t n_pitch, int N, int K,
+                 __nv_bfloat16* out, int64_t ld_out, cudaStream_t s) {
+  return gemm_bf16_out16(act, ld_a, w, ldw, out, ld_out, static_cast<int64_t>(a.max_tiles) * kMoeTile, N, K, 0, a.tiles, a.max_tiles, n_pitch,
+                         a.experts, s);
 }
 
 #define INSTANTIATE(T)                                                                                                            \
   template int moe_gather<T>(const MoeArgs&, const T*, int64_t, T*, int, int64_t, cudaStream_t);                                  \
-  template int moe_combine<T>(const MoeArgs&, const float*, const T*, int64_t, const float*, int64_t, const float*, float*, int, \
+  template int moe_combine<T>(const MoeArgs&, const T*, int64_t, const T*, int64_t, const float*, int64_t, const float*, float*, int, \
                               int64_t, cudaStream_t);
 INSTANTIATE(float)
 INSTANTIATE(__nv_bfloat16)

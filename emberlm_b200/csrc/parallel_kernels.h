@@ -87,10 +87,6 @@ int latent_attention_fp32(const LatentArgs<T>& a, int64_t first, int64_t rows, c
 bool latent_tcgen05_ok(int dim, int rot_dim, int vdim);
 int latent_attention_tcgen05(const LatentArgs<__nv_bfloat16>& a, int64_t first, int64_t rows, cudaStream_t s);
 
-// dst = T(src) for rows of n columns
-template <typename T>
-int cast_rows(const float* src, int64_t lds, T* dst, int64_t ldd, int64_t rows, int n, cudaStream_t s);
-
 // ---- time mixing ----
 // dst[t][c] = tanh(src[t][c]), zero up to ldd
 template <typename T>
@@ -144,15 +140,21 @@ int moe_route(const MoeArgs& a, int64_t rows, cudaStream_t s);
 // xe[slot] = h[row]
 template <typename T>
 int moe_gather(const MoeArgs& a, const T* h, int64_t ld_h, T* xe, int width, int64_t rows, cudaStream_t s);
+// act[slot] = silu(gate) up of the slot's expert: 2 * effp rows of w per expert (gate rows, then up rows), K
+// columns. scratch (fp32 models): [slots, 2 * effp].
+int experts_up(const MoeArgs& a, const float* xe, int64_t ld_x, const float* w, int64_t ldw, int K, int effp, float* act, float* scratch,
+               cudaStream_t s);
+int experts_up(const MoeArgs& a, const __nv_bfloat16* xe, int64_t ld_x, const __nv_bfloat16* w, int64_t ldw, int K, int effp,
+               __nv_bfloat16* act, float* scratch, cudaStream_t s);
+// out[slot] = the down product of the slot's expert: n_pitch rows of w per expert, of which N count, K columns.
+int experts_down(const MoeArgs& a, const float* act, int64_t ld_a, const float* w, int64_t ldw, int64_t n_pitch, int N, int K, float* out,
+                 int64_t ld_out, cudaStream_t s);
+int experts_down(const MoeArgs& a, const __nv_bfloat16* act, int64_t ld_a, const __nv_bfloat16* w, int64_t ldw, int64_t n_pitch, int N, int K,
+                 __nv_bfloat16* out, int64_t ld_out, cudaStream_t s);
 // y[row] = sum weight * (expert_out[slot] or h[row]) + sigmoid(sg) * shared
 template <typename T>
-int moe_combine(const MoeArgs& a, const float* expert_out, const T* h, int64_t ld_h, const float* sg, int64_t ld_sg, const float* shared,
-                float* y, int width, int64_t rows, cudaStream_t s);
-// C[tile rows] = A[tile rows] W[expert of the tile]^T; W has n_pitch rows of ldw elements per expert.
-int grouped_gemm(const __nv_bfloat16* A, int64_t lda, const __nv_bfloat16* W, int64_t ldw, int64_t n_pitch, float* C, int64_t ldc, int N, int K,
-                 int experts, const int32_t* tiles, int max_tiles, cudaStream_t s);
-int grouped_gemm(const float* A, int64_t lda, const float* W, int64_t ldw, int64_t n_pitch, float* C, int64_t ldc, int N, int K, int experts,
-                 const int32_t* tiles, int max_tiles, cudaStream_t s);
+int moe_combine(const MoeArgs& a, const T* expert_out, int64_t ld_eo, const T* h, int64_t ld_h, const float* sg, int64_t ld_sg,
+                const float* shared, float* y, int width, int64_t rows, cudaStream_t s);
 
 #ifdef __CUDACC__
 __device__ __forceinline__ float gelu_tanh_f(float z) { return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z))); }

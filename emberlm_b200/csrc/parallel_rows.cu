@@ -165,8 +165,8 @@ __global__ void __launch_bounds__(256) glu_kernel(const float* __restrict__ gu, 
   }
 }
 
-template <typename T, bool TANH>
-__global__ void __launch_bounds__(256) map_rows_kernel(const float* __restrict__ src, int64_t lds, T* __restrict__ dst, int64_t ldd,
+template <typename T>
+__global__ void __launch_bounds__(256) tanh_rows_kernel(const float* __restrict__ src, int64_t lds, T* __restrict__ dst, int64_t ldd,
                                                        int64_t rows, int n) {
   pdl_launch();
   pdl_wait();
@@ -174,24 +174,9 @@ __global__ void __launch_bounds__(256) map_rows_kernel(const float* __restrict__
   for (int64_t i = static_cast<int64_t>(blockIdx.x) * 256 + threadIdx.x; i < total; i += static_cast<int64_t>(gridDim.x) * 256) {
     const int64_t r = i / n;
     const int c = static_cast<int>(i % n);
-    const float v = src[r * lds + c];
-    dst[r * ldd + c] = from_f<T>(TANH ? tanhf(v) : v);
+    dst[r * ldd + c] = from_f<T>(tanhf(src[r * lds + c]));
   }
 }
-template <typename T>
-__global__ void __launch_bounds__(256) cast_rows4_kernel(const float* __restrict__ src, int64_t lds, T* __restrict__ dst, int64_t ldd,
-                                                         int64_t rows, int n) {
-  pdl_launch();
-  pdl_wait();
-  const int per = n / 4;
-  const int64_t total = rows * per;
-  for (int64_t i = static_cast<int64_t>(blockIdx.x) * 256 + threadIdx.x; i < total; i += static_cast<int64_t>(gridDim.x) * 256) {
-    const int64_t r = i / per;
-    const int c = static_cast<int>(i % per) * 4;
-    store4(dst + r * ldd + c, load4(src + r * lds + c));
-  }
-}
-
 // One warp per (row, head).
 template <typename T>
 __global__ void __launch_bounds__(256)
@@ -256,14 +241,8 @@ int glu_rows(const float* gu, int64_t ldg, T* act, int64_t lda, int64_t rows, in
   LAUNCH("silu glu", (glu_kernel<T, false>), grid, 0, gu, ldg, act, lda, rows, ffp, rows_dev);
 }
 template <typename T>
-int cast_rows(const float* src, int64_t lds, T* dst, int64_t ldd, int64_t rows, int n, cudaStream_t s) {
-  if (n % 4 == 0 && lds % 4 == 0 && ldd % 4 == 0)
-    LAUNCH("cast rows", cast_rows4_kernel<T>, row_grid(rows * (n / 4), 256), 0, src, lds, dst, ldd, rows, n);
-  LAUNCH("cast rows", (map_rows_kernel<T, false>), row_grid(rows * n, 256), 0, src, lds, dst, ldd, rows, n);
-}
-template <typename T>
 int tanh_rows(const float* src, int64_t lds, T* dst, int64_t ldd, int64_t rows, int n, cudaStream_t s) {
-  LAUNCH("tanh rows", (map_rows_kernel<T, true>), row_grid(rows * n, 256), 0, src, lds, dst, ldd, rows, n);
+  LAUNCH("tanh rows", tanh_rows_kernel<T>, row_grid(rows * n, 256), 0, src, lds, dst, ldd, rows, n);
 }
 template <typename T>
 int silu_head_norm_rows(const float* o, const float* w, const float* gate, int64_t ldg, T* dst, int64_t ld, int64_t rows, int H, int dim,
@@ -274,7 +253,6 @@ int silu_head_norm_rows(const float* o, const float* w, const float* gate, int64
 #define INSTANTIATE(T)                                                                                                               \
   template int shift_norm_rows<T>(const ShiftNormArgs<T>&, int64_t, cudaStream_t);                                                   \
   template int glu_rows<T>(const float*, int64_t, T*, int64_t, int64_t, int, Glu, const int32_t*, cudaStream_t);                     \
-  template int cast_rows<T>(const float*, int64_t, T*, int64_t, int64_t, int, cudaStream_t);                                         \
   template int tanh_rows<T>(const float*, int64_t, T*, int64_t, int64_t, int, cudaStream_t);                                         \
   template int silu_head_norm_rows<T>(const float*, const float*, const float*, int64_t, T*, int64_t, int64_t, int, int, float,      \
                                       cudaStream_t);
