@@ -788,6 +788,8 @@ int gemm_bf16_tcgen05(const void* A, const void* B, float* Cp, int64_t M, int64_
   int bn, splits;
   bool use_pair;
   choose_tile(M, N, k_blocks, &bn, &splits, &use_pair);
+  if (bn == 64 && splits == 1)   // one narrow column of tiles (low-rank factors): split K while SMs are idle
+    while ((M + BM - 1) / BM * splits * 2 <= sm_budget() && k_blocks / (splits * 2) >= 8) splits *= 2;
   auto map_bf16 = [](CUtensorMap* map, const void* base, int64_t inner, int64_t outer, int64_t ld, int box_rows) {
     const uint64_t dims[2] = {static_cast<uint64_t>(inner), static_cast<uint64_t>(outer)}, strides[1] = {static_cast<uint64_t>(ld) * 2};
     const uint32_t box[2] = {static_cast<uint32_t>(BKH), static_cast<uint32_t>(box_rows)};

@@ -309,7 +309,7 @@ def test_trace_replay(folder, tmp_path, dtype):
         assert hc.error(got, want) <= lim, step
 
 
-@pytest.mark.parametrize("M,N,K", [(1, 8, 8), (2, 1000, 24), (130, 136, 72), (257, 512, 64), (300, 260, 1000), (512, 1024, 4096), (1000, 72, 136)])
+@pytest.mark.parametrize("M,N,K", [(1, 8, 8), (2, 1000, 24), (130, 136, 72), (257, 512, 64), (300, 260, 1000), (512, 1024, 4096), (1000, 72, 136), (1000, 64, 2048)])
 def test_bf16_product(M, N, K):
     """Small integers are exact in bfloat16 and in the fp32 sums: any misplaced tile shows as a wrong integer."""
     gen = torch.Generator(device="cuda").manual_seed(M + N + K)
